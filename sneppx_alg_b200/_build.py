@@ -33,6 +33,15 @@ NVCC_FLAGS = [
     "--use_fast_math", "-Xcompiler", "-fPIC", "-Xcompiler", "-fvisibility=default",
     "--expt-relaxed-constexpr",
 ]
+# Sources whose arithmetic follows IEEE single precision (no approximate division / square root / exponential, no
+# flush of denormals): recurrent state and the paths that also run models in 32-bit.
+PRECISE_SOURCES = {"decoder_ops.cu", "recurrence.cu", "talking_attn.cu"}
+
+# Named subsets of the sources for programs that need only part of the library; each is linked on its own.
+CUDA_SUBSETS = {
+    "hybrid": ("decoder_ops.cu", "recurrence.cu", "talking_attn.cu", "gemm_tc.cu", "gemm_skinny.cu"),
+}
+
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-pthread", "-Wall", "-Wno-unused-function"]
 
 _lock = threading.Lock()
@@ -88,7 +97,7 @@ def _compile_objects(compiler, flags, sources, headers, tag, verbose):
     for src in sources:
         obj = OBJDIR / f"{tag}_{src.stem}.o"
         stamp = OBJDIR / f"{tag}_{src.stem}.hash"
-        want = _hash_files([src], [hdr_hash])
+        want = _hash_files([src], [hdr_hash, src.name in PRECISE_SOURCES])
         objs.append(obj)
         if obj.exists() and stamp.exists() and stamp.read_text() == want:
             continue
@@ -96,7 +105,8 @@ def _compile_objects(compiler, flags, sources, headers, tag, verbose):
 
     def one(job):
         src, obj, stamp, want = job
-        out = _run([compiler, *flags, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
+        use = [f for f in flags if f != "--use_fast_math"] if src.name in PRECISE_SOURCES else flags
+        out = _run([compiler, *use, "-I", str(CSRC), "-c", str(src), "-o", str(obj)])
         stamp.write_text(want)
         if verbose:
             print(f"[sneppx build] {src.name}", file=sys.stderr)
@@ -109,19 +119,30 @@ def _compile_objects(compiler, flags, sources, headers, tag, verbose):
     return objs
 
 
-def build_cuda(force: bool = False, verbose: bool = False) -> Path:
-    """Compile every ``csrc/*.cu`` for sm_100a and link ``libsneppx_b200.so``."""
+def _current(lib: Path, stamp: Path, want: str) -> bool:
+    return lib.exists() and stamp.exists() and stamp.read_text() == want
+
+
+def build_cuda(force: bool = False, verbose: bool = False, subset: str | None = None) -> Path:
+    """Compile every ``csrc/*.cu`` for sm_100a and link ``libsneppx_b200.so``. ``subset`` (a key of ``CUDA_SUBSETS``)
+    compiles and links only those sources, unless the full library is there and current."""
     LIBDIR.mkdir(parents=True, exist_ok=True)
     lib = LIBDIR / "libsneppx_b200.so"
     stamp = LIBDIR / "libsneppx_b200.hash"
-    want = _hash_files(cuda_sources() + cuda_headers(), NVCC_FLAGS)
-    if not force and lib.exists() and stamp.exists() and stamp.read_text() == want:
+    sources = cuda_sources()
+    flags_key = [*NVCC_FLAGS, *sorted(PRECISE_SOURCES)]
+    want = _hash_files(sources + cuda_headers(), flags_key)
+    if subset is not None and not _current(lib, stamp, want):
+        sources = [s for s in sources if s.name in CUDA_SUBSETS[subset]]
+        lib, stamp = LIBDIR / f"libsneppx_b200_{subset}.so", LIBDIR / f"libsneppx_b200_{subset}.hash"
+        want = _hash_files(sources + cuda_headers(), flags_key)
+    if not force and _current(lib, stamp, want):
         return lib
     nvcc = _nvcc()
     if nvcc is None:
         raise RuntimeError("nvcc not found: cannot build libsneppx_b200.so")
     flags = list(NVCC_FLAGS) + (["-Xptxas", "-v"] if verbose else [])
-    objs = _compile_objects(nvcc, flags, cuda_sources(), cuda_headers(), "cu", verbose)
+    objs = _compile_objects(nvcc, flags, sources, cuda_headers(), "cu", verbose)
     _run([nvcc, "-shared", "-o", str(lib), *map(str, objs), "-lcudart"])
     stamp.write_text(want)
     return lib
@@ -171,14 +192,15 @@ def build_all(force: bool = False, verbose: bool = False):
     return build_cuda(force, verbose), build_host(force, verbose)
 
 
-def load_cuda() -> ctypes.CDLL:
-    """Return the CUDA kernel library, building it first when the sources changed."""
+def load_cuda(subset: str | None = None) -> ctypes.CDLL:
+    """Return the CUDA kernel library, building it first when the sources changed. ``subset``: see ``build_cuda``; it
+    only matters for the first load of a process."""
     global _cuda_lib
     with _lock:
         if _cuda_lib is None:
             lib = LIBDIR / "libsneppx_b200.so"
             try:
-                lib = build_cuda()
+                lib = build_cuda(subset=subset)
             except RuntimeError as e:
                 if not lib.exists():
                     raise

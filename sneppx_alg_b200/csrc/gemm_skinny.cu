@@ -30,10 +30,11 @@ struct SkinnyParams {
   CUtensorMap tmW, tmX;
   void* D;
   const float* bias;
+  const float* C;   // optional fp32 addend (beta * C), same indexing as D; may be D itself
   int* status;
-  long long ldd;
+  long long ldd, ldc;
   int M, N, K, Mpad, stages, tmem_cols, out_fp32, act, flags;
-  float alpha;
+  float alpha, beta, act_a, act_b;
 };
 
 __device__ __forceinline__ uint32_t cluster_rank() {
@@ -66,12 +67,14 @@ __device__ __forceinline__ float4 ld_dsmem_f32x4(uint32_t local_addr, uint32_t r
   return v;
 }
 
-__device__ __forceinline__ float skinny_epilogue(float v, const SkinnyParams& p, int n) {
+__device__ __forceinline__ float skinny_epilogue(float v, const SkinnyParams& p, int m, int n) {
   v *= p.alpha;
   if (p.bias) v += p.bias[n];
+  if (p.C) v += p.beta * p.C[(long long)m * p.ldc + n];
   if (p.act == 1) v = gelu_tanh(v);
   else if (p.act == 2) v = silu(v);
   else if (p.act == 3) v = fmaxf(v, 0.f);
+  else if (p.act == 4) v = xielu(v, p.act_a, p.act_b);
   return v;
 }
 __device__ __forceinline__ void skinny_store(const SkinnyParams& p, int m, int n, float v) {
@@ -205,7 +208,7 @@ __global__ void __launch_bounds__(SK_THREADS, 2) gemm_skinny_kernel(const __grid
       float o[4] = {acc.x, acc.y, acc.z, acc.w};
 #pragma unroll
       for (int j = 0; j < 4; ++j)
-        if (n + j < p.N) o[j] = skinny_epilogue(o[j], p, n + j);
+        if (n + j < p.N) o[j] = skinny_epilogue(o[j], p, m, n + j);
       if (vec_ok) {
         if (p.out_fp32) {
           *reinterpret_cast<float4*>(reinterpret_cast<float*>(p.D) + (long long)m * p.ldd + n) =
@@ -237,7 +240,7 @@ __global__ void __launch_bounds__(SK_THREADS, 2) gemm_skinny_kernel(const __grid
 }  // namespace sx
 using namespace sx;
 
-// 1 when the product is one this kernel takes: plain [M<=128, K] x [N, K]^T, both K-major, no addend.
+// 1 when the product is one this kernel takes: plain [M<=128, K] x [N, K]^T, both K-major, addend fp32 or none.
 extern "C" int sx_gemm_skinny_ok(const SxGemmArgs* a) {
   static int enabled = -1;
   if (enabled < 0) {
@@ -245,7 +248,7 @@ extern "C" int sx_gemm_skinny_ok(const SxGemmArgs* a) {
     enabled = e ? atoi(e) : 1;
   }
   return enabled && a->M >= 1 && a->M <= 128 && a->N >= 128 && a->K >= 256 && a->batch == 1 && !a->a_mn && !a->b_mn &&
-         !(a->C && a->beta != 0.f) && !a->tile_group && !a->k_ranges && a->sm_limit == 0 && a->force_bn == 0;
+         !(a->C && a->beta != 0.f && !a->c_fp32) && !a->tile_group && !a->k_ranges && a->sm_limit == 0 && a->force_bn == 0;
 }
 
 // Cluster size (1, 2, 4 or 8): fill the machine in as few waves as possible; cost of a CTA = its K blocks + a fixed
@@ -301,6 +304,8 @@ extern "C" int sx_gemm_skinny(const SxGemmArgs* a, cudaStream_t st) {
   p.tmem_cols = p.Mpad <= 32 ? 32 : (p.Mpad <= 64 ? 64 : 128);
   p.D = a->D; p.bias = a->bias; p.status = a->status; p.ldd = a->ldd;
   p.M = a->M; p.N = a->N; p.K = a->K; p.out_fp32 = a->out_fp32; p.act = a->act; p.alpha = a->alpha;
+  p.C = a->beta != 0.f ? (const float*)a->C : nullptr;
+  p.ldc = a->ldc; p.beta = a->beta; p.act_a = a->act_a; p.act_b = a->act_b;
   p.flags = a->flags;
   const int smem = stages * stage_bytes + 1024 + 1024;
   static int smem_set = 0;

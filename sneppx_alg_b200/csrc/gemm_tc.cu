@@ -81,7 +81,7 @@ struct GemmKernelParams {
   int M, N, K, batch;
   int a_batched, b_batched;
   int out_fp32, c_fp32, act;
-  float alpha, beta;
+  float alpha, beta, act_a, act_b;
   int m_blks, n_blks;
   CommParams cm;
 };
@@ -518,6 +518,9 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_tc_kernel(const __grid_c
         } else if (p.act == 3) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.f);
+        } else if (p.act == 4) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = xielu(v[j], p.act_a, p.act_b);
         }
         if (COMM == 2) {
           // this lane's 64 bytes of the row go to the warp's slab: 16-byte chunk index XOR row keeps both the writes
@@ -922,6 +925,9 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
         } else if (p.act == 3) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = fmaxf(v[j], 0.f);
+        } else if (p.act == 4) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = xielu(v[j], p.act_a, p.act_b);
         }
         if (p.out_fp32) {
           float* dp = reinterpret_cast<float*>(p.D) + drow + col0;
@@ -1062,6 +1068,7 @@ static int gemm_launch(const SxGemmArgs* a, const SxGemmCommArgs* cm, cudaStream
     kp.M = a->M; kp.N = a->N; kp.K = a->K; kp.batch = a->batch;
     kp.a_batched = a_batched; kp.b_batched = bb2;
     kp.out_fp32 = a->out_fp32; kp.c_fp32 = a->c_fp32; kp.act = a->act; kp.alpha = a->alpha; kp.beta = a->beta;
+    kp.act_a = a->act_a; kp.act_b = a->act_b;
     kp.m_blks = (a->M + 255) / 256; kp.n_blks = (a->N + bn2 - 1) / bn2;
     const int am2 = a->a_mn != 0, bm2 = a->b_mn != 0;
     return bn2 == 256 ? launch_cfg2_any<256>(kp, am2, bm2, sms2, st) : launch_cfg2_any<128>(kp, am2, bm2, sms2, st);
@@ -1091,6 +1098,8 @@ static int gemm_launch(const SxGemmArgs* a, const SxGemmCommArgs* cm, cudaStream
   kp.act = a->act;
   kp.alpha = a->alpha;
   kp.beta = a->beta;
+  kp.act_a = a->act_a;
+  kp.act_b = a->act_b;
   kp.m_blks = (a->M + BM - 1) / BM;
   kp.n_blks = (a->N + BN - 1) / BN;
   int dev = 0, sms = 148;

@@ -22,7 +22,7 @@ typedef struct SxGemmArgs {
   long long strideA, strideB, strideD, strideC;  // batch strides in elements (0: operand shared)
   int a_mn, b_mn;
   int out_fp32, c_fp32;
-  int act;  // 0 none, 1 gelu(tanh), 2 silu, 3 relu
+  int act;  // 0 none, 1 gelu(tanh), 2 silu, 3 relu, 4 xIELU with coefficients act_a (z > 0) and act_b (z <= 0)
   float alpha, beta;
   const int* tile_group;  // grouped GEMM: per 128-row block of A, index of the B matrix (-1 skips the block)
   int num_groups;         // number of B matrices when tile_group is set
@@ -33,6 +33,7 @@ typedef struct SxGemmArgs {
   int force_bn;  // 0 auto, 128 or 256
   int flags;     // bit 0: B is not written by any kernel launched before this one on the stream (a weight at
                  // inference time), so a kernel may start fetching it before its predecessor has finished
+  float act_a, act_b;
 } SxGemmArgs;
 int sx_gemm_bf16(const SxGemmArgs* args, cudaStream_t stream);
 
@@ -217,6 +218,102 @@ int sx_gemm_fp8(const void* xq, long long ldx, const float* sx, const void* wq, 
 int sx_gemm_fp8_grouped(const void* xq, long long ldx, const float* sx, const void* wq, long long ldw, const float* sw,
                         const int* tile_group, int num_experts, void* out, long long ldd, int rows, int N, int K,
                         int* status, cudaStream_t stream);
+
+// ------------------------------------------------------------------ hybrid decoders (ragged batches, fp32 residual)
+// Rows of several sequences, one portion each, packed one after another. Device int32 arrays.
+typedef struct SxRagged {
+  const int* cu;        // [n + 1] first row of each portion
+  const int* pos0;      // [n] position of that row in its sequence; 0 starts from an empty state
+  const int* slot;      // [n] state slot (-1: padding row of a captured launch)
+  const int* tok_seq;   // [T] portion of each row
+  const int* tok_pos;   // [T] position of each row
+  int n;
+} SxRagged;
+// f32: 1 for 32-bit activations, 0 for bf16. Norm weights, convolution weights and biases are fp32.
+int sx_embed_f32(const void* table, const int* ids, float* x, int T, int width, int f32, cudaStream_t stream);
+int sx_rmsnorm_f32(const float* x, const float* w, const int* rows, void* y, int T, int width, float eps, int f32, cudaStream_t stream);
+int sx_head_norm_gate(const float* o, const float* w, const void* gate, long long gate_ld, float mul, void* y, long long y_ld,
+                      int T, int H, int dv, float eps, int f32, cudaStream_t stream);
+// Stores the last min(length, taps - 1) projected rows of every portion: ring [slots, taps, C], position p in entry p % taps.
+int sx_conv_ring(const void* u, long long u_ld, void* ring, const SxRagged* r, int C, int taps, int f32, cudaStream_t stream);
+// Attention operands from projected rows u = q [H d] | k [G d] | v [G dv]: causal convolution over time, RMSNorm of the query
+// and key heads, interleaved rotation of their first `rot` entries, cache append.
+typedef struct SxQkvArgs {
+  const void* u; long long u_ld;
+  const float* wconv;             // [taps, C], C = H d + G d + G dv
+  void* ring;
+  const float* qn; const float* kn;
+  const double* inv_freq;         // [rot / 2]
+  const float* talk;              // [H, H], with qmix_out
+  float* q_out;                   // [T, H, d] or null
+  void* qmix_out;                 // [T, H, G d] queries with the head mix folded in, or null
+  void* k_out; void* v_out;       // packed keys / values, or null; value head j at column j * dvp
+  long long k_ld, v_ld;
+  const int* kv_row;              // [T] packed row (null: row index)
+  void* k_cache; void* v_cache;   // [entries, G, d] / [entries, G, dv]
+  const int* cache_entry;         // [T], -1: not stored
+  SxRagged ragged;
+  int T, H, G, d, dv, dvp, taps, rot, write_ring, f32;
+  float eps;
+} SxQkvArgs;
+int sx_qkv_prep(const SxQkvArgs* args, cudaStream_t stream);
+int sx_kv_gather(const void* cache, const int* entry, const int* row, int n, void* out, long long out_ld, int G, int w, int wp,
+                 int f32, cudaStream_t stream);
+// Delta-rule operands from projected rows u = q [G d] | k [G d] | v [H dv].
+typedef struct SxDeltaArgs {
+  const void* u; long long u_ld;
+  const float* wconv; void* ring;
+  const void* b; long long b_ld;
+  const void* a; long long a_ld;
+  const float* a_log; const float* dt_bias;
+  float* q; float* k; float* g; void* v; float* beta;
+  SxRagged ragged;
+  int T, H, G, d, dv, taps, write_ring, f32;
+} SxDeltaArgs;
+int sx_delta_prep(const SxDeltaArgs* args, cudaStream_t stream);
+int sx_gate_prep(const void* qr, const void* fr, long long ld, const float* bias, const float* lower, float* q, float* f, int T,
+                 int C, int f32, cudaStream_t stream);
+// Scan of a portion; state [slots, H, d, dv] fp32, o [T, H, dv] fp32. Head h reads q / k head h / (H / Hq).
+typedef struct SxScanArgs {
+  const float* q; const float* g; const float* k;
+  const void* v; long long v_ld;
+  const float* beta;
+  float* state; float* o;
+  SxRagged ragged;
+  int H, Hq, d, dv, delta, f32;
+} SxScanArgs;
+int sx_recur_scan(const SxScanArgs* args, cudaStream_t stream);
+// One token per sequence, from the projected rows to the normed and gated output row.
+typedef struct SxStepArgs {
+  SxDeltaArgs in;
+  const void* qr; const void* fr; const void* vr; long long ld;
+  const float* fbias; const float* lower;
+  float* state; const float* norm;
+  const void* gate; long long gate_ld;
+  void* y; long long y_ld;
+  SxRagged ragged;
+  float mul, eps;
+  int H, Hq, d, dv, delta, f32;
+} SxStepArgs;
+int sx_recur_step(const SxStepArgs* args, cudaStream_t stream);
+// Attention whose scores are mixed over the heads before the softmax (score_h <- sum_g talk[h, g] score_g), restricted to
+// the chunk floor(position / size) of each query. SIMT form for any head size: q fp32 [T, H, d]. Keys either packed rows
+// (kv_base[seq] + position) or cache entries through a block table. Output y = o * sigmoid(gate) * mul.
+typedef struct SxTalkArgs {
+  const float* q;
+  const void* k; const void* v;
+  long long k_ld, v_ld; int dvp;
+  const int* kv_base;             // packed form: [n] row of position 0 of each sequence (may be negative)
+  const int* block_table; const int* block_base; int table_ld, block_size;   // paged form (block_table non-null)
+  const float* talk;              // [H, H]
+  const void* gate; long long gate_ld;
+  void* y; long long y_ld;
+  SxRagged ragged;
+  float scale, mul;
+  int T, H, G, d, dv, size, f32;
+  float* part; int splits;        // decode: partial results of key splits [n, splits, H, dv + 2]
+} SxTalkArgs;
+int sx_talk_attn(const SxTalkArgs* args, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

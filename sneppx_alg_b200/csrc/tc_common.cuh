@@ -265,6 +265,10 @@ __device__ __forceinline__ float gelu_tanh(float x) {
   const float k0 = 0.7978845608028654f, k1 = 0.044715f;
   return 0.5f * x * (1.f + tanhf(k0 * (x + k1 * x * x * x)));
 }
+// xIELU: a z^2 + z / 2 above zero, b (e^z - 1 - z) + z / 2 below; a and b are the softplus-transformed coefficients.
+__device__ __forceinline__ float xielu(float z, float a, float b) {
+  return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
+}
 __device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
 
 }  // namespace sx

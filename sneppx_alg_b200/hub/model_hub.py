@@ -13,7 +13,7 @@ from typing import Dict, List, Optional
 import torch
 
 from ..checkpoint.sneppx_format import load_tensors, save_tensors
-from ..models import ModelConfig, build_model, config_from_name
+from ..models import ModelConfig, build_model, complete_config, config_from_name
 from .formats import load_safetensors, save_safetensors
 
 HF_WEIGHT_MAP = [
@@ -88,9 +88,9 @@ class ModelHub:
     @staticmethod
     def from_pretrained(directory: str, dtype=None, device=None):
         cfg = ModelConfig.from_json(os.path.join(directory, "config.json"))
-        model = build_model(cfg, dtype=dtype, device=device)
         st = os.path.join(directory, "model.safetensors")
         sd = load_safetensors(st)[0] if os.path.exists(st) else load_tensors(os.path.join(directory, "model.sneppx"))[0]
+        model = build_model(complete_config(cfg, sd), dtype=dtype, device=device)
         if any(k.startswith("model.layers.") for k in sd):     # raw Hugging Face names
             sd = {map_hf_name(k): v for k, v in sd.items() if map_hf_name(k)}
             sd.setdefault("lm_head", sd.get("embedding"))

@@ -18,4 +18,15 @@ def build_model(cfg, dtype=None, device=None):
     if arch == "deepseek_moe":
         from .deepseek import DeepSeekV2ForCausalLM
         return DeepSeekV2ForCausalLM(cfg, dtype=dtype, device=device)
+    if arch == "rilenex":
+        from .rilenex import RilenexForCausalLM
+        return RilenexForCausalLM(cfg, dtype=dtype, device=device)
     raise ValueError(f"unknown architecture '{arch}'")
+
+
+def complete_config(cfg, tensors):
+    """Fill in the sizes that a checkpoint gives only through its tensors' shapes (a no-op for most families)."""
+    if cfg.architecture == "rilenex":
+        from .rilenex import RilenexForCausalLM
+        return RilenexForCausalLM.config_from_tensors(cfg, tensors)
+    return cfg

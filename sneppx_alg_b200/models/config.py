@@ -10,7 +10,15 @@ from __future__ import annotations
 import dataclasses
 import json
 from dataclasses import dataclass, field
-from typing import Any, Dict, Optional
+from typing import Any, Dict, List, Optional
+
+
+def _rilenex_fields(d: Dict[str, Any]) -> Dict[str, Any]:
+    """The keys of a Rilenex ``config.json`` under this schema's names; other keys pass through."""
+    out = {k: v for k, v in d.items() if k not in ("layers", "vocab", "width", "norm")}
+    out.update(architecture="rilenex", layer_specs=d["layers"], vocab_size=d["vocab"], hidden_size=d["width"],
+               rms_norm_eps=d["norm"]["eps"], num_hidden_layers=len(d["layers"]))
+    return out
 
 
 @dataclass
@@ -23,7 +31,7 @@ class ModelConfig:
     license: str = ""
     repository: str = ""
     homepage: str = ""
-    architecture: str = "transformer"   # transformer | mamba2 | hss_ser | deepseek_moe | bert | gpt | t5 | vit
+    architecture: str = "transformer"   # transformer | mamba2 | hss_ser | deepseek_moe | rilenex | bert | gpt | t5 | vit
     model_type: str = "causal-lm"
     framework: str = "sneppx"
     # shape
@@ -98,6 +106,8 @@ class ModelConfig:
     ssm_ngroups: int = 1
     ssm_conv_kernel: int = 4
     ssm_chunk_size: int = 256
+    # per-layer specifications of hybrid decoders: {"type", "mixer": {sizes}, "mlp": {sizes} or None}
+    layer_specs: List[dict] = field(default_factory=list)
     custom: Dict[str, Any] = field(default_factory=dict)
 
     def __post_init__(self):
@@ -127,6 +137,8 @@ class ModelConfig:
 
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "ModelConfig":
+        if str(d.get("architecture", "")).lower() == "rilenex" and "layers" in d:
+            d = _rilenex_fields(d)
         names = {f.name for f in dataclasses.fields(cls)}
         known = {k: v for k, v in d.items() if k in names}
         extra = {k: v for k, v in d.items() if k not in names}
@@ -157,6 +169,8 @@ class ModelConfig:
 
     def estimate_parameters(self) -> int:
         d, L, V = self.hidden_size, self.num_hidden_layers, self.vocab_size
+        if self.architecture == "rilenex":
+            return _rilenex_parameters(self)
         hd = self.head_dim or 0
         attn = d * (self.num_attention_heads + 2 * self.num_key_value_heads) * hd + self.num_attention_heads * hd * d
         ffn = (3 if self.gated_ffn else 2) * d * self.intermediate_size
@@ -173,6 +187,26 @@ class ModelConfig:
             total = L * (attn + ffn)
         emb = V * d * (1 if self.tie_word_embeddings else 2)
         return total + emb + (2 * L + 1) * d
+
+
+def _rilenex_parameters(cfg: ModelConfig) -> int:
+    d, total = cfg.hidden_size, (2 * cfg.vocab_size + 1) * cfg.hidden_size
+    for s in cfg.layer_specs:
+        m = s["mixer"]
+        if s["type"] == "hgrn2":
+            H, k, v = m["heads"], m["dim"], m["vdim"]
+            total += d * H * (2 * k + 2 * v) + 2 * H * k + v + d
+        else:
+            a, r = m["left"], m["right"]
+            c = a["heads"] * a["dim"] + a["kv_heads"] * (a["dim"] + a["vdim"])
+            total += d * (c + a["heads"] * (1 + a["vdim"])) + a["conv"] * c + a["heads"] ** 2 + 2 * a["dim"]
+            H, k, v = r["heads"], r["dim"], r["vdim"]
+            c = 2 * r["kv_heads"] * k + H * v
+            ra, rg = r.get("decay_rank", k), r.get("gate_rank", k)
+            total += d * (c + H + ra + rg + H * v) + r["conv"] * c + ra * H * k + rg * H * v + H * (k + 1) + v + d
+        if s.get("mlp") is not None:
+            total += 2 * d * s["mlp"]["ff"] + d + 2
+    return total
 
 
 class LlamaConfig(ModelConfig):
@@ -253,6 +287,31 @@ _MODEL_REGISTRY: Dict[str, Dict[str, dict]] = {
     },
 }
 
+
+
+def _rilenex(width, ff, vocab, groups, hgrn2, left, right, max_len=131072):
+    """Layer pattern of the presets: ``groups`` times two recurrent layers followed by one parallel layer."""
+    mlp = {"kind": "dense", "ff": ff}
+    h = {"type": "hgrn2", "mixer": hgrn2, "mlp": mlp}
+    p = {"type": "parallel", "mlp": mlp, "mixer": {"left": left, "right": right, "left_scale": 1.0, "right_scale": 1.0}}
+    return dict(architecture="rilenex", hidden_size=width, vocab_size=vocab, layer_specs=[h, h, p] * groups,
+                num_hidden_layers=3 * groups, max_position_embeddings=max_len, rms_norm_eps=1e-5)
+
+
+_MODEL_REGISTRY["rilenex"] = {
+    "tiny": _rilenex(128, 256, 512, 1, dict(heads=2, dim=16, vdim=32),
+                     dict(heads=4, kv_heads=2, dim=32, vdim=24, conv=4, mask={"size": 40}, rot={"base": 1e4, "dims": 16}, scale=0.2),
+                     dict(heads=4, kv_heads=2, dim=16, vdim=24, conv=4, decay_rank=8, gate_rank=8), max_len=4096),
+    "1B": _rilenex(2048, 8192, 32000, 8, dict(heads=16, dim=128, vdim=128),
+                   dict(heads=16, kv_heads=4, dim=128, vdim=128, conv=4, mask={"size": 2048}, rot={"base": 5e5, "dims": 128},
+                        scale=128 ** -0.5),
+                   dict(heads=16, kv_heads=16, dim=128, vdim=128, conv=4, decay_rank=128, gate_rank=128)),
+    "7B": _rilenex(4096, 14336, 32000, 11, dict(heads=32, dim=128, vdim=128),
+                   dict(heads=32, kv_heads=4, dim=128, vdim=128, conv=4, mask={"size": 4096}, rot={"base": 5e5, "dims": 128},
+                        scale=128 ** -0.5),
+                   dict(heads=32, kv_heads=32, dim=128, vdim=128, conv=4, decay_rank=128, gate_rank=128)),
+}
+
 _ALIASES = {"llama": "llama2", "llama-2": "llama2", "llama-3": "llama3", "deepseek": "deepseek_v2",
             "deepseek-v2": "deepseek_v2", "mamba-2": "mamba2", "hss": "hss_ser"}
 
@@ -275,11 +334,11 @@ def get_model_config(family: str, size: str) -> dict:
 
 
 def config_from_name(name: str) -> ModelConfig:
-    """'llama3-8b', 'meta-llama/Llama-3-8B', 'mistral-7b', 'deepseek-v2-lite', 'mamba2-2.7b', 'hss-ser-tiny' ..."""
+    """'llama3-8b', 'meta-llama/Llama-3-8B', 'mistral-7b', 'deepseek-v2-lite', 'mamba2-2.7b', 'hss-ser-tiny', 'rilenex-1b' ..."""
     n = name.lower().split("/")[-1].replace("_", "-")
     table = [("llama-3", "llama3"), ("llama3", "llama3"), ("llama-2", "llama2"), ("llama2", "llama2"),
              ("llama", "llama2"), ("mistral", "mistral"), ("qwen2", "qwen2"), ("deepseek", "deepseek_v2"),
-             ("mamba", "mamba2"), ("hss", "hss_ser")]
+             ("mamba", "mamba2"), ("hss", "hss_ser"), ("rilenex", "rilenex")]
     for pat, fam in table:
         if pat in n:
             for size in _MODEL_REGISTRY[fam]:

@@ -26,6 +26,7 @@ class SxGemmArgs(C.Structure):
         ("tile_group", c_void_p), ("num_groups", c_int),
         ("k_ranges", c_void_p), ("k_total", c_int),
         ("status", c_void_p), ("sm_limit", c_int), ("force_bn", c_int), ("flags", c_int),
+        ("act_a", c_float), ("act_b", c_float),
     ]
 
 
@@ -42,6 +43,60 @@ class SxAttnArgs(C.Structure):
         ("v_head_div", c_int), ("causal", c_int), ("window", c_int), ("scale", c_float),
         ("status", c_void_p),
         ("block_mask", c_void_p), ("bm_batch_stride", c_ll), ("bm_head_stride", c_ll),
+    ]
+
+
+class SxRagged(C.Structure):
+    _fields_ = [("cu", c_void_p), ("pos0", c_void_p), ("slot", c_void_p), ("tok_seq", c_void_p), ("tok_pos", c_void_p),
+                ("n", c_int)]
+
+
+class SxQkvArgs(C.Structure):
+    _fields_ = [
+        ("u", c_void_p), ("u_ld", c_ll), ("wconv", c_void_p), ("ring", c_void_p), ("qn", c_void_p), ("kn", c_void_p),
+        ("inv_freq", c_void_p), ("talk", c_void_p), ("q_out", c_void_p), ("qmix_out", c_void_p), ("k_out", c_void_p),
+        ("v_out", c_void_p), ("k_ld", c_ll), ("v_ld", c_ll), ("kv_row", c_void_p), ("k_cache", c_void_p),
+        ("v_cache", c_void_p), ("cache_entry", c_void_p), ("ragged", SxRagged),
+        ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("dvp", c_int), ("taps", c_int),
+        ("rot", c_int), ("write_ring", c_int), ("f32", c_int), ("eps", c_float),
+    ]
+
+
+class SxDeltaArgs(C.Structure):
+    _fields_ = [
+        ("u", c_void_p), ("u_ld", c_ll), ("wconv", c_void_p), ("ring", c_void_p), ("b", c_void_p), ("b_ld", c_ll),
+        ("a", c_void_p), ("a_ld", c_ll), ("a_log", c_void_p), ("dt_bias", c_void_p), ("q", c_void_p), ("k", c_void_p),
+        ("g", c_void_p), ("v", c_void_p), ("beta", c_void_p), ("ragged", SxRagged),
+        ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("taps", c_int), ("write_ring", c_int),
+        ("f32", c_int),
+    ]
+
+
+class SxScanArgs(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("g", c_void_p), ("k", c_void_p), ("v", c_void_p), ("v_ld", c_ll), ("beta", c_void_p),
+        ("state", c_void_p), ("o", c_void_p), ("ragged", SxRagged),
+        ("H", c_int), ("Hq", c_int), ("d", c_int), ("dv", c_int), ("delta", c_int), ("f32", c_int),
+    ]
+
+
+class SxStepArgs(C.Structure):
+    _fields_ = [
+        ("inp", SxDeltaArgs), ("qr", c_void_p), ("fr", c_void_p), ("vr", c_void_p), ("ld", c_ll), ("fbias", c_void_p),
+        ("lower", c_void_p), ("state", c_void_p), ("norm", c_void_p), ("gate", c_void_p), ("gate_ld", c_ll),
+        ("y", c_void_p), ("y_ld", c_ll), ("ragged", SxRagged), ("mul", c_float), ("eps", c_float),
+        ("H", c_int), ("Hq", c_int), ("d", c_int), ("dv", c_int), ("delta", c_int), ("f32", c_int),
+    ]
+
+
+class SxTalkArgs(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("k", c_void_p), ("v", c_void_p), ("k_ld", c_ll), ("v_ld", c_ll), ("dvp", c_int),
+        ("kv_base", c_void_p), ("block_table", c_void_p), ("block_base", c_void_p), ("table_ld", c_int),
+        ("block_size", c_int), ("talk", c_void_p), ("gate", c_void_p), ("gate_ld", c_ll), ("y", c_void_p), ("y_ld", c_ll),
+        ("ragged", SxRagged), ("scale", c_float), ("mul", c_float),
+        ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("size", c_int), ("f32", c_int),
+        ("part", c_void_p), ("splits", c_int),
     ]
 
 

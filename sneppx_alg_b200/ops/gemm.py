@@ -19,7 +19,24 @@ from . import _lib
 ACT = {None: 0, "none": 0, "gelu": 1, "silu": 2, "relu": 3}
 
 
+class XIELU:
+    """Activation object for ``gemm(act=...)``: a z^2 + z / 2 for z > 0, b (e^z - 1 - z) + z / 2 for z <= 0, with
+    a = softplus(p) and b = 1/2 + softplus(q) of the two learned numbers."""
+
+    code = 4
+
+    def __init__(self, p: float, q: float):
+        sp = torch.nn.functional.softplus(torch.tensor([p, q], dtype=torch.float64))
+        self.a, self.b = float(sp[0]), float(sp[1]) + 0.5
+
+    def __call__(self, z):
+        zn = z.clamp(max=0)
+        return torch.where(z > 0, self.a * z * z, self.b * (torch.expm1(zn) - zn)) + 0.5 * z
+
+
 def _act_ref(x, act):
+    if isinstance(act, XIELU):
+        return act(x)
     if act in (None, "none", 0):
         return x
     if act in ("gelu", 1):
@@ -196,7 +213,10 @@ def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_dtype=None, c=None, beta
     args.a_mn, args.b_mn = int(a_mn), int(b_mn)
     args.out_fp32 = int(out.dtype == torch.float32)
     args.c_fp32 = int(c is not None and c.dtype == torch.float32)
-    args.act = ACT[act] if not isinstance(act, int) else act
+    if isinstance(act, XIELU):
+        args.act, args.act_a, args.act_b = act.code, act.a, act.b
+    else:
+        args.act = ACT[act] if not isinstance(act, int) else act
     args.alpha, args.beta = float(alpha), float(beta)
     if tile_group is not None:
         args.tile_group = tile_group.data_ptr()

@@ -1,0 +1,199 @@
+"""Front-ends of the hybrid-decoder kernels: fp32-residual norms, the gated recurrences (``csrc/recurrence.cu``), and
+chunked attention with a head mix before the softmax (``csrc/talking_attn.cu``). They run on CUDA tensors only; activations
+are bf16 or fp32, everything that the recurrences and the softmax work on is fp32 inside."""
+from __future__ import annotations
+
+import ctypes as C
+
+import torch
+
+from . import _lib
+from ._lib import c_float, c_int, c_ll, ptr, stream
+from .ragged import RaggedBatch
+
+
+def _f32(t) -> int:
+    if t.dtype == torch.float32:
+        return 1
+    if t.dtype == torch.bfloat16:
+        return 0
+    raise TypeError(f"activation type {t.dtype} is not supported (bfloat16 or float32)")
+
+
+def _need_cuda(t):
+    if not t.is_cuda:
+        raise RuntimeError("this operation runs on a CUDA device only")
+    _lib.lib()
+
+
+def embed_f32(table, ids):
+    """fp32 rows of the embedding table."""
+    _need_cuda(table)
+    x = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
+    _lib.call("sx_embed_f32", ptr(table), ptr(ids), ptr(x), c_int(ids.numel()), c_int(table.shape[1]), c_int(_f32(table)), stream())
+    return x
+
+
+def rmsnorm_f32(x, w, eps, out_dtype, rows=None):
+    """RMSNorm of fp32 rows (all of them, or the listed ones) into activations."""
+    _need_cuda(x)
+    n = x.shape[0] if rows is None else rows.numel()
+    y = torch.empty(n, x.shape[1], dtype=out_dtype, device=x.device)
+    _lib.call("sx_rmsnorm_f32", ptr(x), ptr(w), ptr(rows), ptr(y), c_int(n), c_int(x.shape[1]), c_float(eps), c_int(_f32(y)), stream())
+    return y
+
+
+def head_norm_gate(o, w, y, eps, gate=None, mul=1.0):
+    """y[t, h] = o[t, h] / rms * w * sigmoid(gate) * mul per head; o [T, H, dv] fp32, y [T, H * dv] (a column slice will do)."""
+    T, H, dv = o.shape
+    _lib.call("sx_head_norm_gate", ptr(o), ptr(w), ptr(gate), c_ll(gate.stride(0) if gate is not None else 0), c_float(mul),
+              ptr(y), c_ll(y.stride(0)), c_int(T), c_int(H), c_int(dv), c_float(eps), c_int(_f32(y)), stream())
+
+
+def conv_ring(u, ring, batch: RaggedBatch, channels, taps):
+    """Keep the last ``taps - 1`` projected rows of every portion in its slot's ring."""
+    if taps > 1:
+        r = batch.struct()
+        _lib.call("sx_conv_ring", ptr(u), c_ll(u.stride(0)), ptr(ring), C.byref(r), c_int(channels), c_int(taps), c_int(_f32(u)), stream())
+
+
+# ----------------------------------------------------------------------------- recurrences
+def gate_prep(qr, fr, bias, lower):
+    """silu(q) and the lower-bounded forget gate of a gated-write recurrence, both fp32 [T, H * d]."""
+    T, c = qr.shape
+    q = torch.empty(T, c, dtype=torch.float32, device=qr.device)
+    f = torch.empty_like(q)
+    assert qr.stride(0) == fr.stride(0)
+    _lib.call("sx_gate_prep", ptr(qr), ptr(fr), c_ll(qr.stride(0)), ptr(bias), ptr(lower), ptr(q), ptr(f), c_int(T), c_int(c),
+              c_int(_f32(qr)), stream())
+    return q, f
+
+
+def _delta_args(u, wconv, ring, b, a, a_log, dt_bias, batch, H, G, d, dv, taps):
+    x = _lib.SxDeltaArgs()
+    x.u, x.u_ld, x.wconv, x.ring = u.data_ptr(), u.stride(0), wconv.data_ptr(), ring.data_ptr()
+    x.b, x.b_ld, x.a, x.a_ld = b.data_ptr(), b.stride(0), a.data_ptr(), a.stride(0)
+    x.a_log, x.dt_bias = a_log.data_ptr(), dt_bias.data_ptr()
+    x.ragged = batch.struct()
+    x.T, x.H, x.G, x.d, x.dv, x.taps, x.f32 = batch.T, H, G, d, dv, taps, _f32(u)
+    return x
+
+
+def delta_prep(u, wconv, ring, b, a, a_log, dt_bias, batch: RaggedBatch, H, G, d, dv, taps):
+    """Operands of the gated delta rule from projected rows: q, k [T, G, d], decay [T, H, d], v [T, H * dv], beta [T, H]."""
+    _need_cuda(u)
+    T, dev = batch.T, u.device
+    q, k = (torch.empty(T, G, d, dtype=torch.float32, device=dev) for _ in range(2))
+    g = torch.empty(T, H, d, dtype=torch.float32, device=dev)
+    v = torch.empty(T, H * dv, dtype=u.dtype, device=dev)
+    beta = torch.empty(T, H, dtype=torch.float32, device=dev)
+    x = _delta_args(u, wconv, ring, b, a, a_log, dt_bias, batch, H, G, d, dv, taps)
+    x.q, x.k, x.g, x.v, x.beta = q.data_ptr(), k.data_ptr(), g.data_ptr(), v.data_ptr(), beta.data_ptr()
+    _lib.call("sx_delta_prep", C.byref(x), stream())
+    return q, k, g, v, beta
+
+
+def recur_scan(q, g, v, state, batch: RaggedBatch, H, d, dv, k=None, beta=None):
+    """Walks every portion of the batch from its slot's state (empty at position 0), stores the state back and returns the
+    read-outs [T, H, dv] fp32. With ``k`` and ``beta``: the gated delta rule; without: the gated write with key 1 - g."""
+    _need_cuda(q)
+    o = torch.empty(batch.T, H, dv, dtype=torch.float32, device=q.device)
+    x = _lib.SxScanArgs()
+    x.q, x.g, x.v, x.v_ld = q.data_ptr(), g.data_ptr(), v.data_ptr(), v.stride(0)
+    x.k = k.data_ptr() if k is not None else None
+    x.beta = beta.data_ptr() if beta is not None else None
+    x.state, x.o, x.ragged = state.data_ptr(), o.data_ptr(), batch.struct()
+    x.H, x.Hq, x.d, x.dv, x.delta, x.f32 = H, q.numel() // (batch.T * d), d, dv, int(k is not None), _f32(v)
+    _lib.call("sx_recur_scan", C.byref(x), stream())
+    return o
+
+
+def _step_args(state, norm, y, batch, H, Hq, d, dv, eps, gate, mul):
+    s = _lib.SxStepArgs()
+    s.state, s.norm, s.y, s.y_ld = state.data_ptr(), norm.data_ptr(), y.data_ptr(), y.stride(0)
+    if gate is not None:
+        s.gate, s.gate_ld = gate.data_ptr(), gate.stride(0)
+    s.ragged = batch.struct()
+    s.mul, s.eps = mul, eps
+    s.H, s.Hq, s.d, s.dv, s.f32 = H, Hq, d, dv, _f32(y)
+    return s
+
+
+def gated_write_step(qr, fr, vr, bias, lower, state, norm, y, batch: RaggedBatch, H, d, dv, eps, gate=None, mul=1.0):
+    """One token of every sequence through the gated-write recurrence, from projected rows to normed read-outs in y."""
+    _need_cuda(qr)
+    s = _step_args(state, norm, y, batch, H, H, d, dv, eps, gate, mul)
+    s.qr, s.fr, s.vr, s.ld = qr.data_ptr(), fr.data_ptr(), vr.data_ptr(), qr.stride(0)
+    s.fbias, s.lower, s.delta = bias.data_ptr(), lower.data_ptr(), 0
+    _lib.call("sx_recur_step", C.byref(s), stream())
+
+
+def delta_step(u, wconv, ring, b, a, a_log, dt_bias, state, norm, y, batch: RaggedBatch, H, G, d, dv, taps, eps, gate=None, mul=1.0):
+    """One token of every sequence through the gated delta rule, from projected rows to gated read-outs in y."""
+    _need_cuda(u)
+    s = _step_args(state, norm, y, batch, H, G, d, dv, eps, gate, mul)
+    s.inp = _delta_args(u, wconv, ring, b, a, a_log, dt_bias, batch, H, G, d, dv, taps)
+    s.delta = 1
+    _lib.call("sx_recur_step", C.byref(s), stream())
+
+
+# ----------------------------------------------------------------------------- attention with a head mix
+def qkv_prep(u, wconv, ring, qn, kn, inv_freq, batch: RaggedBatch, k_cache, v_cache, H, G, d, dv, taps, eps, q_out=None,
+             qmix_out=None, talk=None, k_out=None, v_out=None, dvp=0, kv_row=None):
+    """Convolution, query / key norm, rotation and cache append of attention operands (see ``SxQkvArgs``)."""
+    _need_cuda(u)
+    x = _lib.SxQkvArgs()
+    x.u, x.u_ld, x.wconv, x.ring = u.data_ptr(), u.stride(0), wconv.data_ptr(), ring.data_ptr()
+    x.qn, x.kn, x.inv_freq = qn.data_ptr(), kn.data_ptr(), inv_freq.data_ptr()
+    for name, t in (("talk", talk), ("q_out", q_out), ("qmix_out", qmix_out), ("k_out", k_out), ("v_out", v_out), ("kv_row", kv_row)):
+        if t is not None:
+            setattr(x, name, t.data_ptr())
+    if k_out is not None:
+        x.k_ld, x.v_ld = k_out.stride(0), v_out.stride(0)
+    x.k_cache, x.v_cache, x.cache_entry = k_cache.data_ptr(), v_cache.data_ptr(), batch.entry.data_ptr()
+    x.ragged = batch.struct()
+    x.T, x.H, x.G, x.d, x.dv, x.dvp, x.taps = batch.T, H, G, d, dv, dvp or dv, taps
+    x.rot, x.write_ring, x.f32, x.eps = 2 * inv_freq.numel(), int(batch.decode), _f32(u), eps
+    _lib.call("sx_qkv_prep", C.byref(x), stream())
+
+
+def kv_gather(cache, entry, row, out, G, w, wp):
+    """Copy cache entries (earlier positions of the running chunk) in front of a portion's packed rows."""
+    n = entry.numel()
+    if n:
+        _lib.call("sx_kv_gather", ptr(cache), ptr(entry), ptr(row), c_int(n), ptr(out), c_ll(out.stride(0)), c_int(G), c_int(w),
+                  c_int(wp), c_int(_f32(cache)), stream())
+
+
+def _talk_args(q, k, v, k_ld, v_ld, talk, gate, y, batch, scale, mul, H, G, d, dv, dvp, size):
+    a = _lib.SxTalkArgs()
+    a.q, a.k, a.v, a.k_ld, a.v_ld, a.dvp = q.data_ptr(), k.data_ptr(), v.data_ptr(), k_ld, v_ld, dvp
+    a.talk, a.gate, a.gate_ld, a.y, a.y_ld = talk.data_ptr(), gate.data_ptr(), gate.stride(0), y.data_ptr(), y.stride(0)
+    a.ragged = batch.struct()
+    a.scale, a.mul = scale, mul
+    a.T, a.H, a.G, a.d, a.dv, a.size, a.f32, a.splits = batch.T, H, G, d, dv, size, _f32(y), 1
+    return a
+
+
+def talking_attention(q, k, v, talk, gate, y, batch: RaggedBatch, kv_base, scale, mul, H, G, d, dv, dvp, size):
+    """Prompt form over packed keys and values; q fp32 [T, H, d]; y[t, h] = o * sigmoid(gate[t, h]) * mul."""
+    a = _talk_args(q, k, v, k.stride(0), v.stride(0), talk, gate, y, batch, scale, mul, H, G, d, dv, dvp, size)
+    a.kv_base = kv_base.data_ptr()
+    _lib.call("sx_talk_attn", C.byref(a), stream())
+
+
+def decode_splits(n: int, size: int) -> int:
+    """Key splits of one decode step: enough CTAs for the machine, at least 64 keys each."""
+    return max(1, min((size + 63) // 64, 296 // max(n, 1)))
+
+
+def talking_decode(q, k_cache, v_cache, talk, gate, y, batch: RaggedBatch, scale, mul, H, G, d, dv, size):
+    """Decode form: one query per sequence against the block pool."""
+    a = _talk_args(q, k_cache, v_cache, G * d, G * dv, talk, gate, y, batch, scale, mul, H, G, d, dv, dv, size)
+    a.block_table, a.block_base = batch.block_table.data_ptr(), batch.block_base.data_ptr()
+    a.table_ld, a.block_size = batch.table_width, k_cache.shape[1]
+    a.splits = decode_splits(batch.n, size)
+    if a.splits > 1:
+        part = torch.empty(batch.n * a.splits * H * (dv + 2), dtype=torch.float32, device=q.device)
+        a.part = part.data_ptr()
+    _lib.call("sx_talk_attn", C.byref(a), stream())

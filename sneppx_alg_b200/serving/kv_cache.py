@@ -109,18 +109,25 @@ class PrefixCache:
 
 
 class PagedKVCache:
-    def __init__(self, num_layers, num_blocks, block_size, num_kv_heads, head_dim, dtype=torch.bfloat16, device="cuda",
-                 enable_prefix_cache=True):
+    """``layer_shapes`` (one ``(kv heads, key size, value size)`` per layer) replaces ``num_kv_heads`` / ``head_dim`` for
+    models whose layers differ or whose keys and values have different sizes."""
+
+    def __init__(self, num_layers, num_blocks, block_size, num_kv_heads=0, head_dim=0, dtype=torch.bfloat16, device="cuda",
+                 enable_prefix_cache=True, layer_shapes=None):
         self.block_size, self.num_layers = block_size, num_layers
         self.pool = KVBlockPool(num_blocks)
-        shape = (num_blocks, block_size, num_kv_heads, head_dim)
-        self.k = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
-        self.v = [torch.zeros(shape, dtype=dtype, device=device) for _ in range(num_layers)]
+        shapes = layer_shapes if layer_shapes is not None else [(num_kv_heads, head_dim, head_dim)] * num_layers
+        self.k = [torch.zeros(num_blocks, block_size, h, dk, dtype=dtype, device=device) for h, dk, _ in shapes]
+        self.v = [torch.zeros(num_blocks, block_size, h, dv, dtype=dtype, device=device) for h, _, dv in shapes]
         self.tables: Dict[int, List[int]] = {}
         self.lens: Dict[int, int] = {}
         self.prefix = PrefixCache(self.pool, block_size) if enable_prefix_cache else None
         if self.prefix is not None:
             self.pool.reclaim = self.prefix.evict
+
+    def blocks_for(self, n_tokens: int) -> int:
+        """Most blocks a sequence of ``n_tokens`` holds at any time."""
+        return (n_tokens + self.block_size - 1) // self.block_size
 
     def available_blocks(self) -> int:
         """Free blocks plus those the prefix cache would give back."""
@@ -195,3 +202,91 @@ class PagedKVCache:
         k = self.k[layer][blocks].reshape(-1, *self.k[layer].shape[2:])[:n]
         v = self.v[layer][blocks].reshape(-1, *self.v[layer].shape[2:])[:n]
         return k, v
+
+
+class ChunkedKVCache(PagedKVCache):
+    """Paged cache of layers in which a position only sees its own chunk of positions (``sizes``: the chunk lengths that
+    occur). Positions behind the last visible one are never stored, and blocks that fall behind it go back to the pool,
+    so a sequence holds a bounded number of blocks however long it grows. Block tables start at block ``base[seq]``."""
+
+    def __init__(self, layer_shapes, sizes, num_blocks, block_size, dtype=torch.bfloat16, device="cuda"):
+        super().__init__(len(layer_shapes), num_blocks, block_size, dtype=dtype, device=device, enable_prefix_cache=False,
+                         layer_shapes=layer_shapes)
+        self.sizes = sorted(set(sizes))
+        self.base: Dict[int, int] = {}
+
+    @property
+    def table_width(self) -> int:
+        """Blocks that the visible positions of one sequence can touch."""
+        return (self.sizes[-1] + self.block_size - 2) // self.block_size + 1 if self.sizes else 0
+
+    def blocks_for(self, n_tokens: int) -> int:
+        return min(super().blocks_for(n_tokens), self.table_width)
+
+    def first_visible(self, pos: int) -> int:
+        """Earliest position that any layer still sees from ``pos``."""
+        return min(pos // s * s for s in self.sizes) if self.sizes else pos + 1
+
+    def add_sequence(self, seq_id: int, tokens=None) -> int:
+        self.tables[seq_id], self.lens[seq_id], self.base[seq_id] = [], 0, 0
+        return 0
+
+    def reserve(self, seq_id: int, n_new: int) -> List[int]:
+        """Cache entries of the next ``n_new`` tokens; -1 for tokens that no later token sees."""
+        n, table, base = self.lens[seq_id], self.tables[seq_id], self.base[seq_id]
+        end = n + n_new
+        keep = self.first_visible(end - 1)
+        new_base = keep // self.block_size
+        while table and base < new_base:
+            self.pool.release(table.pop(0))
+            base += 1
+        if not table:
+            base = max(base, new_base)
+        entries = []
+        for p in range(n, end):
+            if p < keep:
+                entries.append(-1)
+                continue
+            bi = p // self.block_size - base
+            if bi == len(table):
+                table.append(self.pool.allocate())
+            entries.append(table[bi] * self.block_size + p % self.block_size)
+        self.base[seq_id], self.lens[seq_id] = base, end
+        return entries
+
+    def entries(self, seq_id: int, lo: int, hi: int) -> List[int]:
+        """Entries of the stored positions [lo, hi)."""
+        table, base, bs = self.tables[seq_id], self.base[seq_id], self.block_size
+        return [table[p // bs - base] * bs + p % bs for p in range(lo, hi)]
+
+    def fork(self, src_id: int, dst_id: int) -> None:
+        raise NotImplementedError("a chunked cache does not share blocks between sequences")
+
+    def free_sequence(self, seq_id: int, tokens=None) -> None:
+        self.base.pop(seq_id, None)
+        super().free_sequence(seq_id)
+
+
+class HybridCache(ChunkedKVCache):
+    """Memory of models that mix recurrent layers and chunked attention: the block pool of the attention layers and one
+    slot of fixed-size state per live sequence (``state_spec``: per layer, name -> (shape, dtype) of one slot). A slot is
+    never cleared: the kernels start a sequence's first portion from an empty state whatever the slot holds."""
+
+    def __init__(self, kv_shapes, sizes, state_spec, max_sequences, num_blocks, block_size=16, dtype=torch.bfloat16,
+                 device="cuda"):
+        super().__init__(kv_shapes, sizes, num_blocks, block_size, dtype, device)
+        self.free_slots = list(range(max_sequences - 1, -1, -1))
+        self.slots: Dict[int, int] = {}
+        self.state = [{k: torch.zeros(max_sequences, *shape, dtype=dt, device=device) for k, (shape, dt) in spec.items()}
+                      for spec in state_spec]
+
+    def add_sequence(self, seq_id: int, tokens=None) -> int:
+        if not self.free_slots:
+            raise MemoryError("no free state slot")
+        self.slots[seq_id] = self.free_slots.pop()
+        return super().add_sequence(seq_id, tokens)
+
+    def free_sequence(self, seq_id: int, tokens=None) -> None:
+        if seq_id in self.slots:
+            self.free_slots.append(self.slots.pop(seq_id))
+        super().free_sequence(seq_id)

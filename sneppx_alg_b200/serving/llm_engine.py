@@ -20,6 +20,7 @@ import torch
 from ..ops import functional as ops
 from ..ops import paged
 from .generation import apply_repetition_penalty, sample_from_logits
+from .hybrid_runner import HybridRunner
 from .kv_cache import PagedKVCache
 
 
@@ -309,6 +310,9 @@ class StateCache:
         self.pool = _Slots(max_sequences)
         self._live, self._on_free = set(), on_free
 
+    def blocks_for(self, n_tokens):
+        return 1
+
     def available_blocks(self):
         return self.pool.num_free
 
@@ -375,8 +379,13 @@ class LLMEngine:
         p = next(model.parameters())
         if runner is None and getattr(cfg, "architecture", "transformer") == "mamba2":
             runner = StatefulRunner(model)   # recurrent-state models: no KV cache, one state slot per sequence
+        if runner is None and getattr(cfg, "architecture", "transformer") == "rilenex":
+            # recurrent layers beside chunked attention: state slots and a block pool
+            runner = HybridRunner(model, model.init_cache(max_batch_size, num_blocks, block_size))
         if isinstance(runner, StatefulRunner):
             self.cache = StateCache(max_batch_size, on_free=runner.release)
+        elif isinstance(runner, HybridRunner):
+            self.cache = runner.cache
         elif tp_group is not None:
             import torch.distributed as dist
             tp = dist.get_world_size(tp_group)
@@ -389,7 +398,8 @@ class LLMEngine:
         self.runner = runner or LlamaPagedRunner(model, self.cache)
         # CUDA-graph decode: the single-GPU runner, and the tensor-parallel runner when its all-reduce is the
         # graph-capturable peer-load kernel
-        if cuda_graphs and p.is_cuda and (type(self.runner) is LlamaPagedRunner or getattr(self.runner, "_sg", None) is not None):
+        if cuda_graphs and p.is_cuda and (type(self.runner) in (LlamaPagedRunner, HybridRunner)
+                                          or getattr(self.runner, "_sg", None) is not None):
             limit = max_model_len or min(getattr(cfg, "max_position_embeddings", 4096) or 4096, num_blocks * block_size)
             self.runner.enable_graphs(max_batch_size, limit)
         self.max_batch_size, self.max_prefill_tokens, self.policy = max_batch_size, max_prefill_tokens, policy
@@ -413,8 +423,7 @@ class LLMEngine:
         return bool(self.waiting or self.running)
 
     def _blocks_needed(self, req: Request) -> int:
-        bs = self.cache.block_size
-        return (len(req.prompt) + req.params.max_new_tokens + bs - 1) // bs
+        return self.cache.blocks_for(len(req.prompt) + req.params.max_new_tokens)
 
     def _committed(self) -> int:
         """Blocks the running sequences may still claim before they finish (admission keeps these in hand, so a
@@ -458,12 +467,13 @@ class LLMEngine:
 
     def _admit_same_length(self, first: "Request", budget: int) -> List["Request"]:
         """Pops the waiting requests that can join ``first``'s prefill pass: they are next in queue order, have a
-        prompt of the same length, hit no cached prefix, fit the batch, the token budget and the block pool."""
+        prompt of the same length (any length when the runner packs ragged prompts), hit no cached prefix, fit the batch, the token budget and the block pool."""
         out, T = [], len(first.prompt)
+        ragged = getattr(self.runner, "ragged_prefill", False)
         reserved = self._blocks_needed(first)
-        while self.waiting and len(self.running) + 1 + len(out) < self.max_batch_size and budget >= T and len(out) < 15:
+        while self.waiting and len(self.running) + 1 + len(out) < self.max_batch_size and len(out) < 15:
             nxt = self.waiting[0]
-            if len(nxt.prompt) != T:
+            if (len(nxt.prompt) != T and not ragged) or budget < len(nxt.prompt):
                 break
             need = reserved + self._blocks_needed(nxt) + self._committed()
             if need > self.cache.available_blocks() or not self.cache.make_room(need):
@@ -474,7 +484,7 @@ class LLMEngine:
             heapq.heappop(self.waiting)
             out.append(nxt)
             reserved += self._blocks_needed(nxt)
-            budget -= T
+            budget -= len(nxt.prompt)
         return out
 
     def step(self):
