@@ -39,7 +39,8 @@ PRECISE_SOURCES = {"decoder_ops.cu", "recurrence.cu", "talking_attn.cu"}
 
 # Named subsets of the sources for programs that need only part of the library; each is linked on its own.
 CUDA_SUBSETS = {
-    "hybrid": ("decoder_ops.cu", "recurrence.cu", "talking_attn.cu", "gemm_tc.cu", "gemm_skinny.cu"),
+    "hybrid": ("decoder_ops.cu", "recurrence.cu", "talking_attn.cu", "talking_attn_tc.cu", "talking_decode.cu",
+               "gemm_tc.cu", "gemm_skinny.cu"),
 }
 
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-pthread", "-Wall", "-Wno-unused-function"]

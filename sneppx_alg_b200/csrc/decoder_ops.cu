@@ -118,7 +118,8 @@ struct QkvParams {
   const double* inv_freq;     // [rot / 2]
   const float* talk;          // [H, H] (mixed-query output only)
   float* q_out;               // [T, H, d] fp32, or null
-  void* qmix_out;             // [T, H, G d] activation type, or null
+  void* qmix_out;             // [T, H, qmix_ld] activation type, or null
+  int qmix_ld;
   void* k_out; void* v_out;   // packed rows for the prompt kernels, or null
   long long k_ld, v_ld;       // row pitches; V of head j starts at column j * dvp
   int dvp;
@@ -126,116 +127,137 @@ struct QkvParams {
   void* k_cache; void* v_cache;       // [entries, G, d] / [entries, G, dv]
   const int* cache_entry;     // [T], -1: not kept
   RaggedView rv;
+  ChunkView cv;
   int T, H, G, d, dv, taps, rot;
-  int write_ring;             // one token per sequence: this launch also stores the token's own ring entry
   float eps;
 };
 
-template <typename A>
-__device__ __forceinline__ float conv_at(const QkvParams& p, const A* __restrict__ row, int ch, int pos, int pos0, const A* __restrict__ ring) {
-  const int C = p.H * p.d + p.G * (p.d + p.dv);
-  float acc = 0.f;
-  for (int j = 0; j < p.taps; ++j) {
-    const int b = p.taps - 1 - j;          // tokens back
-    if (b > pos) continue;
-    float x;
-    if (pos - b >= pos0) x = to_f(row[ch - (long long)b * p.u_ld]);
-    else x = to_f(ring[(long long)((pos - b) % p.taps) * C + ch]);
-    acc = fmaf(p.wconv[(long long)j * C + ch], x, acc);
-  }
-  return acc;
-}
-
-template <typename A>
+// One CTA: NT rows of one portion (a chunk of a prompt, or the one row of a decode step) for one key head with its query
+// heads and value head. A thread walks a channel through the rows; heads are then normed and rotated in shared memory.
+template <typename A, int NT, int MT>
 __global__ void __launch_bounds__(256) qkv_prep_kernel(const QkvParams p) {
-  extern __shared__ float sm[];
-  float* cs = sm;                    // [rot/2] cos
-  float* sn = cs + p.rot / 2;        // [rot/2] sin
-  float* sq = sn + p.rot / 2;        // [H, d] rotated queries (mixed-query output)
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const int seq = p.rv.tok_seq[t], pos = p.rv.tok_pos[t], pos0 = p.rv.pos0[seq];
-  const int C = p.H * p.d + p.G * (p.d + p.dv);
-  const A* row = reinterpret_cast<const A*>(p.u) + (long long)t * p.u_ld;
-  A* ring = reinterpret_cast<A*>(p.ring) + (long long)p.rv.slot[seq] * p.taps * C;
-  const int entry = p.cache_entry[t];
-  const long long krow = p.kv_row ? p.kv_row[t] : t;
-  for (int i = threadIdx.x; i < p.rot / 2; i += blockDim.x) {
-    double a = (double)pos * p.inv_freq[i];
+  extern __shared__ __align__(16) float sm[];
+  const int grp = p.H / p.G, nh = grp + 1, d = p.d, j = blockIdx.y;
+  float* cs = sm;                    // [NT, rot/2] cos
+  float* sn = cs + NT * (p.rot / 2); // [NT, rot/2] sin
+  float* sh = sn + NT * (p.rot / 2); // [NT, grp + 1, d] query heads of the group, then the key head
+  float* st = sh + NT * nh * d;      // [H, grp] head mix towards this group's queries
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int seq = NT == 1 ? blockIdx.x : p.cv.seq[blockIdx.x], s0 = NT == 1 ? 0 : p.cv.start[blockIdx.x];
+  const int slot = p.rv.slot[seq];
+  if (slot < 0) return;              // padding row of a captured launch
+  const int row0 = p.rv.cu[seq] + s0, nt = NT == 1 ? 1 : min(NT, p.rv.cu[seq + 1] - row0), pos = p.rv.pos0[seq] + s0;
+  const int C = p.H * d + p.G * (d + p.dv);
+  const A* u = reinterpret_cast<const A*>(p.u) + (long long)row0 * p.u_ld;
+  A* ring = reinterpret_cast<A*>(p.ring) + (long long)slot * p.taps * C;
+  for (int i = tid; i < NT * (p.rot / 2); i += 256) {
+    double a = (double)(pos + i / (p.rot / 2)) * p.inv_freq[i % (p.rot / 2)];
     a -= 6.283185307179586476925286766559 * rint(a * 0.15915494309189533576888376337251);
     float s, c;
     sincosf((float)a, &s, &c);
     cs[i] = c;
     sn[i] = s;
   }
-  __syncthreads();
-  // one warp per query / key head; a lane owns the pairs (2i, 2i + 1) with i = lane, lane + 32, ..
-  for (int hh = warp; hh < p.H + p.G; hh += nw) {
-    const bool is_q = hh < p.H;
-    const int ch0 = hh * p.d;
-    const float* nw_ = is_q ? p.qn : p.kn;
-    float va[QK_PAIRS], vb[QK_PAIRS];
-    float ss = 0.f;
+  if (p.qmix_out)
+    for (int i = tid; i < p.H * grp; i += 256) st[i] = p.talk[(i / grp) * p.H + j * grp + i % grp];
+  const int nqk = nh * d;
+  for (int i = tid; i < nqk + p.dv; i += 256) {
+    const bool is_v = i >= nqk;
+    const int ch = is_v ? (p.H + p.G) * d + j * p.dv + i - nqk : (i < grp * d ? j * grp * d + i : (p.H + j) * d + i - grp * d);
+    float y[NT];
+    conv_walk<A, NT, MT>(u, p.u_ld, p.wconv, p.taps, C, ch, ring, pos, s0, nt, y);
+    if (NT == 1 && p.taps > 1) ring[(long long)(pos % p.taps) * C + ch] = u[ch];   // not an entry that this step reads
+    if (is_v) {
+      const int c = i - nqk;
 #pragma unroll
-    for (int n = 0; n < QK_PAIRS; ++n) {
-      const int i = lane + 32 * n;
-      va[n] = vb[n] = 0.f;
-      if (2 * i < p.d) {
-        va[n] = conv_at<A>(p, row, ch0 + 2 * i, pos, pos0, ring);
-        vb[n] = conv_at<A>(p, row, ch0 + 2 * i + 1, pos, pos0, ring);
-        ss += va[n] * va[n] + vb[n] * vb[n];
+      for (int t = 0; t < NT; ++t) {
+        if (t >= nt) continue;
+        const A v = from_f<A>(y[t]);
+        if (p.v_out) reinterpret_cast<A*>(p.v_out)[(long long)p.kv_row[row0 + t] * p.v_ld + j * p.dvp + c] = v;
+        const int entry = p.cache_entry[row0 + t];
+        if (entry >= 0) reinterpret_cast<A*>(p.v_cache)[((long long)entry * p.G + j) * p.dv + c] = v;
       }
+    } else {
+#pragma unroll
+      for (int t = 0; t < NT; ++t) sh[t * nqk + i] = y[t];
+    }
+  }
+  __syncthreads();
+  // one warp per head row: RMS norm and rotation of the pairs (2i, 2i + 1)
+  for (int it = warp; it < NT * nh; it += 8) {
+    const int t = it / nh, hh = it % nh;
+    if (t >= nt) break;
+    float* x = sh + t * nqk + hh * d;
+    float ss = 0.f;
+    for (int i = lane; i < d / 2; i += 32) {
+      const float2 v = *reinterpret_cast<const float2*>(x + 2 * i);
+      ss += v.x * v.x + v.y * v.y;
     }
     ss = warp_sum(ss);
-    const float r = 1.f / sqrtf(ss / p.d + p.eps);
-#pragma unroll
-    for (int n = 0; n < QK_PAIRS; ++n) {
-      const int i = lane + 32 * n;
-      if (2 * i >= p.d) continue;
-      float a = va[n] * r * nw_[2 * i], b = vb[n] * r * nw_[2 * i + 1];
+    const float r = 1.f / sqrtf(ss / d + p.eps);
+    const bool is_q = hh < grp;
+    const float* w = is_q ? p.qn : p.kn;
+    const long long krow = !is_q && p.k_out ? p.kv_row[row0 + t] : 0;
+    const int entry = is_q ? -1 : p.cache_entry[row0 + t];
+    for (int i = lane; i < d / 2; i += 32) {
+      float2 v = *reinterpret_cast<const float2*>(x + 2 * i);
+      v.x *= r * w[2 * i];
+      v.y *= r * w[2 * i + 1];
       if (2 * i < p.rot) {
-        const float c = cs[i], s = sn[i];
-        const float a2 = a * c - b * s, b2 = b * c + a * s;
-        a = a2;
-        b = b2;
+        const float c = cs[t * (p.rot / 2) + i], s = sn[t * (p.rot / 2) + i];
+        v = make_float2(v.x * c - v.y * s, v.y * c + v.x * s);
       }
       if (is_q) {
-        if (p.q_out) *reinterpret_cast<float2*>(p.q_out + ((long long)t * p.H + hh) * p.d + 2 * i) = make_float2(a, b);
-        if (p.qmix_out) {
-          sq[hh * p.d + 2 * i] = a;
-          sq[hh * p.d + 2 * i + 1] = b;
-        }
+        if (p.q_out) *reinterpret_cast<float2*>(p.q_out + ((long long)(row0 + t) * p.H + j * grp + hh) * d + 2 * i) = v;
+        if (p.qmix_out) *reinterpret_cast<float2*>(x + 2 * i) = v;
       } else {
-        const int col = (hh - p.H) * p.d + 2 * i;
-        if (p.k_out) store2(reinterpret_cast<A*>(p.k_out) + krow * p.k_ld + col, a, b);
-        if (entry >= 0) store2(reinterpret_cast<A*>(p.k_cache) + (long long)entry * p.G * p.d + col, a, b);
+        const int col = j * d + 2 * i;
+        if (p.k_out) store2(reinterpret_cast<A*>(p.k_out) + krow * p.k_ld + col, v.x, v.y);
+        if (entry >= 0) store2(reinterpret_cast<A*>(p.k_cache) + (long long)entry * p.G * d + col, v.x, v.y);
       }
     }
   }
-  const int vch0 = (p.H + p.G) * p.d;
-  for (int c = threadIdx.x; c < p.G * p.dv; c += blockDim.x) {
-    const A v = from_f<A>(conv_at<A>(p, row, vch0 + c, pos, pos0, ring));
-    if (p.v_out) reinterpret_cast<A*>(p.v_out)[krow * p.v_ld + (c / p.dv) * p.dvp + c % p.dv] = v;
-    if (entry >= 0) reinterpret_cast<A*>(p.v_cache)[(long long)entry * p.G * p.dv + c] = v;
-  }
-  if (p.write_ring && p.taps > 1 && p.rv.slot[seq] >= 0)
-    for (int c = threadIdx.x; c < C; c += blockDim.x) ring[(long long)(pos % p.taps) * C + c] = row[c];
-  if (p.qmix_out) {
-    // The head mix is linear in the scores, so it is folded into the queries: mixed head h meets the concatenated key
-    // row of all key heads with sum over the query heads g of key head j of talk[h, g] q_g in block j.
-    __syncthreads();
-    const int grp = p.H / p.G, Gd = p.G * p.d;
-    A* out = reinterpret_cast<A*>(p.qmix_out) + (long long)t * p.H * Gd;
-    for (int i = threadIdx.x; i < p.H * Gd / 2; i += blockDim.x) {
-      const int h = (2 * i) / Gd, c = (2 * i) % Gd, j = c / p.d, e = c % p.d;
-      float a = 0.f, b = 0.f;
-      for (int g = 0; g < grp; ++g) {
-        const float w = p.talk[h * p.H + j * grp + g];
-        const float2 qv = *reinterpret_cast<const float2*>(&sq[(j * grp + g) * p.d + e]);
-        a = fmaf(w, qv.x, a);
-        b = fmaf(w, qv.y, b);
+  if (!p.qmix_out) return;
+  // The head mix is linear in the scores, so it is folded into the queries: mixed head h meets the concatenated key row of
+  // all key heads with sum over the query heads g of key head j of talk[h, g] q_g in block j. This CTA writes block j.
+  __syncthreads();
+  A* out = reinterpret_cast<A*>(p.qmix_out) + (long long)row0 * p.H * p.qmix_ld;
+  const int half = d / 2;
+  for (int i = tid; i < nt * half; i += 256) {
+    const int t = i / half, e = i % half;
+    const float* x = sh + t * nqk + 2 * e;
+    A* o = out + (long long)t * p.H * p.qmix_ld + j * d + 2 * e;
+    if (grp <= 8) {
+      float2 q[8];
+#pragma unroll
+      for (int g = 0; g < 8; ++g) q[g] = g < grp ? *reinterpret_cast<const float2*>(x + g * d) : make_float2(0.f, 0.f);
+      for (int h = 0; h < p.H; ++h) {
+        float a = 0.f, b = 0.f;
+#pragma unroll
+        for (int g = 0; g < 8; ++g)
+          if (g < grp) {
+            const float w = st[h * grp + g];
+            a = fmaf(w, q[g].x, a);
+            b = fmaf(w, q[g].y, b);
+          }
+        store2(o + (long long)h * p.qmix_ld, a, b);
       }
-      store2(out + 2 * i, a, b);
+    } else {
+      for (int h = 0; h < p.H; ++h) {
+        float a = 0.f, b = 0.f;
+        for (int g = 0; g < grp; ++g) {
+          const float w = st[h * grp + g];
+          const float2 q = *reinterpret_cast<const float2*>(x + g * d);
+          a = fmaf(w, q.x, a);
+          b = fmaf(w, q.y, b);
+        }
+        store2(o + (long long)h * p.qmix_ld, a, b);
+      }
     }
+  }
+  if (j == 0) {
+    const int pad = p.qmix_ld - p.G * d;
+    for (int i = tid; i < nt * p.H * pad; i += 256) out[(long long)(i / pad) * p.qmix_ld + p.G * d + i % pad] = from_f<A>(0.f);
   }
 }
 
@@ -277,27 +299,34 @@ extern "C" int sx_conv_ring(const void* u, long long u_ld, void* ring, const SxR
   SX_ACT_DISPATCH(f32, (conv_ring_kernel<A><<<dim3(r->n, taps - 1), 256, 0, st>>>((const A*)u, u_ld, (A*)ring, rv, C, taps)));
   return last_rc();
 }
+template <typename A, int NT, int MT>
+static int launch_qkv(const QkvParams& p, int ctas, cudaStream_t st) {
+  const int grp = p.H / p.G;
+  const int smem = (NT * p.rot + NT * (grp + 1) * p.d + p.H * grp) * 4;
+  static int set = 48 * 1024;
+  if (smem > 227 * 1024) return -2;
+  if (smem > set) {
+    if (cudaFuncSetAttribute(qkv_prep_kernel<A, NT, MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -10;
+    set = smem;
+  }
+  qkv_prep_kernel<A, NT, MT><<<dim3(ctas, p.G), 256, smem, st>>>(p);
+  return last_rc();
+}
 extern "C" int sx_qkv_prep(const SxQkvArgs* a, cudaStream_t st) {
   if (a->T <= 0) return 0;
-  if (a->d % 2 || a->rot % 2 || a->rot > a->d || a->d > 64 * QK_PAIRS || a->G <= 0 || a->H % a->G) return -1;
+  if (a->d % 2 || a->rot % 2 || a->rot > a->d || a->G <= 0 || a->H % a->G || a->taps < 1 || a->taps > 8) return -1;
   QkvParams p;
   p.u = a->u; p.u_ld = a->u_ld; p.wconv = a->wconv; p.ring = a->ring; p.qn = a->qn; p.kn = a->kn; p.inv_freq = a->inv_freq;
-  p.talk = a->talk; p.q_out = a->q_out; p.qmix_out = a->qmix_out; p.k_out = a->k_out; p.v_out = a->v_out;
+  p.talk = a->talk; p.q_out = a->q_out; p.qmix_out = a->qmix_out; p.qmix_ld = a->qmix_ld; p.k_out = a->k_out; p.v_out = a->v_out;
   p.k_ld = a->k_ld; p.v_ld = a->v_ld; p.dvp = a->dvp; p.kv_row = a->kv_row; p.k_cache = a->k_cache; p.v_cache = a->v_cache;
-  p.cache_entry = a->cache_entry; p.rv = view(&a->ragged);
-  p.T = a->T; p.H = a->H; p.G = a->G; p.d = a->d; p.dv = a->dv; p.taps = a->taps; p.rot = a->rot;
-  p.write_ring = a->write_ring; p.eps = a->eps;
-  const int smem = (a->rot + (a->qmix_out ? a->H * a->d : 0)) * 4;
-  if (smem > 200 * 1024) return -2;
+  p.cache_entry = a->cache_entry; p.rv = view(&a->ragged); p.cv = chunks(&a->chunks);
+  p.T = a->T; p.H = a->H; p.G = a->G; p.d = a->d; p.dv = a->dv; p.taps = a->taps; p.rot = a->rot; p.eps = a->eps;
   SX_ACT_DISPATCH(a->f32, {
-    static int set = 0;
-    if (smem > 48 * 1024 && set < smem) {
-      if (cudaFuncSetAttribute(qkv_prep_kernel<A>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return -10;
-      set = smem;
-    }
-    qkv_prep_kernel<A><<<a->T, 256, smem, st>>>(p);
+    if (a->chunks.n == 0) return launch_qkv<A, 1, 8>(p, a->ragged.n, st);     // one row per portion
+    if (!a->kv_row) return -3;
+    return a->taps <= 4 ? launch_qkv<A, RC, 4>(p, a->chunks.n, st) : launch_qkv<A, RC, 8>(p, a->chunks.n, st);
   });
-  return last_rc();
+  return 0;
 }
 extern "C" int sx_kv_gather(const void* cache, const int* entry, const int* row, int n, void* out, long long out_ld, int G, int w,
                             int wp, int f32, cudaStream_t st) {

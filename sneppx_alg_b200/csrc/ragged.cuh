@@ -6,8 +6,6 @@
 
 namespace sx {
 
-constexpr int QK_PAIRS = 4;   // a lane holds up to this many pairs of a query / key head: head sizes up to 256
-
 // Rows of several sequences, one portion each, packed one after another.
 struct RaggedView {
   const int* cu;        // [n + 1] first row of each portion
@@ -40,6 +38,47 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float a, float b, float
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
+
+// NT tokens of one channel of a short causal convolution: y[t] = sum_b w[b] x[t - b]. `u` points at the first token's row;
+// tokens in front of it are earlier rows of the portion (s0 of them are there) or come from the ring, which keeps position p
+// in entry p % taps; positions before the sequence are zero. w [taps, C], last row for the current token; taps <= MT.
+template <typename A, int NT, int MT>
+__device__ __forceinline__ void conv_walk(const A* __restrict__ u, long long ld, const float* __restrict__ w, int taps, int C, int ch,
+                                          const A* ring, int pos, int s0, int nt, float (&y)[NT]) {
+  float x[NT + MT - 1], wb[MT];
+#pragma unroll
+  for (int b = 0; b < MT; ++b) wb[b] = b < taps ? w[(long long)(taps - 1 - b) * C + ch] : 0.f;
+  const int ph = pos % taps;
+#pragma unroll
+  for (int i = 0; i < NT + MT - 1; ++i) {
+    const int t = i - (MT - 1);          // token relative to the first one
+    x[i] = 0.f;
+    if (t < 0) {
+      if (-t < taps) {
+        if (s0 + t >= 0) x[i] = to_f(u[(long long)t * ld + ch]);
+        else if (pos + t >= 0) x[i] = to_f(ring[(long long)(ph + t >= 0 ? ph + t : ph + t + taps) * C + ch]);
+      }
+    } else if (t < nt) {
+      x[i] = to_f(u[(long long)t * ld + ch]);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < NT; ++t) {
+    float a = 0.f;
+#pragma unroll
+    for (int b = MT - 1; b >= 0; --b) a = fmaf(wb[b], x[t + MT - 1 - b], a);
+    y[t] = a;
+  }
+}
+
+struct ChunkView {
+  const int* seq;       // [n_chunks] portion of each chunk
+  const int* start;     // [n_chunks] first row of the chunk within its portion
+  const int* first;     // [n + 1] first chunk of each portion
+  int n_chunks;
+};
+inline ChunkView chunks(const SxChunks* c) { return ChunkView{c->seq, c->start, c->first, c->n}; }
+constexpr int RC = 16;  // rows per chunk
 
 inline int last_rc() { return cudaGetLastError() == cudaSuccess ? 0 : -11; }
 

@@ -6,6 +6,7 @@
 // anywhere. State layout: [slots, H, d, dv].
 #include "common.cuh"
 #include "ragged.cuh"
+#include "tc_common.cuh"
 #include "sx_api.h"
 
 namespace sx {
@@ -19,92 +20,226 @@ struct DeltaParams {
   const void* b; long long b_ld;      // [T, H] write-strength logits
   const void* a; long long a_ld;      // [T, H d] decay inputs (second low-rank product)
   const float* a_log; const float* dt_bias;   // [H], [H d]
-  float* q; float* k;         // [T, G, d]
-  float* g;                   // [T, H, d] decay
-  void* v;                    // [T, H dv] activation type
-  float* beta;                // [T, H]
+  void* v;                    // [T, H dv] convolved values, activation type
   RaggedView rv;
-  int T, H, G, d, dv, taps, write_ring;
+  int T, H, G, d, dv, taps;
 };
 
-template <typename A>
-__device__ __forceinline__ float conv_silu_at(const DeltaParams& p, const A* __restrict__ row, int ch, int C, int pos, int pos0,
-                                              const A* __restrict__ ring) {
-  float acc = 0.f;
-  for (int j = 0; j < p.taps; ++j) {
-    const int b = p.taps - 1 - j;
-    if (b > pos) continue;
-    const float x = pos - b >= pos0 ? to_f(row[ch - (long long)b * p.u_ld]) : to_f(ring[(long long)((pos - b) % p.taps) * C + ch]);
-    acc = fmaf(p.wconv[(long long)j * C + ch], x, acc);
+// ------------------------------------------------------------------ chunk form of the recurrences
+// A portion is walked in chunks of RC tokens. With G_t the product of the decays of the chunk's tokens up to t, the state
+// S0 in front of the chunk and k_t, u_t the written key and value,
+//   o_t = S0^T (G_t q_t) + sum_{i <= t} B_ti u_i,          B_ti = q_t . (prod_{i < j <= t} g_j) k_i
+//   S   = G_last S0 + sum_t (prod_{j > t} g_j) k_t u_t^T
+// u_t is v_t for the gated write; for the delta rule (I + diag(beta) A) U = diag(beta) (V - S0^T (G k)) with A_ti the
+// strictly lower part of k_t . (prod g) k_i, and the inverse is formed once per chunk and head. Products of decays are
+// formed by multiplication only, so no decay is ever divided out. A preparation kernel writes everything of a (chunk,
+// head) that does not depend on the state as one contiguous record of fp32 values:
+//   Gq [RC, DP] | Kd [RC, DP] | Gk [RC, DP] (delta) | G_last [DP] | B [RC, RC] | (I + diag(beta) A)^-1 diag(beta) (delta)
+__host__ __device__ constexpr int rec_floats(int DP, bool delta) { return (2 + delta) * RC * DP + DP + (1 + delta) * RC * RC; }
+
+// Sums of v[16] over the lanes that share a column group (LANES neighbouring lanes): lane rl is left with the sums of
+// tokens rl * TPL .. rl * TPL + TPL - 1 in v[0 .. TPL).
+template <int LANES>
+__device__ __forceinline__ void reduce_tokens(float (&v)[RC], int rl) {
+  int n = RC;
+#pragma unroll
+  for (int m = LANES / 2; m >= 1; m >>= 1) {
+    n >>= 1;
+    const bool up = (rl & m) != 0;
+#pragma unroll
+    for (int i = 0; i < RC / 2; ++i)
+      if (i < n) {
+        const float mine = up ? v[i + n] : v[i], other = up ? v[i] : v[i + n];
+        v[i] = mine + __shfl_xor_sync(0xffffffffu, other, m);
+      }
   }
-  return acc * sigmoid_f(acc);
 }
 
-template <typename A>
-__global__ void __launch_bounds__(256) delta_prep_kernel(const DeltaParams p) {
-  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-  const int seq = p.rv.tok_seq[t], pos = p.rv.tok_pos[t], pos0 = p.rv.pos0[seq];
-  const int C = 2 * p.G * p.d + p.H * p.dv;
-  const A* row = reinterpret_cast<const A*>(p.u) + (long long)t * p.u_ld;
-  A* ring = reinterpret_cast<A*>(p.ring) + (long long)p.rv.slot[seq] * p.taps * C;
-  for (int hh = warp; hh < 2 * p.G; hh += nw) {
-    float v[2 * QK_PAIRS];
+// Writes the record from q, k, g [RC][DP] in shared memory (rows past nt and columns past d: q = k = 0, g = 1 resp. 0).
+template <int DP, bool DELTA>
+__device__ __forceinline__ void write_record(const float* __restrict__ sq, const float* __restrict__ sk, const float* __restrict__ sg,
+                                             const float* __restrict__ sbeta, float* __restrict__ sA, float* __restrict__ rec, int nt) {
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  float* Gq = rec;
+  float* Kd = rec + RC * DP;
+  float* Gk = rec + 2 * RC * DP;
+  float* Gl = rec + (2 + DELTA) * RC * DP;
+  float* B = Gl + DP;
+  float* Tm = B + RC * RC;
+  for (int i = tid; i < 2 * DP; i += 256) {
+    const int c = i % DP;
+    float p = 1.f;
+    if (i < DP) {
+#pragma unroll
+      for (int t = 0; t < RC; ++t) {
+        p *= sg[t * DP + c];
+        Gq[t * DP + c] = sq[t * DP + c] * p;
+        if (DELTA) Gk[t * DP + c] = sk[t * DP + c] * p;
+      }
+      Gl[c] = p;
+    } else {
+#pragma unroll
+      for (int t = RC - 1; t >= 0; --t) {
+        Kd[t * DP + c] = sk[t * DP + c] * p;
+        p *= sg[t * DP + c];
+      }
+    }
+  }
+  constexpr int NC = (DP + 31) / 32;
+#pragma unroll 1
+  for (int half = 0; half < 2; ++half) {
+    const int t = half ? RC - 1 - warp : warp;     // a warp takes a short and a long row
+    float qp[NC], kp[NC], bq[RC], ak[RC];
+#pragma unroll
+    for (int n = 0; n < NC; ++n) {
+      const int c = lane + 32 * n;
+      qp[n] = c < DP ? sq[t * DP + c] : 0.f;
+      if (DELTA) kp[n] = c < DP ? sk[t * DP + c] : 0.f;
+    }
+#pragma unroll
+    for (int i = RC - 1; i >= 0; --i) {
+      bq[i] = ak[i] = 0.f;
+      if (i > t) continue;
+#pragma unroll
+      for (int n = 0; n < NC; ++n) {
+        const int c = lane + 32 * n;
+        if (DP >= 32 || c < DP) {
+          const float k = sk[i * DP + c], g = sg[i * DP + c];
+          bq[i] = fmaf(qp[n], k, bq[i]);
+          qp[n] *= g;
+          if (DELTA) {
+            ak[i] = fmaf(kp[n], k, ak[i]);
+            kp[n] *= g;
+          }
+        }
+      }
+    }
+    // over 32 lanes: the halves first, then the transposed reduction over 16 lanes
+#pragma unroll
+    for (int i = 0; i < RC; ++i) bq[i] += __shfl_xor_sync(0xffffffffu, bq[i], 16);
+    reduce_tokens<16>(bq, lane & 15);
+    if (lane < 16) B[t * RC + lane] = lane <= t ? bq[0] : 0.f;
+    if constexpr (DELTA) {
+#pragma unroll
+      for (int i = 0; i < RC; ++i) ak[i] += __shfl_xor_sync(0xffffffffu, ak[i], 16);
+      reduce_tokens<16>(ak, lane & 15);
+      if (lane < 16) sA[t * RC + lane] = lane < t ? ak[0] : 0.f;
+    }
+  }
+  if constexpr (DELTA) {
+    __syncthreads();
+    if (tid < RC) {        // column tid of the inverse, by forward substitution
+      float x[RC];
+#pragma unroll
+      for (int t = 0; t < RC; ++t) {
+        float s = t == tid ? 1.f : 0.f;
+#pragma unroll
+        for (int i = 0; i < t; ++i) s = fmaf(-sA[t * RC + i], x[i], s);
+        x[t] = sbeta[t] * s;
+        Tm[t * RC + tid] = x[t];
+      }
+    }
+  }
+}
+
+template <typename A, int DP>
+__global__ void __launch_bounds__(256) gate_chunk_kernel(const A* __restrict__ qr, const A* __restrict__ fr, long long ld,
+                                                         const float* __restrict__ bias, const float* __restrict__ lower,
+                                                         float* __restrict__ rec, const RaggedView rv, const ChunkView cv, int H, int d) {
+  extern __shared__ __align__(16) float sm[];
+  float* sq = sm;
+  float* sk = sq + RC * DP;
+  float* sg = sk + RC * DP;
+  const int ch = blockIdx.x, h = blockIdx.y, seq = cv.seq[ch], s0 = cv.start[ch];
+  const int row0 = rv.cu[seq] + s0, nt = min(RC, rv.cu[seq + 1] - row0);
+#pragma unroll 4
+  for (int i = threadIdx.x; i < RC * DP; i += 256) {
+    const int t = i / DP, c = i % DP;
+    float q = 0.f, f = 1.f;
+    if (t < nt && c < d) {
+      const long long o = (long long)(row0 + t) * ld + h * d + c;
+      const float z = to_f(qr[o]), l = lower[h * d + c];
+      q = z * sigmoid_f(z);
+      f = l + (1.f - l) * sigmoid_f(to_f(fr[o]) + bias[h * d + c]);
+    }
+    sq[i] = q;
+    sg[i] = f;
+    sk[i] = 1.f - f;       // 0 on padding
+  }
+  __syncthreads();
+  write_record<DP, false>(sq, sk, sg, nullptr, nullptr, rec + ((long long)ch * H + h) * rec_floats(DP, false), nt);
+}
+
+template <typename A, int DP, int MT>
+__global__ void __launch_bounds__(256) delta_chunk_kernel(const DeltaParams p, float* __restrict__ rec, const ChunkView cv) {
+  extern __shared__ __align__(16) float sm[];
+  float* sq = sm;
+  float* sk = sq + RC * DP;
+  float* sg = sk + RC * DP;
+  float* sA = sg + RC * DP;            // [RC, RC]
+  float* sb = sA + RC * RC;            // [RC]
+  const int ch = blockIdx.x, h = blockIdx.y, hq = h / (p.H / p.G), tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int seq = cv.seq[ch], s0 = cv.start[ch], row0 = p.rv.cu[seq] + s0, nt = min(RC, p.rv.cu[seq + 1] - row0);
+  const int pos = p.rv.pos0[seq] + s0, C = 2 * p.G * p.d + p.H * p.dv;
+  const A* u = reinterpret_cast<const A*>(p.u) + (long long)row0 * p.u_ld;
+  const A* ring = reinterpret_cast<const A*>(p.ring) + (long long)p.rv.slot[seq] * p.taps * C;
+  for (int i = tid; i < 2 * DP + p.dv; i += 256) {
+    const bool is_v = i >= 2 * DP;
+    const int which = i / DP, c = is_v ? i - 2 * DP : i % DP;
+    float y[RC];
+    if (is_v || c < p.d) {
+      const int col = is_v ? 2 * p.G * p.d + h * p.dv + c : (which * p.G + hq) * p.d + c;
+      conv_walk<A, RC, MT>(u, p.u_ld, p.wconv, p.taps, C, col, ring, pos, s0, nt, y);
+#pragma unroll
+      for (int t = 0; t < RC; ++t) y[t] *= sigmoid_f(y[t]);
+    } else {
+#pragma unroll
+      for (int t = 0; t < RC; ++t) y[t] = 0.f;
+    }
+    if (is_v) {
+      A* v = reinterpret_cast<A*>(p.v) + (long long)row0 * p.H * p.dv + (long long)h * p.dv + c;
+#pragma unroll
+      for (int t = 0; t < RC; ++t)
+        if (t < nt) v[(long long)t * p.H * p.dv] = from_f<A>(y[t]);
+    } else {
+      float* dst = which ? sk : sq;
+#pragma unroll
+      for (int t = 0; t < RC; ++t) dst[t * DP + c] = t < nt ? y[t] : 0.f;
+    }
+  }
+  const float al = -expf(p.a_log[h]);
+  const A* ar = reinterpret_cast<const A*>(p.a) + (long long)row0 * p.a_ld + (long long)h * p.d;
+#pragma unroll 4
+  for (int i = tid; i < RC * DP; i += 256) {
+    const int t = i / DP, c = i % DP;
+    sg[i] = (t < nt && c < p.d) ? expf(al * softplus_f(to_f(ar[(long long)t * p.a_ld + c]) + p.dt_bias[h * p.d + c])) : 1.f;
+  }
+  if (tid < RC)
+    sb[tid] = tid < nt ? sigmoid_f(to_f(reinterpret_cast<const A*>(p.b)[(long long)(row0 + tid) * p.b_ld + h])) : 0.f;
+  __syncthreads();
+  const float qs = 1.f / sqrtf((float)p.d);
+  for (int i = warp; i < 2 * RC; i += 8) {
+    float* row = (i < RC ? sq + i * DP : sk + (i - RC) * DP);
     float ss = 0.f;
-#pragma unroll
-    for (int n = 0; n < 2 * QK_PAIRS; ++n) {
-      const int i = lane + 32 * n;
-      v[n] = i < p.d ? conv_silu_at<A>(p, row, hh * p.d + i, C, pos, pos0, ring) : 0.f;
-      ss += v[n] * v[n];
-    }
+    for (int c = lane; c < DP; c += 32) ss += row[c] * row[c];
     ss = warp_sum(ss);
-    float r = 1.f / sqrtf(ss + 1e-6f);
-    if (hh < p.G) r *= 1.f / sqrtf((float)p.d);
-    float* out = (hh < p.G ? p.q + ((long long)t * p.G + hh) * p.d : p.k + ((long long)t * p.G + hh - p.G) * p.d);
-#pragma unroll
-    for (int n = 0; n < 2 * QK_PAIRS; ++n) {
-      const int i = lane + 32 * n;
-      if (i < p.d) out[i] = v[n] * r;
-    }
+    const float r = (i < RC ? qs : 1.f) / sqrtf(ss + 1e-6f);
+    for (int c = lane; c < DP; c += 32) row[c] *= r;
   }
-  for (int c = threadIdx.x; c < p.H * p.dv; c += blockDim.x)
-    reinterpret_cast<A*>(p.v)[(long long)t * p.H * p.dv + c] =
-        from_f<A>(conv_silu_at<A>(p, row, 2 * p.G * p.d + c, C, pos, pos0, ring));
-  const A* ar = reinterpret_cast<const A*>(p.a) + (long long)t * p.a_ld;
-  for (int c = threadIdx.x; c < p.H * p.d; c += blockDim.x) {
-    const float z = to_f(ar[c]) + p.dt_bias[c];
-    p.g[(long long)t * p.H * p.d + c] = expf(-expf(p.a_log[c / p.d]) * softplus_f(z));
-  }
-  for (int h = threadIdx.x; h < p.H; h += blockDim.x)
-    p.beta[(long long)t * p.H + h] = sigmoid_f(to_f(reinterpret_cast<const A*>(p.b)[(long long)t * p.b_ld + h]));
-  if (p.write_ring && p.taps > 1 && p.rv.slot[seq] >= 0)
-    for (int c = threadIdx.x; c < C; c += blockDim.x) ring[(long long)(pos % p.taps) * C + c] = row[c];
+  __syncthreads();
+  write_record<DP, true>(sq, sk, sg, sb, sA, rec + ((long long)ch * p.H + h) * rec_floats(DP, true), nt);
 }
 
-// ------------------------------------------------------------------ gated-write recurrence operands
-// q = silu(q_raw), f = lower + (1 - lower) sigmoid(f_raw + bias)
-template <typename A>
-__global__ void __launch_bounds__(256) gate_prep_kernel(const A* __restrict__ qr, const A* __restrict__ fr, long long ld,
-                                                        const float* __restrict__ bias, const float* __restrict__ lower,
-                                                        float* __restrict__ q, float* __restrict__ f, long long n, int C) {
-  const long long i = (long long)blockIdx.x * 256 + threadIdx.x;
-  if (i >= n) return;
-  const long long t = i / C;
-  const int c = (int)(i % C);
-  const float z = to_f(qr[t * ld + c]);
-  q[i] = z * sigmoid_f(z);
-  const float l = lower[c];
-  f[i] = l + (1.f - l) * sigmoid_f(to_f(fr[t * ld + c]) + bias[c]);
-}
-
-// ------------------------------------------------------------------ scan over the tokens of a portion
+// ------------------------------------------------------------------ scan over the chunks of a portion
 struct ScanParams {
-  const float* q; const float* g; const float* k;   // [T, Hq, d], [T, H, d] decay, [T, Hq, d] (delta rule only)
+  const float* rec;
   const void* v; long long v_ld;                    // [T, H dv]
-  const float* beta;                                // [T, H] (delta rule only)
   float* state;                                     // [slots, H, d, dv]
   float* o;                                         // [T, H, dv]
   RaggedView rv;
-  int H, Hq, d, dv;
+  ChunkView cv;
+  int* status;
+  int H, d, dv;
 };
 
 typedef unsigned long long u64;
@@ -128,47 +263,55 @@ __device__ __forceinline__ u64 mul2(u64 a, u64 b) {
   asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
   return r;
 }
-__device__ __forceinline__ void cp_async4(void* dst, const void* src) {
-  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+__device__ __forceinline__ void bulk_load(void* dst, const void* src, unsigned bytes, uint64_t* bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(smem_u32(dst)),
+               "l"(src), "r"(bytes), "r"(smem_u32(bar))
+               : "memory");
 }
-__device__ __forceinline__ void cp_async16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
 
-// One CTA walks the tokens of one portion for one head and a tile of value columns. The state tile lives in registers:
-// a thread holds 16 rows of CN columns, LANES neighbouring lanes share a column. Operand rows of TT tokens at a time are
-// copied to shared memory ahead of their use. The read-out sums of LANES tokens are reduced across the lanes together
-// (lane i ends up with token i), so they cost LANES - 1 shuffles per LANES tokens and stay off the recurrence's chain.
+// One CTA walks one portion for one head and a tile of value columns. The state tile lives in registers: a thread holds 16
+// rows of CN columns, LANES neighbouring lanes share a column. Records arrive by bulk copies one chunk ahead. A column
+// belongs to one warp, so the exchange of written values inside a chunk needs no block barrier.
 template <typename A, bool DELTA, int LANES, int CN>
 struct ScanCfg {
   static constexpr int DP = LANES * 16;              // padded rows
-  static constexpr int TT = DP <= 128 ? 16 : 8;
-  static constexpr int CT = 4 * (32 / LANES) * CN;   // columns per CTA
-  static constexpr int NARR = DELTA ? 3 : 2;
-  static constexpr int BUF = NARR * TT * DP;         // floats per buffer
-  static constexpr int VN = (TT * CT + 127) / 128;
-  static constexpr int SMEM = (2 * BUF + 2 * TT * CT + 2 * TT) * 4;
+  static constexpr int GW = 32 / LANES;              // column groups per warp
+  static constexpr int CW = GW * CN;                 // columns per warp
+  static constexpr int CT = 4 * CW;                  // columns per CTA
+  static constexpr int TPL = RC / LANES;             // tokens whose sums a lane ends up with
+  static constexpr int REC = rec_floats(DP, DELTA);
+  static constexpr int VN = (RC * CT + 127) / 128;
+  static constexpr int SMEM = (2 * REC + 2 * RC * CT + (DELTA ? 2 * RC * CT : 0)) * 4 + 64;
 };
 
 template <typename A, bool DELTA, int LANES, int CN>
 __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
   using Cfg = ScanCfg<A, DELTA, LANES, CN>;
-  constexpr int DP = Cfg::DP, TT = Cfg::TT, CT = Cfg::CT, BUF = Cfg::BUF, VN = Cfg::VN, GW = 32 / LANES;
-  constexpr int STEP = LANES < TT ? LANES : TT;      // tokens whose read-outs are reduced together
-  extern __shared__ __align__(16) float sm[];
-  float* sOp = sm;                       // [2][NARR][TT][DP]: q, decay, k
-  float* sV = sm + 2 * BUF;              // [2][TT][CT]
-  float* sB = sV + 2 * TT * CT;          // [2][TT]
-  const int seq = blockIdx.z, h = blockIdx.y, hq = h / (p.H / p.Hq);
+  constexpr int DP = Cfg::DP, CT = Cfg::CT, CW = Cfg::CW, GW = Cfg::GW, REC = Cfg::REC, TPL = Cfg::TPL, VN = Cfg::VN;
+  extern __shared__ __align__(128) float sm[];
+  float* sV = sm + 2 * REC;                          // [2][RC][CT]
+  float* sX = sV + 2 * RC * CT;                      // [RC][CT] per-warp column blocks: V - W, then U
+  float* sU = sX + RC * CT;
+  uint64_t* full = reinterpret_cast<uint64_t*>(sm + (Cfg::SMEM - 64) / 4);
+  volatile int* s_abort = reinterpret_cast<volatile int*>(full + 2);
+  const int seq = blockIdx.z, h = blockIdx.y;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int rl = lane % LANES, cloc = (warp * GW + lane / LANES) * CN, c0 = blockIdx.x * CT;
+  const int rl = lane % LANES, cw = (lane / LANES) * CN, cloc = warp * CW + cw, c0 = blockIdx.x * CT;
   const int row0 = p.rv.cu[seq], len = p.rv.cu[seq + 1] - row0;
   if (len <= 0) return;
+  const int ch0 = p.cv.first[seq], n_ch = (len + RC - 1) / RC;
   float* st = p.state + ((long long)p.rv.slot[seq] * p.H + h) * p.d * p.dv;
   const bool fresh = p.rv.pos0[seq] == 0;
-
+  const float* rec = p.rec + ((long long)ch0 * p.H + h) * REC;
+  const long long rec_step = (long long)p.H * REC;
+  if (tid == 0) {
+    mbar_init(&full[0], 1);
+    mbar_init(&full[1], 1);
+    *s_abort = 0;
+    mbar_fence_init();
+    mbar_expect_tx(&full[0], REC * 4);
+    bulk_load(sm, rec, REC * 4, &full[0]);
+  }
   u64 S[CN][8];
 #pragma unroll
   for (int cn = 0; cn < CN; ++cn) {
@@ -184,170 +327,170 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
       S[cn][i] = pack2(a, b);
     }
   }
-  if (p.d < DP)   // padding rows: zero operands, never overwritten
-    for (int i = tid; i < 2 * Cfg::NARR * TT * (DP - p.d); i += 128) sOp[(i / (DP - p.d)) * DP + p.d + i % (DP - p.d)] = 0.f;
-
-  const bool vec = (p.d & 3) == 0;
-  auto fetch = [&](int t0, int buf) {
-    const int nt = min(TT, len - t0);
-    float* dst = sOp + buf * BUF;
-#pragma unroll
-    for (int a = 0; a < Cfg::NARR; ++a) {
-      const float* src = a == 0 ? p.q : (a == 1 ? p.g : p.k);
-      const int heads = a == 1 ? p.H : p.Hq, hh = a == 1 ? h : hq;
-      if (vec) {
-        const int per = p.d / 4;
-        for (int i = tid; i < nt * per; i += 128) {
-          const int t = i / per, c = (i % per) * 4;
-          cp_async16(dst + (a * TT + t) * DP + c, src + ((long long)(row0 + t0 + t) * heads + hh) * p.d + c);
-        }
-      } else {
-        for (int i = tid; i < nt * p.d; i += 128) {
-          const int t = i / p.d, c = i % p.d;
-          cp_async4(dst + (a * TT + t) * DP + c, src + ((long long)(row0 + t0 + t) * heads + hh) * p.d + c);
-        }
-      }
-    }
-    cp_async_commit();
-  };
-  float vreg[VN], breg = 0.f;
+  float vreg[VN];
   auto load_v = [&](int t0) {
-    const int nt = min(TT, len - t0);
+    const int nt = min(RC, len - t0);
 #pragma unroll
     for (int n = 0; n < VN; ++n) {
       const int i = tid + n * 128, t = i / CT, c = c0 + i % CT;
-      vreg[n] = (i < TT * CT && t < nt && c < p.dv)
+      vreg[n] = (i < RC * CT && t < nt && c < p.dv)
                     ? to_f(reinterpret_cast<const A*>(p.v)[(long long)(row0 + t0 + t) * p.v_ld + (long long)h * p.dv + c])
                     : 0.f;
     }
-    if (DELTA && tid < TT) breg = tid < nt ? p.beta[(long long)(row0 + t0 + tid) * p.H + h] : 0.f;
   };
   auto put_v = [&](int buf) {
 #pragma unroll
     for (int n = 0; n < VN; ++n) {
       const int i = tid + n * 128;
-      if (i < TT * CT) sV[buf * TT * CT + i] = vreg[n];
+      if (i < RC * CT) sV[buf * RC * CT + i] = vreg[n];
     }
-    if (DELTA && tid < TT) sB[buf * TT + tid] = breg;
   };
-
-  const u64 one2 = pack2(1.f, 1.f), neg2 = pack2(-1.f, -1.f);
-  fetch(0, 0);
   load_v(0);
   put_v(0);
-  int buf = 0;
-  for (int t0 = 0; t0 < len; t0 += TT, buf ^= 1) {
-    const int nt = min(TT, len - t0);
-    const bool more = t0 + TT < len;
-    if (more) {
-      fetch(t0 + TT, buf ^ 1);
-      load_v(t0 + TT);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
-    const float* op = sOp + buf * BUF + rl * 4;
-    const float* vp = sV + buf * TT * CT + cloc;
-    for (int ts = 0; ts < nt; ts += STEP) {
-      float oacc[CN][STEP];
+  __syncthreads();
+  // sum over this thread's rows of S[cn] * op[t][rows], for the 16 tokens, then over the lanes of the column
+  auto project = [&](const float* op, float (&acc)[CN][RC]) {
 #pragma unroll
-      for (int s = 0; s < STEP; ++s) {
-        const int t = ts + s;
+    for (int t = 0; t < RC; ++t) {
+      u64 a[CN][2];
 #pragma unroll
-        for (int cn = 0; cn < CN; ++cn) oacc[cn][s] = 0.f;
-        if (t < nt) {
-          u64 q[8], g[8], k[8];
+      for (int cn = 0; cn < CN; ++cn) a[cn][0] = a[cn][1] = 0;
 #pragma unroll
-          for (int c = 0; c < 4; ++c) {
-            const ulonglong2 q4 = *reinterpret_cast<const ulonglong2*>(op + t * DP + c * LANES * 4);
-            const ulonglong2 g4 = *reinterpret_cast<const ulonglong2*>(op + (TT + t) * DP + c * LANES * 4);
-            q[2 * c] = q4.x; q[2 * c + 1] = q4.y;
-            g[2 * c] = g4.x; g[2 * c + 1] = g4.y;
-            if constexpr (DELTA) {
-              const ulonglong2 k4 = *reinterpret_cast<const ulonglong2*>(op + (2 * TT + t) * DP + c * LANES * 4);
-              k[2 * c] = k4.x; k[2 * c + 1] = k4.y;
-            } else {
-              k[2 * c] = fma2(g4.x, neg2, one2);
-              k[2 * c + 1] = fma2(g4.y, neg2, one2);
-            }
-          }
-          if constexpr (DELTA) {
-            const float beta = sB[buf * TT + t];
-            float w[CN];
+      for (int c = 0; c < 4; ++c) {
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(op + t * DP + c * LANES * 4 + rl * 4);
 #pragma unroll
-            for (int cn = 0; cn < CN; ++cn) {
-              u64 a0 = 0, a1 = 0;
-#pragma unroll
-              for (int i = 0; i < 8; i += 2) {
-                S[cn][i] = mul2(g[i], S[cn][i]);
-                S[cn][i + 1] = mul2(g[i + 1], S[cn][i + 1]);
-                a0 = fma2(S[cn][i], k[i], a0);
-                a1 = fma2(S[cn][i + 1], k[i + 1], a1);
-              }
-              const float2 x = unpack2(a0), y = unpack2(a1);
-              w[cn] = (x.x + x.y) + (y.x + y.y);
-            }
-#pragma unroll
-            for (int m = LANES / 2; m >= 1; m >>= 1)
-#pragma unroll
-              for (int cn = 0; cn < CN; ++cn) w[cn] += __shfl_xor_sync(0xffffffffu, w[cn], m);
-#pragma unroll
-            for (int cn = 0; cn < CN; ++cn) {
-              const float u = beta * (vp[t * CT + cn] - w[cn]);
-              const u64 u2 = pack2(u, u);
-              u64 a0 = 0, a1 = 0;
-#pragma unroll
-              for (int i = 0; i < 8; i += 2) {
-                S[cn][i] = fma2(k[i], u2, S[cn][i]);
-                S[cn][i + 1] = fma2(k[i + 1], u2, S[cn][i + 1]);
-                a0 = fma2(S[cn][i], q[i], a0);
-                a1 = fma2(S[cn][i + 1], q[i + 1], a1);
-              }
-              const float2 x = unpack2(a0), y = unpack2(a1);
-              oacc[cn][s] = (x.x + x.y) + (y.x + y.y);
-            }
-          } else {
-#pragma unroll
-            for (int cn = 0; cn < CN; ++cn) {
-              const float v = vp[t * CT + cn];
-              const u64 v2 = pack2(v, v);
-              u64 a0 = 0, a1 = 0;
-#pragma unroll
-              for (int i = 0; i < 8; i += 2) {
-                S[cn][i] = fma2(g[i], S[cn][i], mul2(k[i], v2));
-                S[cn][i + 1] = fma2(g[i + 1], S[cn][i + 1], mul2(k[i + 1], v2));
-                a0 = fma2(S[cn][i], q[i], a0);
-                a1 = fma2(S[cn][i + 1], q[i + 1], a1);
-              }
-              const float2 x = unpack2(a0), y = unpack2(a1);
-              oacc[cn][s] = (x.x + x.y) + (y.x + y.y);
-            }
-          }
+        for (int cn = 0; cn < CN; ++cn) {
+          a[cn][0] = fma2(S[cn][2 * c], x.x, a[cn][0]);
+          a[cn][1] = fma2(S[cn][2 * c + 1], x.y, a[cn][1]);
         }
       }
-      // token-transposed reduction over the lanes that share a column (LANES can exceed STEP: plain steps first)
 #pragma unroll
       for (int cn = 0; cn < CN; ++cn) {
-#pragma unroll
-        for (int m = LANES / 2; m >= STEP && m >= 1; m >>= 1)
-#pragma unroll
-          for (int s = 0; s < STEP; ++s) oacc[cn][s] += __shfl_xor_sync(0xffffffffu, oacc[cn][s], m);
-#pragma unroll
-        for (int m = STEP / 2; m >= 1; m >>= 1) {
-          const bool up = (rl & m) != 0;
-#pragma unroll
-          for (int s = 0; s < m; ++s) {
-            const float mine = up ? oacc[cn][s + m] : oacc[cn][s], other = up ? oacc[cn][s] : oacc[cn][s + m];
-            oacc[cn][s] = mine + __shfl_xor_sync(0xffffffffu, other, m);
-          }
-        }
-        const int t = ts + rl % STEP, col = c0 + cloc + cn;
-        if (rl < STEP && t < nt && col < p.dv) p.o[((long long)(row0 + t0 + t) * p.H + h) * p.dv + col] = oacc[cn][0];
+        const float2 x = unpack2(a[cn][0]), y = unpack2(a[cn][1]);
+        acc[cn][t] = (x.x + x.y) + (y.x + y.y);
       }
     }
-    if (more) put_v(buf ^ 1);
+#pragma unroll
+    for (int cn = 0; cn < CN; ++cn) reduce_tokens<LANES>(acc[cn], rl);
+  };
+  bool ok = true;
+  for (int ci = 0; ci < n_ch; ++ci) {
+    const int buf = ci & 1, t0 = ci * RC, nt = min(RC, len - t0);
+    if (ci + 1 < n_ch) {
+      if (tid == 0) {
+        mbar_expect_tx(&full[buf ^ 1], REC * 4);
+        bulk_load(sm + (buf ^ 1) * REC, rec + (ci + 1) * rec_step, REC * 4, &full[buf ^ 1]);
+      }
+      load_v(t0 + RC);
+    }
+    ok = mbar_wait_warp(&full[buf], (ci >> 1) & 1, s_abort, p.status, ST_TIMEOUT_PRODUCER);
+    if (!ok) break;
+    const float* R = sm + buf * REC;
+    const float* Kd = R + RC * DP;
+    const float* Gl = R + (2 + DELTA) * RC * DP;
+    const float* B = Gl + DP;
+    const float* V = sV + buf * RC * CT;
+    const float* U = V;
+    if constexpr (DELTA) {
+      float w[CN][RC];
+      project(R + 2 * RC * DP, w);
+#pragma unroll
+      for (int i = 0; i < TPL; ++i)
+#pragma unroll
+        for (int cn = 0; cn < CN; ++cn) {
+          const int t = rl * TPL + i;
+          sX[t * CT + cloc + cn] = V[t * CT + cloc + cn] - w[cn][i];
+        }
+    }
+    float q[CN][RC];
+    project(R, q);
+    if constexpr (DELTA) {
+      __syncwarp();
+      const float* Tm = B + RC * RC;
+      float x[CN][TPL];
+#pragma unroll
+      for (int cn = 0; cn < CN; ++cn)
+#pragma unroll
+        for (int i = 0; i < TPL; ++i) x[cn][i] = 0.f;
+#pragma unroll
+      for (int j = 0; j < RC; j += 4) {
+        float xv[CN][4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int cn = 0; cn < CN; ++cn) xv[cn][e] = sX[(j + e) * CT + cloc + cn];
+#pragma unroll
+        for (int i = 0; i < TPL; ++i) {
+          const float4 m = *reinterpret_cast<const float4*>(Tm + (rl * TPL + i) * RC + j);
+#pragma unroll
+          for (int cn = 0; cn < CN; ++cn)
+            x[cn][i] = fmaf(m.w, xv[cn][3], fmaf(m.z, xv[cn][2], fmaf(m.y, xv[cn][1], fmaf(m.x, xv[cn][0], x[cn][i]))));
+        }
+      }
+#pragma unroll
+      for (int i = 0; i < TPL; ++i)
+#pragma unroll
+        for (int cn = 0; cn < CN; ++cn) sU[(rl * TPL + i) * CT + cloc + cn] = x[cn][i];
+      __syncwarp();
+      U = sU;
+    }
+    // read-out: the chunk's own writes join what the state held before it
+#pragma unroll
+    for (int j = 0; j < RC; j += 4) {
+      float uv[CN][4];
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+#pragma unroll
+        for (int cn = 0; cn < CN; ++cn) uv[cn][e] = U[(j + e) * CT + cloc + cn];
+#pragma unroll
+      for (int i = 0; i < TPL; ++i) {
+        const float4 m = *reinterpret_cast<const float4*>(B + (rl * TPL + i) * RC + j);
+#pragma unroll
+        for (int cn = 0; cn < CN; ++cn)
+          q[cn][i] = fmaf(m.w, uv[cn][3], fmaf(m.z, uv[cn][2], fmaf(m.y, uv[cn][1], fmaf(m.x, uv[cn][0], q[cn][i]))));
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < TPL; ++i) {
+      const int t = rl * TPL + i;
+#pragma unroll
+      for (int cn = 0; cn < CN; ++cn)
+        if (t < nt && c0 + cloc + cn < p.dv) p.o[((long long)(row0 + t0 + t) * p.H + h) * p.dv + c0 + cloc + cn] = q[cn][i];
+    }
+    // state behind the chunk
+#pragma unroll
+    for (int c = 0; c < 4; ++c) {
+      const ulonglong2 g = *reinterpret_cast<const ulonglong2*>(Gl + c * LANES * 4 + rl * 4);
+#pragma unroll
+      for (int cn = 0; cn < CN; ++cn) {
+        S[cn][2 * c] = mul2(S[cn][2 * c], g.x);
+        S[cn][2 * c + 1] = mul2(S[cn][2 * c + 1], g.y);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < RC; ++t) {
+      u64 u2[CN];
+#pragma unroll
+      for (int cn = 0; cn < CN; ++cn) {
+        const float x = U[t * CT + cloc + cn];
+        u2[cn] = pack2(x, x);
+      }
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(Kd + t * DP + c * LANES * 4 + rl * 4);
+#pragma unroll
+        for (int cn = 0; cn < CN; ++cn) {
+          S[cn][2 * c] = fma2(k.x, u2[cn], S[cn][2 * c]);
+          S[cn][2 * c + 1] = fma2(k.y, u2[cn], S[cn][2 * c + 1]);
+        }
+      }
+    }
+    if (ci + 1 < n_ch) put_v(buf ^ 1);
     __syncthreads();
+  }
+  if (*s_abort) {
+    bounded_delay_ns(2000000);
+    return;
   }
 #pragma unroll
   for (int cn = 0; cn < CN; ++cn) {
@@ -367,7 +510,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
 // One CTA per (head, sequence): operands from the projected rows (convolution, unit norms, gates), one state update with
 // the state tile in registers between its two passes, read-out, per-head norm and output gate.
 struct StepParams {
-  DeltaParams in;             // delta rule: projected rows and constants (q, k, g, v, beta unused)
+  DeltaParams in;             // delta rule: projected rows and constants (v unused)
   const void* qr; const void* fr; const void* vr; long long ld;   // gated write: projected rows
   const float* fbias; const float* lower;
   float* state;
@@ -380,7 +523,7 @@ struct StepParams {
 };
 
 template <typename A, bool DELTA, int VEC, int NR>
-__global__ void __launch_bounds__(256) recur_step_kernel(const StepParams p) {
+__global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1) recur_step_kernel(const StepParams p) {
   extern __shared__ __align__(16) float sm[];
   float* sq = sm;             // [d]
   float* sk = sq + p.d;       // [d]
@@ -394,76 +537,17 @@ __global__ void __launch_bounds__(256) recur_step_kernel(const StepParams p) {
   const int slot = p.rv.slot[seq];
   if (slot < 0) return;       // padding row of a captured launch
   const int pos = p.rv.pos0[seq];
-  float beta = 0.f;
-  if constexpr (DELTA) {
-    const DeltaParams& in = p.in;
-    const int C = 2 * in.G * in.d + in.H * in.dv;
-    const A* row = reinterpret_cast<const A*>(in.u) + (long long)t * in.u_ld;
-    A* ring = reinterpret_cast<A*>(in.ring) + (long long)slot * in.taps * C;
-    if (warp < 2) {           // warp 0: query, warp 1: key
-      const int ch0 = (warp * in.G + hq) * in.d;
-      float ss = 0.f;
-      float* dst = warp ? sk : sq;
-      for (int i = lane; i < in.d; i += 32) {
-        const float x = conv_silu_at<A>(in, row, ch0 + i, C, pos, pos, ring);
-        dst[i] = x;
-        ss += x * x;
-      }
-      ss = warp_sum(ss);
-      float r = 1.f / sqrtf(ss + 1e-6f);
-      if (warp == 0) r *= 1.f / sqrtf((float)in.d);
-      for (int i = lane; i < in.d; i += 32) dst[i] *= r;
-    } else if (warp < 5) {
-      for (int c = tid - 64; c < in.dv; c += 96)
-        sv[c] = to_f(from_f<A>(conv_silu_at<A>(in, row, 2 * in.G * in.d + h * in.dv + c, C, pos, pos, ring)));
-    } else {
-      const A* ar = reinterpret_cast<const A*>(in.a) + (long long)t * in.a_ld + (long long)h * in.d;
-      const float al = -expf(in.a_log[h]);
-      for (int i = tid - 160; i < in.d; i += 96) sg[i] = expf(al * softplus_f(to_f(ar[i]) + in.dt_bias[h * in.d + i]));
-    }
-    beta = sigmoid_f(to_f(reinterpret_cast<const A*>(in.b)[(long long)t * in.b_ld + h]));
-    if (in.taps > 1) {
-      // the entry this token fills is not one that any head reads in this step
-      A* e = ring + (long long)(pos % in.taps) * C;
-      if (h % (p.H / p.Hq) == 0)
-        for (int i = tid; i < 2 * in.d; i += 256) {
-          const int ch = ((i / in.d) * in.G + hq) * in.d + i % in.d;
-          e[ch] = row[ch];
-        }
-      for (int c = tid; c < in.dv; c += 256) {
-        const int ch = 2 * in.G * in.d + h * in.dv + c;
-        e[ch] = row[ch];
-      }
-    }
-  } else {
-    const A* qr = reinterpret_cast<const A*>(p.qr) + (long long)t * p.ld + (long long)h * p.d;
-    const A* fr = reinterpret_cast<const A*>(p.fr) + (long long)t * p.ld + (long long)h * p.d;
-    const A* vr = reinterpret_cast<const A*>(p.vr) + (long long)t * p.ld + (long long)h * p.dv;
-    for (int i = tid; i < p.d; i += 256) {
-      const float z = to_f(qr[i]);
-      sq[i] = z * sigmoid_f(z);
-      const float l = p.lower[h * p.d + i];
-      const float f = l + (1.f - l) * sigmoid_f(to_f(fr[i]) + p.fbias[h * p.d + i]);
-      sg[i] = f;
-      sk[i] = 1.f - f;
-    }
-    for (int c = tid; c < p.dv; c += 256) sv[c] = to_f(vr[c]);
-  }
-  __syncthreads();
-
   const int lpr = p.lpr, RG = 256 / lpr, rg = tid / lpr, cl = tid % lpr;
   float* st = p.state + ((long long)slot * p.H + h) * p.d * p.dv;
   const bool fresh = pos == 0;
-  for (int ct = 0; ct < p.dv; ct += lpr * VEC) {
-    const int col = ct + cl * VEC;
-    const bool on = col < p.dv;
-    float S[NR][VEC];
+  float S[NR][VEC];
+  auto load_state = [&](int col) {
 #pragma unroll
     for (int n = 0; n < NR; ++n) {
       const int r = rg + n * RG;
 #pragma unroll
       for (int e = 0; e < VEC; ++e) S[n][e] = 0.f;
-      if (!fresh && on && r < p.d) {
+      if (!fresh && col < p.dv && r < p.d) {
         if constexpr (VEC == 4) {
           const float4 x = *reinterpret_cast<const float4*>(st + (long long)r * p.dv + col);
           S[n][0] = x.x; S[n][1] = x.y; S[n][2] = x.z; S[n][3] = x.w;
@@ -472,6 +556,63 @@ __global__ void __launch_bounds__(256) recur_step_kernel(const StepParams p) {
         }
       }
     }
+  };
+  load_state(cl * VEC);       // in flight while the operands are prepared
+  float beta = 0.f;
+  if constexpr (DELTA) {
+    const DeltaParams& in = p.in;
+    const int C = 2 * in.G * in.d + in.H * in.dv;
+    const A* row = reinterpret_cast<const A*>(in.u) + (long long)t * in.u_ld;
+    A* ring = reinterpret_cast<A*>(in.ring) + (long long)slot * in.taps * C;
+    A* e = ring + (long long)(pos % in.taps) * C;     // the entry this token fills; no head reads it in this step
+    const bool owner = h % (p.H / p.Hq) == 0;
+    for (int i = tid; i < 2 * in.d + in.dv; i += 256) {
+      const bool is_v = i >= 2 * in.d;
+      const int which = i / in.d, c = is_v ? i - 2 * in.d : i % in.d;
+      const int col = is_v ? 2 * in.G * in.d + h * in.dv + c : (which * in.G + hq) * in.d + c;
+      float y[1];
+      conv_walk<A, 1, 8>(row, in.u_ld, in.wconv, in.taps, C, col, ring, pos, 0, 1, y);
+      const float x = y[0] * sigmoid_f(y[0]);
+      if (is_v) sv[c] = to_f(from_f<A>(x));
+      else (which ? sk : sq)[c] = x;
+      if (in.taps > 1 && (is_v || owner)) e[col] = row[col];
+    }
+    const A* ar = reinterpret_cast<const A*>(in.a) + (long long)t * in.a_ld + (long long)h * in.d;
+    const float al = -expf(in.a_log[h]);
+    for (int i = tid; i < in.d; i += 256) sg[i] = expf(al * softplus_f(to_f(ar[i]) + in.dt_bias[h * in.d + i]));
+    beta = sigmoid_f(to_f(reinterpret_cast<const A*>(in.b)[(long long)t * in.b_ld + h]));
+    __syncthreads();
+    if (warp < 2) {           // unit norms; the query also takes d^-1/2
+      float* x = warp ? sk : sq;
+      float ss = 0.f;
+      for (int i = lane; i < in.d; i += 32) ss += x[i] * x[i];
+      ss = warp_sum(ss);
+      const float r = (warp ? 1.f : 1.f / sqrtf((float)in.d)) / sqrtf(ss + 1e-6f);
+      for (int i = lane; i < in.d; i += 32) x[i] *= r;
+    }
+  } else {
+    const A* qr = reinterpret_cast<const A*>(p.qr) + (long long)t * p.ld + (long long)h * p.d;
+    const A* fr = reinterpret_cast<const A*>(p.fr) + (long long)t * p.ld + (long long)h * p.d;
+    const A* vr = reinterpret_cast<const A*>(p.vr) + (long long)t * p.ld + (long long)h * p.dv;
+    for (int i = tid; i < p.d + p.dv; i += 256) {
+      if (i < p.d) {
+        const float z = to_f(qr[i]);
+        sq[i] = z * sigmoid_f(z);
+        const float l = p.lower[h * p.d + i];
+        const float f = l + (1.f - l) * sigmoid_f(to_f(fr[i]) + p.fbias[h * p.d + i]);
+        sg[i] = f;
+        sk[i] = 1.f - f;
+      } else {
+        sv[i - p.d] = to_f(vr[i - p.d]);
+      }
+    }
+  }
+  __syncthreads();
+
+  for (int ct = 0; ct < p.dv; ct += lpr * VEC) {
+    const int col = ct + cl * VEC;
+    const bool on = col < p.dv;
+    if (ct) load_state(col);
     // sum over the state rows of acc[VEC], result for this thread's columns in every thread
     auto reduce = [&](float (&acc)[VEC]) {
       for (int m = lpr; m < 32; m <<= 1)
@@ -555,35 +696,87 @@ using namespace sx;
 
 static void fill_delta(DeltaParams* p, const SxDeltaArgs* a) {
   p->u = a->u; p->u_ld = a->u_ld; p->wconv = a->wconv; p->ring = a->ring; p->b = a->b; p->b_ld = a->b_ld; p->a = a->a; p->a_ld = a->a_ld;
-  p->a_log = a->a_log; p->dt_bias = a->dt_bias; p->q = a->q; p->k = a->k; p->g = a->g; p->v = a->v; p->beta = a->beta;
+  p->a_log = a->a_log; p->dt_bias = a->dt_bias; p->v = a->v;
   p->rv = view(&a->ragged);
-  p->T = a->T; p->H = a->H; p->G = a->G; p->d = a->d; p->dv = a->dv; p->taps = a->taps; p->write_ring = a->write_ring;
+  p->T = a->T; p->H = a->H; p->G = a->G; p->d = a->d; p->dv = a->dv; p->taps = a->taps;
 }
-extern "C" int sx_delta_prep(const SxDeltaArgs* a, cudaStream_t st) {
-  if (a->T <= 0) return 0;
-  if (a->d > 64 * QK_PAIRS || a->G <= 0 || a->H % a->G) return -1;
+static int pad_rows(int d) { return d <= 16 ? 16 : d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
+
+// Floats of scratch that the records of one (chunk, head) take.
+extern "C" int sx_recur_record(int d, int delta) { return rec_floats(pad_rows(d), delta != 0); }
+
+template <typename K>
+static int allow_smem(K kern, int bytes, bool* done) {
+  if (!*done && bytes > 48 * 1024) {
+    if (cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, bytes) != cudaSuccess) return -10;
+    *done = true;
+  }
+  return 0;
+}
+
+template <typename A, int DP>
+static int launch_gate_chunks(const SxGateArgs* a, cudaStream_t st) {
+  static bool set = false;
+  const int smem = 3 * RC * DP * 4;
+  if (int rc = allow_smem(gate_chunk_kernel<A, DP>, smem, &set)) return rc;
+  gate_chunk_kernel<A, DP><<<dim3(a->chunks.n, a->H), 256, smem, st>>>((const A*)a->q, (const A*)a->f, a->ld, a->bias, a->lower, a->rec,
+                                                                       view(&a->ragged), chunks(&a->chunks), a->H, a->d);
+  return last_rc();
+}
+
+// Records of the gated-write recurrence from projected rows (q and forget-gate logits).
+extern "C" int sx_gate_chunks(const SxGateArgs* a, cudaStream_t st) {
+  if (a->chunks.n <= 0) return 0;
+  if (a->d <= 0 || a->d > 256) return -1;
+  SX_ACT_DISPATCH(a->f32, {
+    switch (pad_rows(a->d)) {
+      case 16: return launch_gate_chunks<A, 16>(a, st);
+      case 32: return launch_gate_chunks<A, 32>(a, st);
+      case 64: return launch_gate_chunks<A, 64>(a, st);
+      case 128: return launch_gate_chunks<A, 128>(a, st);
+      default: return launch_gate_chunks<A, 256>(a, st);
+    }
+  });
+  return 0;
+}
+
+template <typename A, int DP, int MT>
+static int launch_delta_chunks(const DeltaParams& p, float* rec, const ChunkView& cv, cudaStream_t st) {
+  static bool set = false;
+  const int smem = (3 * RC * DP + RC * RC + RC) * 4;
+  if (int rc = allow_smem(delta_chunk_kernel<A, DP, MT>, smem, &set)) return rc;
+  delta_chunk_kernel<A, DP, MT><<<dim3(cv.n_chunks, p.H), 256, smem, st>>>(p, rec, cv);
+  return last_rc();
+}
+template <typename A, int DP>
+static int pick_delta_chunks(const DeltaParams& p, float* rec, const ChunkView& cv, cudaStream_t st) {
+  return p.taps <= 4 ? launch_delta_chunks<A, DP, 4>(p, rec, cv, st) : launch_delta_chunks<A, DP, 8>(p, rec, cv, st);
+}
+
+// Records and convolved values of the gated delta rule from projected rows.
+extern "C" int sx_delta_chunks(const SxDeltaArgs* a, const SxChunks* c, float* rec, cudaStream_t st) {
+  if (c->n <= 0) return 0;
+  if (a->d <= 0 || a->d > 256 || a->G <= 0 || a->H % a->G || a->taps < 1 || a->taps > 8) return -1;
   DeltaParams p;
   fill_delta(&p, a);
-  SX_ACT_DISPATCH(a->f32, (delta_prep_kernel<A><<<a->T, 256, 0, st>>>(p)));
-  return last_rc();
-}
-extern "C" int sx_gate_prep(const void* qr, const void* fr, long long ld, const float* bias, const float* lower, float* q, float* f,
-                            int T, int C, int f32, cudaStream_t st) {
-  const long long n = (long long)T * C;
-  if (n <= 0) return 0;
-  SX_ACT_DISPATCH(f32, (gate_prep_kernel<A><<<(unsigned)((n + 255) / 256), 256, 0, st>>>((const A*)qr, (const A*)fr, ld, bias, lower, q, f, n, C)));
-  return last_rc();
+  const ChunkView cv = chunks(c);
+  SX_ACT_DISPATCH(a->f32, {
+    switch (pad_rows(a->d)) {
+      case 16: return pick_delta_chunks<A, 16>(p, rec, cv, st);
+      case 32: return pick_delta_chunks<A, 32>(p, rec, cv, st);
+      case 64: return pick_delta_chunks<A, 64>(p, rec, cv, st);
+      case 128: return pick_delta_chunks<A, 128>(p, rec, cv, st);
+      default: return pick_delta_chunks<A, 256>(p, rec, cv, st);
+    }
+  });
+  return 0;
 }
 
 template <typename A, bool DELTA, int LANES, int CN>
 static int launch_scan(const ScanParams& p, cudaStream_t st) {
   using Cfg = ScanCfg<A, DELTA, LANES, CN>;
   static bool set = false;
-  if (!set) {
-    if (cudaFuncSetAttribute(recur_scan_kernel<A, DELTA, LANES, CN>, cudaFuncAttributeMaxDynamicSharedMemorySize, Cfg::SMEM) != cudaSuccess)
-      return -10;
-    set = true;
-  }
+  if (int rc = allow_smem(recur_scan_kernel<A, DELTA, LANES, CN>, Cfg::SMEM, &set)) return rc;
   dim3 grid((p.dv + Cfg::CT - 1) / Cfg::CT, p.H, p.rv.n);
   recur_scan_kernel<A, DELTA, LANES, CN><<<grid, 128, Cfg::SMEM, st>>>(p);
   return last_rc();
@@ -591,8 +784,7 @@ static int launch_scan(const ScanParams& p, cudaStream_t st) {
 template <typename A, bool DELTA>
 static int pick_scan(const ScanParams& p, cudaStream_t st) {
   // two columns per thread once one column per thread would put more than two CTAs on every SM
-  const int lanes = p.d <= 16 ? 1 : p.d <= 32 ? 2 : p.d <= 64 ? 4 : p.d <= 128 ? 8 : 16;
-  const int ct1 = 4 * (32 / lanes);
+  const int lanes = pad_rows(p.d) / 16, ct1 = 4 * (32 / lanes);
   const bool wide = (long long)((p.dv + ct1 - 1) / ct1) * p.H * p.rv.n > 2 * 148;
 #define SX_SCAN(L) return wide ? launch_scan<A, DELTA, L, 2>(p, st) : launch_scan<A, DELTA, L, 1>(p, st)
   switch (lanes) {
@@ -605,14 +797,14 @@ static int pick_scan(const ScanParams& p, cudaStream_t st) {
 #undef SX_SCAN
 }
 
-// delta != 0: gated delta rule; else the gated write. The portion's rows must be in order; portions are independent.
+// delta != 0: gated delta rule; else the gated write. Portions are independent of each other.
 extern "C" int sx_recur_scan(const SxScanArgs* a, cudaStream_t st) {
   if (a->ragged.n <= 0) return 0;
-  if (a->d <= 0 || a->d > 256 || a->dv <= 0 || a->Hq <= 0 || a->H % a->Hq) return -1;
+  if (a->d <= 0 || a->d > 256 || a->dv <= 0) return -1;
   ScanParams p;
-  p.q = a->q; p.g = a->g; p.k = a->k; p.v = a->v; p.v_ld = a->v_ld; p.beta = a->beta; p.state = a->state; p.o = a->o;
-  p.rv = view(&a->ragged);
-  p.H = a->H; p.Hq = a->Hq; p.d = a->d; p.dv = a->dv;
+  p.rec = a->rec; p.v = a->v; p.v_ld = a->v_ld; p.state = a->state; p.o = a->o; p.status = a->status;
+  p.rv = view(&a->ragged); p.cv = chunks(&a->chunks);
+  p.H = a->H; p.d = a->d; p.dv = a->dv;
   SX_ACT_DISPATCH(a->f32, { return a->delta ? pick_scan<A, true>(p, st) : pick_scan<A, false>(p, st); });
   return 0;
 }
@@ -633,7 +825,7 @@ static int launch_step(const StepParams& p, cudaStream_t st) {
 
 extern "C" int sx_recur_step(const SxStepArgs* a, cudaStream_t st) {
   if (a->ragged.n <= 0) return 0;
-  if (a->d <= 0 || a->d > 256 || a->dv <= 0 || a->Hq <= 0 || a->H % a->Hq) return -1;
+  if (a->d <= 0 || a->d > 256 || a->dv <= 0 || a->Hq <= 0 || a->H % a->Hq || (a->delta && (a->in.taps < 1 || a->in.taps > 8))) return -1;
   StepParams p;
   p.rv = view(&a->ragged);
   if (a->delta) {

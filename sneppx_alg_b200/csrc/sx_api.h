@@ -229,6 +229,13 @@ typedef struct SxRagged {
   const int* tok_pos;   // [T] position of each row
   int n;
 } SxRagged;
+// The portions of a batch cut into chunks of 16 rows. Device int32 arrays.
+typedef struct SxChunks {
+  const int* seq;       // [n] portion of each chunk
+  const int* start;     // [n] first row of the chunk within its portion
+  const int* first;     // [portions + 1] first chunk of each portion
+  int n;
+} SxChunks;
 // f32: 1 for 32-bit activations, 0 for bf16. Norm weights, convolution weights and biases are fp32.
 int sx_embed_f32(const void* table, const int* ids, float* x, int T, int width, int f32, cudaStream_t stream);
 int sx_rmsnorm_f32(const float* x, const float* w, const int* rows, void* y, int T, int width, float eps, int f32, cudaStream_t stream);
@@ -246,14 +253,16 @@ typedef struct SxQkvArgs {
   const double* inv_freq;         // [rot / 2]
   const float* talk;              // [H, H], with qmix_out
   float* q_out;                   // [T, H, d] or null
-  void* qmix_out;                 // [T, H, G d] queries with the head mix folded in, or null
+  void* qmix_out;                 // [T, H, qmix_ld] queries with the head mix folded in (zeros past G d), or null
+  int qmix_ld;
   void* k_out; void* v_out;       // packed keys / values, or null; value head j at column j * dvp
   long long k_ld, v_ld;
   const int* kv_row;              // [T] packed row (null: row index)
   void* k_cache; void* v_cache;   // [entries, G, d] / [entries, G, dv]
   const int* cache_entry;         // [T], -1: not stored
   SxRagged ragged;
-  int T, H, G, d, dv, dvp, taps, rot, write_ring, f32;
+  SxChunks chunks;                // n == 0: one row per portion (decoding); the row then also goes to its ring entry
+  int T, H, G, d, dv, dvp, taps, rot, f32;
   float eps;
 } SxQkvArgs;
 int sx_qkv_prep(const SxQkvArgs* args, cudaStream_t stream);
@@ -266,21 +275,31 @@ typedef struct SxDeltaArgs {
   const void* b; long long b_ld;
   const void* a; long long a_ld;
   const float* a_log; const float* dt_bias;
-  float* q; float* k; float* g; void* v; float* beta;
+  void* v;                        // [T, H dv] convolved values (prompt form)
   SxRagged ragged;
-  int T, H, G, d, dv, taps, write_ring, f32;
+  int T, H, G, d, dv, taps, f32;
 } SxDeltaArgs;
-int sx_delta_prep(const SxDeltaArgs* args, cudaStream_t stream);
-int sx_gate_prep(const void* qr, const void* fr, long long ld, const float* bias, const float* lower, float* q, float* f, int T,
-                 int C, int f32, cudaStream_t stream);
-// Scan of a portion; state [slots, H, d, dv] fp32, o [T, H, dv] fp32. Head h reads q / k head h / (H / Hq).
-typedef struct SxScanArgs {
-  const float* q; const float* g; const float* k;
-  const void* v; long long v_ld;
-  const float* beta;
-  float* state; float* o;
+// Prompt form of the recurrences: a preparation kernel writes one record of `sx_recur_record` floats per (chunk, head), then
+// the scan walks each portion from its slot's state (empty at position 0), stores the state back and writes the read-outs.
+typedef struct SxGateArgs {
+  const void* q; const void* f; long long ld;     // projected rows [T, H d] each
+  const float* bias; const float* lower;          // [H d]
+  float* rec;
   SxRagged ragged;
-  int H, Hq, d, dv, delta, f32;
+  SxChunks chunks;
+  int H, d, f32;
+} SxGateArgs;
+int sx_recur_record(int d, int delta);
+int sx_gate_chunks(const SxGateArgs* args, cudaStream_t stream);
+int sx_delta_chunks(const SxDeltaArgs* args, const SxChunks* chunks, float* rec, cudaStream_t stream);
+typedef struct SxScanArgs {
+  const float* rec;
+  const void* v; long long v_ld;
+  float* state; float* o;         // [slots, H, d, dv], [T, H, dv]
+  SxRagged ragged;
+  SxChunks chunks;
+  int* status;
+  int H, d, dv, delta, f32;
 } SxScanArgs;
 int sx_recur_scan(const SxScanArgs* args, cudaStream_t stream);
 // One token per sequence, from the projected rows to the normed and gated output row.
@@ -314,6 +333,26 @@ typedef struct SxTalkArgs {
   float* part; int splits;        // decode: partial results of key splits [n, splits, H, dv + 2]
 } SxTalkArgs;
 int sx_talk_attn(const SxTalkArgs* args, cudaStream_t stream);
+int sx_talk_merge(const SxTalkArgs* args, cudaStream_t stream);
+// Tensor-core decode form over the block pool (bf16): queries with the head mix folded in, [n, H, q_ld].
+int sx_talk_decode_ok(int H, int G, int d, int dv);
+int sx_talk_decode(const SxTalkArgs* args, const void* qmix, int q_ld, cudaStream_t stream);
+// Tensor-core prompt form (bf16, value heads up to 128): queries with the head mix folded in, [T, H, nq * 64] with
+// nq = ceil(G d / 64) and zeros past G d; packed keys [kv_rows, k_ld] and values (head j at column j * dvp).
+typedef struct SxTalkTcArgs {
+  const void* qmix; const void* k; const void* v;
+  long long k_ld, v_ld, kv_rows;
+  const int* kv_base;
+  const int* tiles;               // [n_tiles, 2]: portion, first of up to 128 rows of it
+  const void* gate; long long gate_ld;
+  void* y; long long y_ld;
+  SxRagged ragged;
+  float scale, mul;
+  int T, n_tiles, H, G, d, dv, dvp, size;
+  int* status;
+} SxTalkTcArgs;
+int sx_talk_attn_tc_ok(int H, int G, int d, int dv);
+int sx_talk_attn_tc(const SxTalkTcArgs* args, cudaStream_t stream);
 
 #ifdef __cplusplus
 }

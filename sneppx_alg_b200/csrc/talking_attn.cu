@@ -161,6 +161,16 @@ static int launch_talk(const TalkParams& P, cudaStream_t st) {
   return last_rc();
 }
 
+// Merges the partial results of a->splits key slices per query into y.
+extern "C" int sx_talk_merge(const SxTalkArgs* a, cudaStream_t st) {
+  if (a->T <= 0) return 0;
+  TalkParams P;
+  P.a = *a;
+  P.rv = view(&a->ragged);
+  SX_ACT_DISPATCH(a->f32, (talk_merge_kernel<A><<<dim3(a->H, a->T), 128, 0, st>>>(P)));
+  return last_rc();
+}
+
 extern "C" int sx_talk_attn(const SxTalkArgs* a, cudaStream_t st) {
   if (a->T <= 0) return 0;
   if (a->G <= 0 || a->H % a->G || a->d % 2 || a->size <= 0 || a->splits < 1) return -1;

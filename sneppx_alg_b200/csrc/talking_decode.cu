@@ -1,0 +1,281 @@
+// Decode attention with a head mix in front of the softmax over the block pool (bf16): one query per sequence, keys limited
+// to the query's chunk of positions.
+//
+// The mix is folded into the queries (sx_qkv_prep writes q'), so the scores of all heads are one product of q' [H, G d] with
+// the cache rows as they lie in memory [keys, G d]. One CTA serves a slice of the visible keys of one sequence for all heads:
+// cache rows stream through shared memory with cp.async, scores and P V run on tensor cores (mma.sync: the work is bound by
+// reading the cache, the products are a few percent of it), and a second kernel merges the slices (talking_attn.cu).
+#include "common.cuh"
+#include "ragged.cuh"
+#include "tc_common.cuh"
+#include "sx_api.h"
+
+namespace sx {
+
+struct TalkDecParams {
+  const __nv_bfloat16* qmix;  // [n, H, q_ld]
+  const __nv_bfloat16* k; const __nv_bfloat16* v;   // cache rows [entries, G d], [entries, G dv]
+  const int* block_table; const int* block_base;
+  const __nv_bfloat16* gate;
+  __nv_bfloat16* y;
+  float* part;
+  RaggedView rv;
+  long long gate_ld, y_ld;
+  int q_ld, table_ld, block_size, H, G, d, dv, size, splits, stages, ksplit;
+  float scale, mul;
+};
+
+__device__ __forceinline__ void dec_cp16(void* dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm2(uint32_t (&r)[2], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void ldsm2t(uint32_t (&r)[2], const void* p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)) : "memory");
+}
+__device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
+}
+
+struct DecLayout {
+  int HP, D16, ldq, ldk, ldv, ldp, lds, stage;   // elements (stage: bf16 elements of one K + V tile)
+  int off_k, off_s, off_p, off_m, bytes;         // bytes
+};
+__host__ __device__ inline DecLayout dec_layout(int H, int G, int d, int dv, int KT, int stages, int ksplit) {
+  DecLayout L;
+  L.HP = (H + 15) / 16 * 16;
+  L.D16 = (G * d + 15) / 16 * 16;
+  L.ldq = L.D16 + 8;
+  L.ldk = L.D16 + 8;
+  L.ldv = G * dv + 8;
+  L.ldp = KT + 8;
+  L.lds = KT + 2;
+  L.stage = KT * (L.ldk + L.ldv);
+  L.off_k = L.HP * L.ldq * 2;
+  L.off_s = L.off_k + stages * L.stage * 2;
+  L.off_p = L.off_s + ksplit * L.HP * L.lds * 4;
+  L.off_m = L.off_p + (L.HP + 16) * L.ldp * 2;
+  L.bytes = L.off_m + 3 * L.HP * 4;
+  return L;
+}
+
+template <int KT, int MAXI>
+__global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p) {
+  extern __shared__ __align__(16) uint8_t smem[];
+  const DecLayout L = dec_layout(p.H, p.G, p.d, p.dv, KT, p.stages, p.ksplit);
+  __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);
+  __nv_bfloat16* sKV = reinterpret_cast<__nv_bfloat16*>(smem + L.off_k);
+  float* sS = reinterpret_cast<float*>(smem + L.off_s);
+  __nv_bfloat16* sP = reinterpret_cast<__nv_bfloat16*>(smem + L.off_p);
+  float* sM = reinterpret_cast<float*>(smem + L.off_m);
+  float* sL = sM + L.HP;
+  float* sC = sL + L.HP;
+  const int n = blockIdx.x, split = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  if (p.rv.slot[n] < 0) return;            // padding row of a captured launch
+  const int t = p.rv.cu[n], pos = p.rv.pos0[n];
+  const int H = p.H, G = p.G, Gd = G * p.d, Gv = G * p.dv, grp = H / G;
+  const int first = pos / p.size * p.size, n_vis = pos - first + 1;
+  const int per = (n_vis + p.splits - 1) / p.splits;
+  const int lo = first + split * per, hi = min(pos + 1, lo + per);
+  const int n_tiles = hi > lo ? (hi - lo + KT - 1) / KT : 0;
+
+  const int base = p.block_base[n];
+  const int* table = p.block_table + (long long)n * p.table_ld;
+  auto fetch = [&](int tile) {
+    if (tile < n_tiles) {
+      __nv_bfloat16* sk = sKV + (tile % p.stages) * L.stage;
+      __nv_bfloat16* sv = sk + KT * L.ldk;
+      const int j0 = lo + tile * KT;
+      for (int r = warp; r < KT; r += 8) {
+        const int j = min(j0 + r, hi - 1);          // rows past the end repeat the last key and are masked
+        const long long e = (long long)table[j / p.block_size - base] * p.block_size + j % p.block_size;
+        const __nv_bfloat16* kr = p.k + e * Gd;
+        const __nv_bfloat16* vr = p.v + e * Gv;
+        for (int c = lane; c < Gd / 8; c += 32) dec_cp16(sk + r * L.ldk + c * 8, kr + c * 8);
+        for (int c = lane; c < Gv / 8; c += 32) dec_cp16(sv + r * L.ldv + c * 8, vr + c * 8);
+      }
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+  for (int s = 0; s < p.stages - 1; ++s) fetch(s);
+  // queries, zero padding
+  const __nv_bfloat16* q = p.qmix + (long long)t * H * p.q_ld;
+  for (int i = tid; i < L.HP * (L.D16 / 8); i += 256) {
+    const int h = i / (L.D16 / 8), c = i % (L.D16 / 8) * 8;
+    uint4 x = make_uint4(0, 0, 0, 0);
+    if (h < H) x = *reinterpret_cast<const uint4*>(q + (long long)h * p.q_ld + c);
+    *reinterpret_cast<uint4*>(sQ + h * L.ldq + c) = x;
+  }
+  if (Gd < L.D16)
+    for (int i = tid; i < p.stages * KT * (L.D16 - Gd); i += 256) {
+      const int w = L.D16 - Gd, s = i / (KT * w), r = i / w % KT;
+      sKV[s * L.stage + r * L.ldk + Gd + i % w] = __float2bfloat16_rn(0.f);
+    }
+  for (int i = tid; i < (L.HP + 16) * L.ldp; i += 256) sP[i] = __float2bfloat16_rn(0.f);
+  for (int i = tid; i < L.HP; i += 256) {
+    sM[i] = -INFINITY;
+    sL[i] = 0.f;
+    sC[i] = 1.f;
+  }
+  float O[MAXI][4];
+#pragma unroll
+  for (int i = 0; i < MAXI; ++i) O[i][0] = O[i][1] = O[i][2] = O[i][3] = 0.f;
+  const int nt8 = p.dv / 8, items = G * nt8, units = (KT / 8) * (L.HP / 16), ksteps = L.D16 / 16;
+
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    if (p.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    else asm volatile("cp.async.wait_group 1;" ::: "memory");
+    __syncthreads();
+    fetch(tile + p.stages - 1);
+    const __nv_bfloat16* sk = sKV + (tile % p.stages) * L.stage;
+    const __nv_bfloat16* sv = sk + KT * L.ldk;
+    for (int it = warp; it < units * p.ksplit; it += 8) {
+      const int unit = it % units, ks = it / units, n0 = (unit % (KT / 8)) * 8, m0 = unit / (KT / 8) * 16;
+      const int k0 = ksteps * ks / p.ksplit, k1 = ksteps * (ks + 1) / p.ksplit;
+      const __nv_bfloat16* qa = sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8;
+      const __nv_bfloat16* kb = sk + (n0 + (lane & 7)) * L.ldk + ((lane >> 3) & 1) * 8;
+      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
+      int kk = k0;
+      for (; kk + 1 < k1; kk += 2) {
+        uint32_t a[4], b[2], a2[4], b2[2];
+        ldsm4(a, qa + kk * 16);
+        ldsm2(b, kb + kk * 16);
+        ldsm4(a2, qa + kk * 16 + 16);
+        ldsm2(b2, kb + kk * 16 + 16);
+        mma16816(c0, a, b);
+        mma16816(c1, a2, b2);
+      }
+      if (kk < k1) {
+        uint32_t a[4], b[2];
+        ldsm4(a, qa + kk * 16);
+        ldsm2(b, kb + kk * 16);
+        mma16816(c0, a, b);
+      }
+      float* s = sS + (ks * L.HP + m0 + (lane >> 2)) * L.lds + n0 + (lane & 3) * 2;
+      *reinterpret_cast<float2*>(s) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+      *reinterpret_cast<float2*>(s + 8 * L.lds) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+    }
+    __syncthreads();
+    const int nk = min(KT, hi - lo - tile * KT);
+    for (int h = warp; h < H; h += 8) {
+      float s = -INFINITY;
+      if (lane < nk) {
+        s = 0.f;
+        for (int ks = 0; ks < p.ksplit; ++ks) s += sS[(ks * L.HP + h) * L.lds + lane];
+        s *= p.scale;
+      }
+      const float m_old = sM[h], m = fmaxf(m_old, warp_max(s));
+      const __nv_bfloat16 e = __float2bfloat16_rn(exp2f((s - m) * 1.4426950408889634f));
+      const float l = warp_sum(__bfloat162float(e));
+      if (lane < KT) sP[h * L.ldp + lane] = e;
+      if (lane == 0) {
+        const float c = exp2f((m_old - m) * 1.4426950408889634f);
+        sC[h] = c;
+        sM[h] = m;
+        sL[h] = sL[h] * c + l;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < MAXI; ++i) {
+      const int it = warp + i * 8;
+      if (it >= items) break;
+      const int j = it / nt8, c = j * p.dv + (it % nt8) * 8, r = lane >> 2;
+      const float f0 = r < grp ? sC[j * grp + r] : 0.f, f1 = r + 8 < grp ? sC[j * grp + r + 8] : 0.f;
+      O[i][0] *= f0; O[i][1] *= f0; O[i][2] *= f1; O[i][3] *= f1;
+#pragma unroll
+      for (int kk = 0; kk < KT / 16; ++kk) {
+        uint32_t a[4], b[2];
+        ldsm4(a, sP + (j * grp + (lane & 15)) * L.ldp + kk * 16 + (lane >> 4) * 8);
+        ldsm2t(b, sv + (kk * 16 + (lane & 15)) * L.ldv + c);
+        mma16816(O[i], a, b);
+      }
+    }
+  }
+  __syncthreads();
+#pragma unroll
+  for (int i = 0; i < MAXI; ++i) {
+    const int it = warp + i * 8;
+    if (it >= items) break;
+    const int j = it / nt8, c = (it % nt8) * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int half = 0; half < 2; ++half) {
+      const int r = (lane >> 2) + half * 8;
+      if (r >= grp) continue;
+      const int h = j * grp + r;
+      const float a = O[i][2 * half], b = O[i][2 * half + 1];
+      if (p.splits > 1) {
+        float* o = p.part + (((long long)n * p.splits + split) * H + h) * (p.dv + 2) + 2 + c;
+        o[0] = a;
+        o[1] = b;
+      } else {
+        const float g = p.mul / ((1.f + __expf(-__bfloat162float(p.gate[(long long)t * p.gate_ld + h]))) * sL[h]);
+        store2(p.y + (long long)t * p.y_ld + (long long)h * p.dv + c, a * g, b * g);
+      }
+    }
+  }
+  if (p.splits > 1)
+    for (int h = tid; h < H; h += 256) {
+      float* o = p.part + (((long long)n * p.splits + split) * H + h) * (p.dv + 2);
+      o[0] = sM[h];
+      o[1] = sL[h];
+    }
+}
+
+struct DecPlan { int kt, stages, ksplit, maxi; };
+static DecPlan dec_plan(int H, int G, int d, int dv) {
+  DecPlan pl{0, 0, 0, 0};
+  if (H <= 0 || G <= 0 || H % G || H / G > 16 || (G * d) % 8 || (d % 2) || dv % 8) return pl;
+  const int per_warp = (G * (dv / 8) + 7) / 8;
+  if (per_warp > 32) return pl;
+  for (int kt = 32; kt >= 16; kt -= 16)
+    for (int stages = 3; stages >= 2; --stages) {
+      const int units = (kt / 8) * ((H + 15) / 16), ks = units >= 8 ? 1 : (units >= 4 ? 2 : 4);
+      if (dec_layout(H, G, d, dv, kt, stages, ks).bytes <= 227 * 1024) return DecPlan{kt, stages, ks, per_warp <= 8 ? 8 : per_warp <= 16 ? 16 : 32};
+    }
+  return pl;
+}
+
+}  // namespace sx
+using namespace sx;
+
+// 1 when sx_talk_decode takes these sizes.
+extern "C" int sx_talk_decode_ok(int H, int G, int d, int dv) { return dec_plan(H, G, d, dv).kt > 0; }
+
+template <int KT, int MAXI>
+static int launch_dec(const TalkDecParams& p, int n, int smem, cudaStream_t st) {
+  static bool set = false;
+  if (!set) {
+    if (cudaFuncSetAttribute(talk_decode_kernel<KT, MAXI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -10;
+    set = true;
+  }
+  talk_decode_kernel<KT, MAXI><<<dim3(n, p.splits), 256, smem, st>>>(p);
+  return last_rc();
+}
+
+// Paged form only; `qmix` [n, H, q_ld] (zeros from G d up to the next multiple of 64). With splits > 1 the partial results go
+// to a->part and the caller merges them (sx_talk_merge).
+extern "C" int sx_talk_decode(const SxTalkArgs* a, const void* qmix, int q_ld, cudaStream_t st) {
+  if (a->T <= 0) return 0;
+  const DecPlan pl = dec_plan(a->H, a->G, a->d, a->dv);
+  if (!pl.kt || !a->block_table || a->f32 || a->splits < 1) return -1;
+  TalkDecParams p;
+  p.qmix = (const __nv_bfloat16*)qmix; p.q_ld = q_ld; p.k = (const __nv_bfloat16*)a->k; p.v = (const __nv_bfloat16*)a->v;
+  p.block_table = a->block_table; p.block_base = a->block_base; p.table_ld = a->table_ld; p.block_size = a->block_size;
+  p.gate = (const __nv_bfloat16*)a->gate; p.gate_ld = a->gate_ld; p.y = (__nv_bfloat16*)a->y; p.y_ld = a->y_ld; p.part = a->part;
+  p.rv = view(&a->ragged);
+  p.H = a->H; p.G = a->G; p.d = a->d; p.dv = a->dv; p.size = a->size; p.splits = a->splits; p.stages = pl.stages; p.ksplit = pl.ksplit;
+  p.scale = a->scale; p.mul = a->mul;
+  const int smem = dec_layout(a->H, a->G, a->d, a->dv, pl.kt, pl.stages, pl.ksplit).bytes;
+  int rc;
+  if (pl.kt == 32) rc = pl.maxi == 8 ? launch_dec<32, 8>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<32, 16>(p, a->T, smem, st) : launch_dec<32, 32>(p, a->T, smem, st);
+  else rc = pl.maxi == 8 ? launch_dec<16, 8>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<16, 16>(p, a->T, smem, st) : launch_dec<16, 32>(p, a->T, smem, st);
+  if (rc == 0 && a->splits > 1) rc = sx_talk_merge(a, st);
+  return rc;
+}

@@ -81,8 +81,8 @@ class GatedWriteBranch(Branch):
             hybrid.gated_write_step(u["q"], u["f"], u["v"], self.f_bias, self.lower, state["S"], self.norm, y, batch, H, d, dv,
                                     self.eps, mul=scale)
             return
-        q, f = hybrid.gate_prep(u["q"], u["f"], self.f_bias, self.lower)
-        o = hybrid.recur_scan(q, f, u["v"], state["S"], batch, H, d, dv)
+        rec = hybrid.gate_chunks(u["q"], u["f"], self.f_bias, self.lower, batch, H, d)
+        o = hybrid.recur_scan(rec, u["v"], state["S"], batch, H, d, dv, delta=False)
         hybrid.head_norm_gate(o, self.norm, y, self.eps, mul=scale)
 
 
@@ -131,10 +131,9 @@ class DeltaBranch(Branch):
             hybrid.delta_step(qkv, self.conv, state["ring"], u["b"], a, self.a_log, self.dt_bias, state["S"], self.norm, y, batch,
                               H, G, d, dv, self.taps, self.eps, gate=gate, mul=scale)
             return
-        q, k, g, v, beta = hybrid.delta_prep(qkv, self.conv, state["ring"], u["b"], a, self.a_log, self.dt_bias, batch, H, G, d, dv,
-                                             self.taps)
+        rec, v = hybrid.delta_chunks(qkv, self.conv, state["ring"], u["b"], a, self.a_log, self.dt_bias, batch, H, G, d, dv, self.taps)
         hybrid.conv_ring(qkv, state["ring"], batch, self.channels, self.taps)
-        o = hybrid.recur_scan(q, g, v, state["S"], batch, H, d, dv, k=k, beta=beta)
+        o = hybrid.recur_scan(rec, v, state["S"], batch, H, d, dv, delta=True)
         hybrid.head_norm_gate(o, self.norm, y, self.eps, gate=gate, mul=scale)
 
 
@@ -183,9 +182,13 @@ class TalkingAttentionBranch(Branch):
         common = (qkv, self.conv, state["ring"], self.q_norm, self.k_norm, self.inv_freq(dev), batch, k_cache, v_cache, H, G, d, dv,
                   self.taps, self.eps)
         if batch.decode:
-            q = torch.empty(batch.T, H, d, dtype=torch.float32, device=dev)
-            hybrid.qkv_prep(*common, q_out=q)
-            hybrid.talking_decode(q, k_cache, v_cache, self.talk, gate, y, batch, self.scale, scale, H, G, d, dv, self.chunk)
+            q = qmix = None
+            if hybrid.talking_decode_tc(act, H, G, d, dv):
+                qmix = torch.empty(batch.T, H, _up(G * d, 64), dtype=act, device=dev)
+            else:
+                q = torch.empty(batch.T, H, d, dtype=torch.float32, device=dev)
+            hybrid.qkv_prep(*common, q_out=q, qmix_out=qmix, talk=self.talk)
+            hybrid.talking_decode(q, k_cache, v_cache, self.talk, gate, y, batch, self.scale, scale, H, G, d, dv, self.chunk, qmix=qmix)
             return
         view = batch.views[self.chunk]
         dvp = _up(dv)
@@ -194,6 +197,12 @@ class TalkingAttentionBranch(Branch):
         # before the append: the append may reuse blocks that earlier positions still occupy
         hybrid.kv_gather(k_cache, view.gather_entry, view.gather_row, k, G, d, d)
         hybrid.kv_gather(v_cache, view.gather_entry, view.gather_row, v, G, dv, dvp)
+        if hybrid.talking_tc(act, H, G, d, dv):
+            qmix = torch.empty(batch.T, H, _up(G * d, 64), dtype=act, device=dev)
+            hybrid.qkv_prep(*common, qmix_out=qmix, talk=self.talk, k_out=k, v_out=v, dvp=dvp, kv_row=view.kv_row)
+            hybrid.conv_ring(qkv, state["ring"], batch, self.channels, self.taps)
+            hybrid.talking_attention_tc(qmix, k, v, gate, y, batch, view, self.scale, scale, H, G, d, dv, dvp, self.chunk)
+            return
         q = torch.empty(batch.T, H, d, dtype=torch.float32, device=dev)
         hybrid.qkv_prep(*common, q_out=q, k_out=k, v_out=v, dvp=dvp, kv_row=view.kv_row)
         hybrid.conv_ring(qkv, state["ring"], batch, self.channels, self.taps)

@@ -51,32 +51,41 @@ class SxRagged(C.Structure):
                 ("n", c_int)]
 
 
+class SxChunks(C.Structure):
+    _fields_ = [("seq", c_void_p), ("start", c_void_p), ("first", c_void_p), ("n", c_int)]
+
+
 class SxQkvArgs(C.Structure):
     _fields_ = [
         ("u", c_void_p), ("u_ld", c_ll), ("wconv", c_void_p), ("ring", c_void_p), ("qn", c_void_p), ("kn", c_void_p),
-        ("inv_freq", c_void_p), ("talk", c_void_p), ("q_out", c_void_p), ("qmix_out", c_void_p), ("k_out", c_void_p),
+        ("inv_freq", c_void_p), ("talk", c_void_p), ("q_out", c_void_p), ("qmix_out", c_void_p),
+        ("qmix_ld", c_int), ("k_out", c_void_p),
         ("v_out", c_void_p), ("k_ld", c_ll), ("v_ld", c_ll), ("kv_row", c_void_p), ("k_cache", c_void_p),
         ("v_cache", c_void_p), ("cache_entry", c_void_p), ("ragged", SxRagged),
-        ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("dvp", c_int), ("taps", c_int),
-        ("rot", c_int), ("write_ring", c_int), ("f32", c_int), ("eps", c_float),
+        ("chunks", SxChunks), ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("dvp", c_int),
+        ("taps", c_int), ("rot", c_int), ("f32", c_int), ("eps", c_float),
     ]
 
 
 class SxDeltaArgs(C.Structure):
     _fields_ = [
         ("u", c_void_p), ("u_ld", c_ll), ("wconv", c_void_p), ("ring", c_void_p), ("b", c_void_p), ("b_ld", c_ll),
-        ("a", c_void_p), ("a_ld", c_ll), ("a_log", c_void_p), ("dt_bias", c_void_p), ("q", c_void_p), ("k", c_void_p),
-        ("g", c_void_p), ("v", c_void_p), ("beta", c_void_p), ("ragged", SxRagged),
-        ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("taps", c_int), ("write_ring", c_int),
-        ("f32", c_int),
+        ("a", c_void_p), ("a_ld", c_ll), ("a_log", c_void_p), ("dt_bias", c_void_p), ("v", c_void_p), ("ragged", SxRagged),
+        ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("taps", c_int), ("f32", c_int),
+    ]
+
+
+class SxGateArgs(C.Structure):
+    _fields_ = [
+        ("q", c_void_p), ("f", c_void_p), ("ld", c_ll), ("bias", c_void_p), ("lower", c_void_p), ("rec", c_void_p),
+        ("ragged", SxRagged), ("chunks", SxChunks), ("H", c_int), ("d", c_int), ("f32", c_int),
     ]
 
 
 class SxScanArgs(C.Structure):
     _fields_ = [
-        ("q", c_void_p), ("g", c_void_p), ("k", c_void_p), ("v", c_void_p), ("v_ld", c_ll), ("beta", c_void_p),
-        ("state", c_void_p), ("o", c_void_p), ("ragged", SxRagged),
-        ("H", c_int), ("Hq", c_int), ("d", c_int), ("dv", c_int), ("delta", c_int), ("f32", c_int),
+        ("rec", c_void_p), ("v", c_void_p), ("v_ld", c_ll), ("state", c_void_p), ("o", c_void_p), ("ragged", SxRagged),
+        ("chunks", SxChunks), ("status", c_void_p), ("H", c_int), ("d", c_int), ("dv", c_int), ("delta", c_int), ("f32", c_int),
     ]
 
 
@@ -97,6 +106,16 @@ class SxTalkArgs(C.Structure):
         ("ragged", SxRagged), ("scale", c_float), ("mul", c_float),
         ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("size", c_int), ("f32", c_int),
         ("part", c_void_p), ("splits", c_int),
+    ]
+
+
+class SxTalkTcArgs(C.Structure):
+    _fields_ = [
+        ("qmix", c_void_p), ("k", c_void_p), ("v", c_void_p), ("k_ld", c_ll), ("v_ld", c_ll), ("kv_rows", c_ll),
+        ("kv_base", c_void_p), ("tiles", c_void_p), ("gate", c_void_p), ("gate_ld", c_ll), ("y", c_void_p), ("y_ld", c_ll),
+        ("ragged", SxRagged), ("scale", c_float), ("mul", c_float),
+        ("T", c_int), ("n_tiles", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int), ("dvp", c_int),
+        ("size", c_int), ("status", c_void_p),
     ]
 
 

@@ -58,15 +58,21 @@ def conv_ring(u, ring, batch: RaggedBatch, channels, taps):
 
 
 # ----------------------------------------------------------------------------- recurrences
-def gate_prep(qr, fr, bias, lower):
-    """silu(q) and the lower-bounded forget gate of a gated-write recurrence, both fp32 [T, H * d]."""
-    T, c = qr.shape
-    q = torch.empty(T, c, dtype=torch.float32, device=qr.device)
-    f = torch.empty_like(q)
+def _records(batch, H, d, delta, device):
+    n = _lib.lib().sx_recur_record(c_int(d), c_int(int(delta)))
+    return torch.empty(batch.n_chunks * H * n, dtype=torch.float32, device=device)
+
+
+def gate_chunks(qr, fr, bias, lower, batch: RaggedBatch, H, d):
+    """State-independent operands of a gated-write recurrence (q = silu, lower-bounded forget gate) for ``recur_scan``."""
+    _need_cuda(qr)
     assert qr.stride(0) == fr.stride(0)
-    _lib.call("sx_gate_prep", ptr(qr), ptr(fr), c_ll(qr.stride(0)), ptr(bias), ptr(lower), ptr(q), ptr(f), c_int(T), c_int(c),
-              c_int(_f32(qr)), stream())
-    return q, f
+    rec = _records(batch, H, d, False, qr.device)
+    a = _lib.SxGateArgs()
+    a.q, a.f, a.ld, a.bias, a.lower, a.rec = qr.data_ptr(), fr.data_ptr(), qr.stride(0), bias.data_ptr(), lower.data_ptr(), rec.data_ptr()
+    a.ragged, a.chunks, a.H, a.d, a.f32 = batch.struct(), batch.chunks(), H, d, _f32(qr)
+    _lib.call("sx_gate_chunks", C.byref(a), stream())
+    return rec
 
 
 def _delta_args(u, wconv, ring, b, a, a_log, dt_bias, batch, H, G, d, dv, taps):
@@ -79,31 +85,26 @@ def _delta_args(u, wconv, ring, b, a, a_log, dt_bias, batch, H, G, d, dv, taps):
     return x
 
 
-def delta_prep(u, wconv, ring, b, a, a_log, dt_bias, batch: RaggedBatch, H, G, d, dv, taps):
-    """Operands of the gated delta rule from projected rows: q, k [T, G, d], decay [T, H, d], v [T, H * dv], beta [T, H]."""
+def delta_chunks(u, wconv, ring, b, a, a_log, dt_bias, batch: RaggedBatch, H, G, d, dv, taps):
+    """State-independent operands of the gated delta rule for ``recur_scan``, and the convolved values [T, H * dv]."""
     _need_cuda(u)
-    T, dev = batch.T, u.device
-    q, k = (torch.empty(T, G, d, dtype=torch.float32, device=dev) for _ in range(2))
-    g = torch.empty(T, H, d, dtype=torch.float32, device=dev)
-    v = torch.empty(T, H * dv, dtype=u.dtype, device=dev)
-    beta = torch.empty(T, H, dtype=torch.float32, device=dev)
+    rec = _records(batch, H, d, True, u.device)
+    v = torch.empty(batch.T, H * dv, dtype=u.dtype, device=u.device)
     x = _delta_args(u, wconv, ring, b, a, a_log, dt_bias, batch, H, G, d, dv, taps)
-    x.q, x.k, x.g, x.v, x.beta = q.data_ptr(), k.data_ptr(), g.data_ptr(), v.data_ptr(), beta.data_ptr()
-    _lib.call("sx_delta_prep", C.byref(x), stream())
-    return q, k, g, v, beta
+    x.v = v.data_ptr()
+    ch = batch.chunks()
+    _lib.call("sx_delta_chunks", C.byref(x), C.byref(ch), ptr(rec), stream())
+    return rec, v
 
 
-def recur_scan(q, g, v, state, batch: RaggedBatch, H, d, dv, k=None, beta=None):
+def recur_scan(rec, v, state, batch: RaggedBatch, H, d, dv, delta):
     """Walks every portion of the batch from its slot's state (empty at position 0), stores the state back and returns the
-    read-outs [T, H, dv] fp32. With ``k`` and ``beta``: the gated delta rule; without: the gated write with key 1 - g."""
-    _need_cuda(q)
-    o = torch.empty(batch.T, H, dv, dtype=torch.float32, device=q.device)
+    read-outs [T, H, dv] fp32."""
+    o = torch.empty(batch.T, H, dv, dtype=torch.float32, device=v.device)
     x = _lib.SxScanArgs()
-    x.q, x.g, x.v, x.v_ld = q.data_ptr(), g.data_ptr(), v.data_ptr(), v.stride(0)
-    x.k = k.data_ptr() if k is not None else None
-    x.beta = beta.data_ptr() if beta is not None else None
-    x.state, x.o, x.ragged = state.data_ptr(), o.data_ptr(), batch.struct()
-    x.H, x.Hq, x.d, x.dv, x.delta, x.f32 = H, q.numel() // (batch.T * d), d, dv, int(k is not None), _f32(v)
+    x.rec, x.v, x.v_ld, x.state, x.o = rec.data_ptr(), v.data_ptr(), v.stride(0), state.data_ptr(), o.data_ptr()
+    x.ragged, x.chunks, x.status = batch.struct(), batch.chunks(), _lib.status_word(v.device).data_ptr()
+    x.H, x.d, x.dv, x.delta, x.f32 = H, d, dv, int(delta), _f32(v)
     _lib.call("sx_recur_scan", C.byref(x), stream())
     return o
 
@@ -148,12 +149,16 @@ def qkv_prep(u, wconv, ring, qn, kn, inv_freq, batch: RaggedBatch, k_cache, v_ca
     for name, t in (("talk", talk), ("q_out", q_out), ("qmix_out", qmix_out), ("k_out", k_out), ("v_out", v_out), ("kv_row", kv_row)):
         if t is not None:
             setattr(x, name, t.data_ptr())
+    if qmix_out is not None:
+        x.qmix_ld = qmix_out.shape[-1]
     if k_out is not None:
         x.k_ld, x.v_ld = k_out.stride(0), v_out.stride(0)
     x.k_cache, x.v_cache, x.cache_entry = k_cache.data_ptr(), v_cache.data_ptr(), batch.entry.data_ptr()
     x.ragged = batch.struct()
     x.T, x.H, x.G, x.d, x.dv, x.dvp, x.taps = batch.T, H, G, d, dv, dvp or dv, taps
-    x.rot, x.write_ring, x.f32, x.eps = 2 * inv_freq.numel(), int(batch.decode), _f32(u), eps
+    x.rot, x.f32, x.eps = 2 * inv_freq.numel(), _f32(u), eps
+    if not batch.decode:
+        x.chunks = batch.chunks()
     _lib.call("sx_qkv_prep", C.byref(x), stream())
 
 
@@ -182,18 +187,46 @@ def talking_attention(q, k, v, talk, gate, y, batch: RaggedBatch, kv_base, scale
     _lib.call("sx_talk_attn", C.byref(a), stream())
 
 
+def talking_tc(act_dtype, H, G, d, dv) -> bool:
+    """Whether the tensor-core prompt kernel takes these sizes."""
+    return act_dtype == torch.bfloat16 and bool(_lib.lib().sx_talk_attn_tc_ok(c_int(H), c_int(G), c_int(d), c_int(dv)))
+
+
+def talking_attention_tc(qmix, k, v, gate, y, batch: RaggedBatch, view, scale, mul, H, G, d, dv, dvp, size):
+    """Tensor-core prompt form: ``qmix`` [T, H, ceil(G d / 64) * 64] from ``qkv_prep``."""
+    a = _lib.SxTalkTcArgs()
+    a.qmix, a.k, a.v = qmix.data_ptr(), k.data_ptr(), v.data_ptr()
+    a.k_ld, a.v_ld, a.kv_rows = k.stride(0), v.stride(0), k.shape[0]
+    a.kv_base, a.tiles, a.n_tiles = view.kv_base.data_ptr(), view.tiles.data_ptr(), view.n_tiles
+    a.gate, a.gate_ld, a.y, a.y_ld = gate.data_ptr(), gate.stride(0), y.data_ptr(), y.stride(0)
+    a.ragged = batch.struct()
+    a.scale, a.mul = scale, mul
+    a.T, a.H, a.G, a.d, a.dv, a.dvp, a.size = batch.T, H, G, d, dv, dvp, size
+    a.status = _lib.status_word(y.device).data_ptr()
+    _lib.call("sx_talk_attn_tc", C.byref(a), stream())
+
+
 def decode_splits(n: int, size: int) -> int:
-    """Key splits of one decode step: enough CTAs for the machine, at least 64 keys each."""
-    return max(1, min((size + 63) // 64, 296 // max(n, 1)))
+    """Key slices of one decode step: one CTA per SM, at least 64 keys each."""
+    return max(1, min((size + 63) // 64, 148 // max(n, 1)))
 
 
-def talking_decode(q, k_cache, v_cache, talk, gate, y, batch: RaggedBatch, scale, mul, H, G, d, dv, size):
-    """Decode form: one query per sequence against the block pool."""
-    a = _talk_args(q, k_cache, v_cache, G * d, G * dv, talk, gate, y, batch, scale, mul, H, G, d, dv, dv, size)
+def talking_decode_tc(act_dtype, H, G, d, dv) -> bool:
+    """Whether the tensor-core decode kernel takes these sizes."""
+    return act_dtype == torch.bfloat16 and bool(_lib.lib().sx_talk_decode_ok(c_int(H), c_int(G), c_int(d), c_int(dv)))
+
+
+def talking_decode(q, k_cache, v_cache, talk, gate, y, batch: RaggedBatch, scale, mul, H, G, d, dv, size, qmix=None):
+    """Decode form: one query per sequence against the block pool. Either ``q`` (fp32 [T, H, d], any sizes) or ``qmix``
+    (bf16 [T, H, q_ld] from ``qkv_prep``, the tensor-core kernel)."""
+    a = _talk_args(q if q is not None else qmix, k_cache, v_cache, G * d, G * dv, talk, gate, y, batch, scale, mul, H, G, d, dv, dv, size)
     a.block_table, a.block_base = batch.block_table.data_ptr(), batch.block_base.data_ptr()
     a.table_ld, a.block_size = batch.table_width, k_cache.shape[1]
     a.splits = decode_splits(batch.n, size)
     if a.splits > 1:
-        part = torch.empty(batch.n * a.splits * H * (dv + 2), dtype=torch.float32, device=q.device)
+        part = torch.empty(batch.n * a.splits * H * (dv + 2), dtype=torch.float32, device=y.device)
         a.part = part.data_ptr()
-    _lib.call("sx_talk_attn", C.byref(a), stream())
+    if qmix is not None:
+        _lib.call("sx_talk_decode", C.byref(a), ptr(qmix), c_int(qmix.shape[-1]), stream())
+    else:
+        _lib.call("sx_talk_attn", C.byref(a), stream())

@@ -11,6 +11,9 @@ import torch
 from . import _lib
 
 
+RECUR_CHUNK = 16     # tokens per chunk of the recurrence kernels
+
+
 @dataclass
 class ChunkView:
     """Packed keys and values of one chunk length: rows of the portion, preceded by the rows of earlier positions that
@@ -40,6 +43,11 @@ class RaggedBatch:
         r.tok_seq, r.tok_pos, r.n = self.tok_seq.data_ptr(), self.tok_pos.data_ptr(), self.n
         return r
 
+    def chunks(self) -> "_lib.SxChunks":
+        c = _lib.SxChunks()
+        c.seq, c.start, c.first, c.n = self.chunk_seq.data_ptr(), self.chunk_start.data_ptr(), self.chunk_first.data_ptr(), self.n_chunks
+        return c
+
     @classmethod
     def prompt(cls, device, tokens: List[List[int]], pos0: List[int], slots: List[int], entries: List[List[int]],
                earlier: Dict[int, List[List[int]]], want: List[int], tile_rows: int = 128) -> "RaggedBatch":
@@ -58,21 +66,27 @@ class RaggedBatch:
                  np.asarray(want, dtype=np.int32)]
         tiles = np.array([(i, r) for i in range(b.n) for r in range(0, int(lens[i]), tile_rows)], dtype=np.int32)
         parts.append(tiles.reshape(-1))
+        per = (lens + RECUR_CHUNK - 1) // RECUR_CHUNK
+        first = np.zeros(b.n + 1, dtype=np.int32)
+        np.cumsum(per, out=first[1:])
+        chunk_seq = np.repeat(np.arange(b.n, dtype=np.int32), per)
+        parts += [chunk_seq, (np.arange(first[-1], dtype=np.int32) - first[chunk_seq]) * RECUR_CHUNK, first]
+        b.n_chunks = int(first[-1])
         sizes = sorted(earlier)
         rows = []
         for size in sizes:
             carry = np.array([len(e) for e in earlier[size]], dtype=np.int32)
             start = np.zeros(b.n + 1, dtype=np.int32)
             np.cumsum(carry + lens, out=start[1:])
-            first = start[:-1] + carry                              # packed row of the portion's first token
-            parts += [first[seq] + local, first - p0,
+            row0 = start[:-1] + carry                               # packed row of the portion's first token
+            parts += [row0[seq] + local, row0 - p0,
                       np.concatenate([np.asarray(e, dtype=np.int32) for e in earlier[size]]) if carry.sum() else np.zeros(0, np.int32),
                       np.concatenate([start[i] + np.arange(carry[i], dtype=np.int32) for i in range(b.n)])]
             rows.append(int(start[-1]))
         dev = cls._upload(device, parts)
-        b.ids, b.cu, b.pos0, b.slot, b.tok_seq, b.tok_pos, b.entry, b.want, tl = dev[:9]
+        b.ids, b.cu, b.pos0, b.slot, b.tok_seq, b.tok_pos, b.entry, b.want, tl, b.chunk_seq, b.chunk_start, b.chunk_first = dev[:12]
         for i, size in enumerate(sizes):
-            r, base, ge, gr = dev[9 + 4 * i: 13 + 4 * i]
+            r, base, ge, gr = dev[12 + 4 * i: 16 + 4 * i]
             b.views[size] = ChunkView(rows[i], r, base, ge, gr, tl, len(tiles))
         if len(want) == b.T:
             b.want = None

@@ -50,7 +50,7 @@ def main(argv=None) -> int:
     from .hybrid_runner import HybridRunner
     torch.backends.cuda.matmul.allow_tf32 = False
     torch.set_float32_matmul_precision("highest")
-    model = ModelHub.from_pretrained(a.model, dtype=getattr(torch, a.dtype), device="cuda").eval()
+    model = ModelHub.from_pretrained(a.model, dtype=getattr(torch, a.dtype), device="cuda")
     if not hasattr(model, "init_cache"):
         print(f"trace_run: {type(model).__name__} is not served by the hybrid runner", file=sys.stderr)
         return 2
