@@ -81,12 +81,25 @@ __global__ void __launch_bounds__(256) head_norm_gate_kernel(const float* __rest
   const long long t = item / H;
   const int h = (int)(item % H);
   const float* oh = o + (t * H + h) * dv;
+  const A* gr = gate ? gate + t * gate_ld + (long long)h * dv : nullptr;
+  A* yr = y + t * y_ld + (long long)h * dv;
   float ss = 0.f;
+  if (dv == 128) {     // one 16-byte piece per lane
+    const float4 v = *reinterpret_cast<const float4*>(oh + lane * 4);
+    ss = warp_sum(v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w);
+    const float r = mul / sqrtf(ss / dv + eps);
+    const float4 g = *reinterpret_cast<const float4*>(w + lane * 4);
+    float out[4] = {v.x * r * g.x, v.y * r * g.y, v.z * r * g.z, v.w * r * g.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i)
+      if (gr) out[i] *= sigmoid_f(to_f(gr[lane * 4 + i]));
+#pragma unroll
+    for (int i = 0; i < 4; i += 2) store2(yr + lane * 4 + i, out[i], out[i + 1]);
+    return;
+  }
   for (int c = lane; c < dv; c += 32) ss += oh[c] * oh[c];
   ss = warp_sum(ss);
   const float r = mul / sqrtf(ss / dv + eps);
-  const A* gr = gate ? gate + t * gate_ld + (long long)h * dv : nullptr;
-  A* yr = y + t * y_ld + (long long)h * dv;
   for (int c = lane; c < dv; c += 32) {
     float v = oh[c] * r * w[c];
     if (gr) v *= sigmoid_f(to_f(gr[c]));

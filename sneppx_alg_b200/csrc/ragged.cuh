@@ -37,6 +37,10 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float a, float b, float
   *reinterpret_cast<uint2*>(p) = v;
 }
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+// silu of an activation: 32-bit runs take the accurate forms, 16-bit ones the hardware exponential and reciprocal
+template <typename A> __device__ __forceinline__ float silu_act(float x) {
+  return sizeof(A) == 4 ? x * sigmoid_f(x) : __fdividef(x, 1.f + __expf(-x));
+}
 __device__ __forceinline__ float softplus_f(float x) { return fmaxf(x, 0.f) + log1pf(expf(-fabsf(x))); }
 
 // NT tokens of one channel of a short causal convolution: y[t] = sum_b w[b] x[t - b]. `u` points at the first token's row;

@@ -35,7 +35,14 @@ struct DeltaParams {
 // formed by multiplication only, so no decay is ever divided out. A preparation kernel writes everything of a (chunk,
 // head) that does not depend on the state as one contiguous record of fp32 values:
 //   Gq [RC, DP] | Kd [RC, DP] | Gk [RC, DP] (delta) | G_last [DP] | B [RC, RC] | (I + diag(beta) A)^-1 diag(beta) (delta)
-__host__ __device__ constexpr int rec_floats(int DP, bool delta) { return (2 + delta) * RC * DP + DP + (1 + delta) * RC * RC; }
+// with padded row pitches (DP + 8, DP + 4, DP + 8; RC + 8) that keep the tensor-core kernel's fragment reads free of bank
+// conflicts.
+template <int DP, bool DELTA>
+struct Rec {
+  static constexpr int LQ = DP + 8, LK = DP + 4, LB = RC + 8;
+  static constexpr int KD = RC * LQ, GK = KD + RC * LK, GL = GK + (DELTA ? RC * LQ : 0), B = GL + DP, TM = B + RC * LB;
+  static constexpr int FLOATS = TM + (DELTA ? RC * LB : 0);
+};
 
 // Sums of v[16] over the lanes that share a column group (LANES neighbouring lanes): lane rl is left with the sums of
 // tokens rl * TPL .. rl * TPL + TPL - 1 in v[0 .. TPL).
@@ -60,12 +67,13 @@ template <int DP, bool DELTA>
 __device__ __forceinline__ void write_record(const float* __restrict__ sq, const float* __restrict__ sk, const float* __restrict__ sg,
                                              const float* __restrict__ sbeta, float* __restrict__ sA, float* __restrict__ rec, int nt) {
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  using R = Rec<DP, DELTA>;
   float* Gq = rec;
-  float* Kd = rec + RC * DP;
-  float* Gk = rec + 2 * RC * DP;
-  float* Gl = rec + (2 + DELTA) * RC * DP;
-  float* B = Gl + DP;
-  float* Tm = B + RC * RC;
+  float* Kd = rec + R::KD;
+  float* Gk = rec + R::GK;
+  float* Gl = rec + R::GL;
+  float* B = rec + R::B;
+  float* Tm = rec + R::TM;
   for (int i = tid; i < 2 * DP; i += 256) {
     const int c = i % DP;
     float p = 1.f;
@@ -73,14 +81,14 @@ __device__ __forceinline__ void write_record(const float* __restrict__ sq, const
 #pragma unroll
       for (int t = 0; t < RC; ++t) {
         p *= sg[t * DP + c];
-        Gq[t * DP + c] = sq[t * DP + c] * p;
-        if (DELTA) Gk[t * DP + c] = sk[t * DP + c] * p;
+        Gq[t * R::LQ + c] = sq[t * DP + c] * p;
+        if (DELTA) Gk[t * R::LQ + c] = sk[t * DP + c] * p;
       }
       Gl[c] = p;
     } else {
 #pragma unroll
       for (int t = RC - 1; t >= 0; --t) {
-        Kd[t * DP + c] = sk[t * DP + c] * p;
+        Kd[t * R::LK + c] = sk[t * DP + c] * p;
         p *= sg[t * DP + c];
       }
     }
@@ -103,7 +111,7 @@ __device__ __forceinline__ void write_record(const float* __restrict__ sq, const
 #pragma unroll
       for (int n = 0; n < NC; ++n) {
         const int c = lane + 32 * n;
-        if (DP >= 32 || c < DP) {
+        {
           const float k = sk[i * DP + c], g = sg[i * DP + c];
           bq[i] = fmaf(qp[n], k, bq[i]);
           qp[n] *= g;
@@ -118,7 +126,7 @@ __device__ __forceinline__ void write_record(const float* __restrict__ sq, const
 #pragma unroll
     for (int i = 0; i < RC; ++i) bq[i] += __shfl_xor_sync(0xffffffffu, bq[i], 16);
     reduce_tokens<16>(bq, lane & 15);
-    if (lane < 16) B[t * RC + lane] = lane <= t ? bq[0] : 0.f;
+    if (lane < 16) B[t * R::LB + lane] = lane <= t ? bq[0] : 0.f;
     if constexpr (DELTA) {
 #pragma unroll
       for (int i = 0; i < RC; ++i) ak[i] += __shfl_xor_sync(0xffffffffu, ak[i], 16);
@@ -136,7 +144,7 @@ __device__ __forceinline__ void write_record(const float* __restrict__ sq, const
 #pragma unroll
         for (int i = 0; i < t; ++i) s = fmaf(-sA[t * RC + i], x[i], s);
         x[t] = sbeta[t] * s;
-        Tm[t * RC + tid] = x[t];
+        Tm[t * R::LB + tid] = x[t];
       }
     }
   }
@@ -146,7 +154,7 @@ template <typename A, int DP>
 __global__ void __launch_bounds__(256) gate_chunk_kernel(const A* __restrict__ qr, const A* __restrict__ fr, long long ld,
                                                          const float* __restrict__ bias, const float* __restrict__ lower,
                                                          float* __restrict__ rec, const RaggedView rv, const ChunkView cv, int H, int d) {
-  extern __shared__ __align__(16) float sm[];
+  extern __shared__ __align__(128) float sm[];
   float* sq = sm;
   float* sk = sq + RC * DP;
   float* sg = sk + RC * DP;
@@ -159,7 +167,7 @@ __global__ void __launch_bounds__(256) gate_chunk_kernel(const A* __restrict__ q
     if (t < nt && c < d) {
       const long long o = (long long)(row0 + t) * ld + h * d + c;
       const float z = to_f(qr[o]), l = lower[h * d + c];
-      q = z * sigmoid_f(z);
+      q = silu_act<A>(z);
       f = l + (1.f - l) * sigmoid_f(to_f(fr[o]) + bias[h * d + c]);
     }
     sq[i] = q;
@@ -167,12 +175,12 @@ __global__ void __launch_bounds__(256) gate_chunk_kernel(const A* __restrict__ q
     sk[i] = 1.f - f;       // 0 on padding
   }
   __syncthreads();
-  write_record<DP, false>(sq, sk, sg, nullptr, nullptr, rec + ((long long)ch * H + h) * rec_floats(DP, false), nt);
+  write_record<DP, false>(sq, sk, sg, nullptr, nullptr, rec + ((long long)ch * H + h) * Rec<DP, false>::FLOATS, nt);
 }
 
 template <typename A, int DP, int MT>
-__global__ void __launch_bounds__(256) delta_chunk_kernel(const DeltaParams p, float* __restrict__ rec, const ChunkView cv) {
-  extern __shared__ __align__(16) float sm[];
+__global__ void __launch_bounds__(256, MT <= 4 && DP <= 128 ? 4 : 1) delta_chunk_kernel(const DeltaParams p, float* __restrict__ rec, const ChunkView cv) {
+  extern __shared__ __align__(128) float sm[];
   float* sq = sm;
   float* sk = sq + RC * DP;
   float* sg = sk + RC * DP;
@@ -183,6 +191,16 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const DeltaParams p, f
   const int pos = p.rv.pos0[seq] + s0, C = 2 * p.G * p.d + p.H * p.dv;
   const A* u = reinterpret_cast<const A*>(p.u) + (long long)row0 * p.u_ld;
   const A* ring = reinterpret_cast<const A*>(p.ring) + (long long)p.rv.slot[seq] * p.taps * C;
+  // decay inputs and write strengths: in flight while the convolutions run
+  constexpr int NA = RC * DP / 256;
+  const A* ar = reinterpret_cast<const A*>(p.a) + (long long)row0 * p.a_ld + (long long)h * p.d;
+  A av[NA], bv = from_f<A>(0.f);
+#pragma unroll
+  for (int n = 0; n < NA; ++n) {
+    const int t = (tid + n * 256) / DP, c = tid % DP;
+    av[n] = (t < nt && c < p.d) ? ar[(long long)t * p.a_ld + c] : from_f<A>(0.f);
+  }
+  if (tid < nt) bv = reinterpret_cast<const A*>(p.b)[(long long)(row0 + tid) * p.b_ld + h];
   for (int i = tid; i < 2 * DP + p.dv; i += 256) {
     const bool is_v = i >= 2 * DP;
     const int which = i / DP, c = is_v ? i - 2 * DP : i % DP;
@@ -191,7 +209,7 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const DeltaParams p, f
       const int col = is_v ? 2 * p.G * p.d + h * p.dv + c : (which * p.G + hq) * p.d + c;
       conv_walk<A, RC, MT>(u, p.u_ld, p.wconv, p.taps, C, col, ring, pos, s0, nt, y);
 #pragma unroll
-      for (int t = 0; t < RC; ++t) y[t] *= sigmoid_f(y[t]);
+      for (int t = 0; t < RC; ++t) y[t] = silu_act<A>(y[t]);
     } else {
 #pragma unroll
       for (int t = 0; t < RC; ++t) y[t] = 0.f;
@@ -208,14 +226,12 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const DeltaParams p, f
     }
   }
   const float al = -expf(p.a_log[h]);
-  const A* ar = reinterpret_cast<const A*>(p.a) + (long long)row0 * p.a_ld + (long long)h * p.d;
-#pragma unroll 4
-  for (int i = tid; i < RC * DP; i += 256) {
-    const int t = i / DP, c = i % DP;
-    sg[i] = (t < nt && c < p.d) ? expf(al * softplus_f(to_f(ar[(long long)t * p.a_ld + c]) + p.dt_bias[h * p.d + c])) : 1.f;
+#pragma unroll
+  for (int n = 0; n < NA; ++n) {
+    const int i = tid + n * 256, t = i / DP, c = i % DP;
+    sg[i] = (t < nt && c < p.d) ? expf(al * softplus_f(to_f(av[n]) + p.dt_bias[h * p.d + c])) : 1.f;
   }
-  if (tid < RC)
-    sb[tid] = tid < nt ? sigmoid_f(to_f(reinterpret_cast<const A*>(p.b)[(long long)(row0 + tid) * p.b_ld + h])) : 0.f;
+  if (tid < RC) sb[tid] = tid < nt ? sigmoid_f(to_f(bv)) : 0.f;
   __syncthreads();
   const float qs = 1.f / sqrtf((float)p.d);
   for (int i = warp; i < 2 * RC; i += 8) {
@@ -227,7 +243,7 @@ __global__ void __launch_bounds__(256) delta_chunk_kernel(const DeltaParams p, f
     for (int c = lane; c < DP; c += 32) row[c] *= r;
   }
   __syncthreads();
-  write_record<DP, true>(sq, sk, sg, sb, sA, rec + ((long long)ch * p.H + h) * rec_floats(DP, true), nt);
+  write_record<DP, true>(sq, sk, sg, sb, sA, rec + ((long long)ch * p.H + h) * Rec<DP, true>::FLOATS, nt);
 }
 
 // ------------------------------------------------------------------ scan over the chunks of a portion
@@ -279,7 +295,7 @@ struct ScanCfg {
   static constexpr int CW = GW * CN;                 // columns per warp
   static constexpr int CT = 4 * CW;                  // columns per CTA
   static constexpr int TPL = RC / LANES;             // tokens whose sums a lane ends up with
-  static constexpr int REC = rec_floats(DP, DELTA);
+  static constexpr int REC = Rec<DP, DELTA>::FLOATS;
   static constexpr int VN = (RC * CT + 127) / 128;
   static constexpr int SMEM = (2 * REC + 2 * RC * CT + (DELTA ? 2 * RC * CT : 0)) * 4 + 64;
 };
@@ -287,7 +303,7 @@ struct ScanCfg {
 template <typename A, bool DELTA, int LANES, int CN>
 __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
   using Cfg = ScanCfg<A, DELTA, LANES, CN>;
-  constexpr int DP = Cfg::DP, CT = Cfg::CT, CW = Cfg::CW, GW = Cfg::GW, REC = Cfg::REC, TPL = Cfg::TPL, VN = Cfg::VN;
+  constexpr int DP = Cfg::DP, CT = Cfg::CT, CW = Cfg::CW, REC = Cfg::REC, TPL = Cfg::TPL, VN = Cfg::VN;
   extern __shared__ __align__(128) float sm[];
   float* sV = sm + 2 * REC;                          // [2][RC][CT]
   float* sX = sV + 2 * RC * CT;                      // [RC][CT] per-warp column blocks: V - W, then U
@@ -349,6 +365,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
   put_v(0);
   __syncthreads();
   // sum over this thread's rows of S[cn] * op[t][rows], for the 16 tokens, then over the lanes of the column
+  using RL = Rec<DP, DELTA>;
   auto project = [&](const float* op, float (&acc)[CN][RC]) {
 #pragma unroll
     for (int t = 0; t < RC; ++t) {
@@ -357,7 +374,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
       for (int cn = 0; cn < CN; ++cn) a[cn][0] = a[cn][1] = 0;
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(op + t * DP + c * LANES * 4 + rl * 4);
+        const ulonglong2 x = *reinterpret_cast<const ulonglong2*>(op + t * RL::LQ + c * LANES * 4 + rl * 4);
 #pragma unroll
         for (int cn = 0; cn < CN; ++cn) {
           a[cn][0] = fma2(S[cn][2 * c], x.x, a[cn][0]);
@@ -386,14 +403,14 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
     ok = mbar_wait_warp(&full[buf], (ci >> 1) & 1, s_abort, p.status, ST_TIMEOUT_PRODUCER);
     if (!ok) break;
     const float* R = sm + buf * REC;
-    const float* Kd = R + RC * DP;
-    const float* Gl = R + (2 + DELTA) * RC * DP;
-    const float* B = Gl + DP;
+    const float* Kd = R + RL::KD;
+    const float* Gl = R + RL::GL;
+    const float* B = R + RL::B;
     const float* V = sV + buf * RC * CT;
     const float* U = V;
     if constexpr (DELTA) {
       float w[CN][RC];
-      project(R + 2 * RC * DP, w);
+      project(R + RL::GK, w);
 #pragma unroll
       for (int i = 0; i < TPL; ++i)
 #pragma unroll
@@ -406,7 +423,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
     project(R, q);
     if constexpr (DELTA) {
       __syncwarp();
-      const float* Tm = B + RC * RC;
+      const float* Tm = R + RL::TM;
       float x[CN][TPL];
 #pragma unroll
       for (int cn = 0; cn < CN; ++cn)
@@ -421,7 +438,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
           for (int cn = 0; cn < CN; ++cn) xv[cn][e] = sX[(j + e) * CT + cloc + cn];
 #pragma unroll
         for (int i = 0; i < TPL; ++i) {
-          const float4 m = *reinterpret_cast<const float4*>(Tm + (rl * TPL + i) * RC + j);
+          const float4 m = *reinterpret_cast<const float4*>(Tm + (rl * TPL + i) * RL::LB + j);
 #pragma unroll
           for (int cn = 0; cn < CN; ++cn)
             x[cn][i] = fmaf(m.w, xv[cn][3], fmaf(m.z, xv[cn][2], fmaf(m.y, xv[cn][1], fmaf(m.x, xv[cn][0], x[cn][i]))));
@@ -444,7 +461,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
         for (int cn = 0; cn < CN; ++cn) uv[cn][e] = U[(j + e) * CT + cloc + cn];
 #pragma unroll
       for (int i = 0; i < TPL; ++i) {
-        const float4 m = *reinterpret_cast<const float4*>(B + (rl * TPL + i) * RC + j);
+        const float4 m = *reinterpret_cast<const float4*>(B + (rl * TPL + i) * RL::LB + j);
 #pragma unroll
         for (int cn = 0; cn < CN; ++cn)
           q[cn][i] = fmaf(m.w, uv[cn][3], fmaf(m.z, uv[cn][2], fmaf(m.y, uv[cn][1], fmaf(m.x, uv[cn][0], q[cn][i]))));
@@ -477,7 +494,7 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
       }
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
-        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(Kd + t * DP + c * LANES * 4 + rl * 4);
+        const ulonglong2 k = *reinterpret_cast<const ulonglong2*>(Kd + t * RL::LK + c * LANES * 4 + rl * 4);
 #pragma unroll
         for (int cn = 0; cn < CN; ++cn) {
           S[cn][2 * c] = fma2(k.x, u2[cn], S[cn][2 * c]);
@@ -506,6 +523,224 @@ __global__ void __launch_bounds__(128) recur_scan_kernel(const ScanParams p) {
   }
 }
 
+// ------------------------------------------------------------------ the same scan on tensor cores
+// All products of a chunk are small matrix products with the transposed state S^T [columns, d] as an operand or result:
+//   W^T = S^T (G k)^T, Q^T = S^T (G q)^T,  U^T = (V - W)^T Tm^T,  O^T = Q^T + U^T B^T,  S^T <- S^T G_last + U^T Kd
+// They run as mma.m16n8k8 with every fp32 operand split into two TF32 terms (x = hi + lo with lo = x - hi exactly) and three
+// products hi hi + hi lo + lo hi accumulated in fp32: what is dropped, lo lo and the rounding of lo, is below 2^-21 of a
+// product. The accumulator layout of m16n8 (columns 2t, 2t + 1 of row g) is read back as an A operand whose k index t / t + 4
+// stands for 2t / 2t + 1; the B operands are fetched in that order, so state, W, Q, U and O never leave their registers.
+// A warp owns 16 value columns. SPLITD: the four warps of a CTA share those columns and own a quarter of d each (few
+// sequences: more CTAs); otherwise they own 16 columns each.
+__device__ __forceinline__ void mma_tf32(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k8.row.col.f32.tf32.tf32.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void split_tf32(float x, uint32_t& hi, uint32_t& lo) {
+  hi = __float_as_uint(x) & 0xffffe000u;
+  lo = __float_as_uint(x - __uint_as_float(hi));
+}
+// accumulator fragment -> A operand terms
+__device__ __forceinline__ void split_frag(const float (&c)[4], uint32_t (&hi)[4], uint32_t (&lo)[4]) {
+  split_tf32(c[0], hi[0], lo[0]);
+  split_tf32(c[2], hi[1], lo[1]);
+  split_tf32(c[1], hi[2], lo[2]);
+  split_tf32(c[3], hi[3], lo[3]);
+}
+template <bool A_EXACT>
+__device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], float b0, float b1) {
+  uint32_t h0, l0, h1, l1;
+  split_tf32(b0, h0, l0);
+  split_tf32(b1, h1, l1);
+  mma_tf32(c, ah, l0, l1);
+  if (!A_EXACT) mma_tf32(c, al, h0, h1);
+  mma_tf32(c, ah, h0, h1);
+}
+
+template <bool DELTA, int DP, bool SPLITD>
+struct TcScanCfg {
+  static constexpr int COLS = SPLITD ? 16 : 64;
+  static constexpr int ND = (SPLITD ? DP / 4 : DP) / 8;       // 8-row tiles of d per warp
+  static constexpr int REC = Rec<DP, DELTA>::FLOATS;
+  static constexpr int XCH = SPLITD ? 2 * 4 * (1 + DELTA) * 8 * 32 : 0;   // [2][warp][quantity][8 values][lane]
+  static constexpr int FIT = (227 * 256 - 16 - XCH) / REC;
+  static constexpr int STAGES = FIT < (SPLITD ? 5 : 3) ? FIT : (SPLITD ? 5 : 3);   // a copy takes longer than a chunk
+  static constexpr int SMEM = (STAGES * REC + XCH) * 4 + 64;
+  static_assert(STAGES >= 2 && SMEM <= 227 * 1024, "shared memory");
+};
+
+template <typename A, bool DELTA, int DP, bool SPLITD>
+__global__ void __launch_bounds__(128) recur_scan_tc_kernel(const ScanParams p) {
+  using Cfg = TcScanCfg<DELTA, DP, SPLITD>;
+  using RL = Rec<DP, DELTA>;
+  constexpr int ND = Cfg::ND, REC = Cfg::REC, STAGES = Cfg::STAGES;
+  constexpr bool V_EXACT = !DELTA && sizeof(A) == 2;          // bf16 values have no low TF32 term
+  extern __shared__ __align__(128) float sm[];
+  float* xch = sm + STAGES * REC;
+  uint64_t* full = reinterpret_cast<uint64_t*>(sm + (Cfg::SMEM - 64) / 4);
+  volatile int* s_abort = reinterpret_cast<volatile int*>(full + STAGES);
+  const int seq = blockIdx.z, h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t = lane & 3;
+  const int c0 = blockIdx.x * Cfg::COLS + (SPLITD ? 0 : warp * 16), d0 = SPLITD ? warp * (DP / 4) : 0;
+  const int row0 = p.rv.cu[seq], len = p.rv.cu[seq + 1] - row0;
+  if (len <= 0) return;
+  const int n_ch = (len + RC - 1) / RC;
+  float* st = p.state + ((long long)p.rv.slot[seq] * p.H + h) * p.d * p.dv;
+  const bool fresh = p.rv.pos0[seq] == 0;
+  const float* rec = p.rec + ((long long)p.cv.first[seq] * p.H + h) * REC;
+  const long long rec_step = (long long)p.H * REC;
+  if (tid == 0) {
+    for (int s = 0; s < STAGES; ++s) mbar_init(&full[s], 1);
+    *s_abort = 0;
+    mbar_fence_init();
+    for (int s = 0; s < STAGES && s < n_ch; ++s) {
+      mbar_expect_tx(&full[s], REC * 4);
+      bulk_load(sm + s * REC, rec + s * rec_step, REC * 4, &full[s]);
+    }
+  }
+  float S[ND][4];
+#pragma unroll
+  for (int j = 0; j < ND; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = d0 + 8 * j + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+      S[j][e] = (!fresh && r < p.d && c < p.dv) ? st[(long long)r * p.dv + c] : 0.f;
+    }
+  // values of a chunk in accumulator layout: token 8 n + 2 t + (e & 1), column g + 8 (e >> 1)
+  const A* vp = reinterpret_cast<const A*>(p.v) + (long long)h * p.dv;
+  auto load_v = [&](int t0, float (&v)[2][4]) {
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int tok = t0 + 8 * n + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+        v[n][e] = (tok < len && c < p.dv) ? to_f(vp[(long long)(row0 + tok) * p.v_ld + c]) : 0.f;
+      }
+  };
+  float vn[2][4];
+  load_v(0, vn);
+  __syncthreads();
+  for (int ci = 0; ci < n_ch; ++ci) {
+    const int buf = ci % STAGES, t0 = ci * RC;
+    float v[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) v[n][e] = vn[n][e];
+    if (ci + 1 < n_ch) load_v(t0 + RC, vn);
+    if (!mbar_wait_warp(&full[buf], (ci / STAGES) & 1, s_abort, p.status, ST_TIMEOUT_PRODUCER)) break;
+    const float* R = sm + buf * REC;
+    float q[2][4], w[2][4];
+#pragma unroll
+    for (int n = 0; n < 2; ++n)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) q[n][e] = w[n][e] = 0.f;
+#pragma unroll
+    for (int j = 0; j < ND; ++j) {
+      uint32_t ah[4], al[4];
+      split_frag(S[j], ah, al);
+      const float* base = R + g * RL::LQ + d0 + 8 * j + 2 * t;
+#pragma unroll
+      for (int n = 0; n < 2; ++n) {
+        if constexpr (DELTA) {
+          const float2 b = *reinterpret_cast<const float2*>(base + RL::GK + n * 8 * RL::LQ);
+          mma_split<false>(w[n], ah, al, b.x, b.y);
+        }
+        const float2 b = *reinterpret_cast<const float2*>(base + n * 8 * RL::LQ);
+        mma_split<false>(q[n], ah, al, b.x, b.y);
+      }
+    }
+    if constexpr (SPLITD) {
+      float* x = xch + (ci & 1) * 4 * (1 + DELTA) * 256;
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          x[(warp * (1 + DELTA)) * 256 + (n * 4 + e) * 32 + lane] = q[n][e];
+          if (DELTA) x[(warp * 2 + 1) * 256 + (n * 4 + e) * 32 + lane] = w[n][e];
+        }
+      __syncthreads();
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int i = (n * 4 + e) * 32 + lane;
+          q[n][e] = (x[i] + x[(1 + DELTA) * 256 + i]) + (x[2 * (1 + DELTA) * 256 + i] + x[3 * (1 + DELTA) * 256 + i]);
+          if (DELTA) w[n][e] = (x[256 + i] + x[768 + i]) + (x[1280 + i] + x[1792 + i]);
+        }
+    }
+    uint32_t uh[2][4], ul[2][4];       // written values as A operand
+    if constexpr (DELTA) {
+      float u[2][4];
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          w[n][e] = v[n][e] - w[n][e];
+          u[n][e] = 0.f;
+        }
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        uint32_t xh[4], xl[4];
+        split_frag(w[k], xh, xl);
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+          if (k <= n) {                // lower triangular
+            const float2 b = *reinterpret_cast<const float2*>(R + RL::TM + (n * 8 + g) * RL::LB + k * 8 + 2 * t);
+            mma_split<false>(u[n], xh, xl, b.x, b.y);
+          }
+      }
+#pragma unroll
+      for (int n = 0; n < 2; ++n) split_frag(u[n], uh[n], ul[n]);
+    } else {
+#pragma unroll
+      for (int n = 0; n < 2; ++n) split_frag(v[n], uh[n], ul[n]);
+    }
+    if (!SPLITD || warp == (ci & 3)) {
+#pragma unroll
+      for (int k = 0; k < 2; ++k)
+#pragma unroll
+        for (int n = 0; n < 2; ++n)
+          if (k <= n) {
+            const float2 b = *reinterpret_cast<const float2*>(R + RL::B + (n * 8 + g) * RL::LB + k * 8 + 2 * t);
+            mma_split<V_EXACT>(q[n], uh[k], ul[k], b.x, b.y);
+          }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          const int tok = t0 + 8 * n + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+          if (tok < len && c < p.dv) p.o[((long long)(row0 + tok) * p.H + h) * p.dv + c] = q[n][e];
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < ND; ++j) {
+      const float2 gl = *reinterpret_cast<const float2*>(R + RL::GL + d0 + 8 * j + 2 * t);
+      S[j][0] *= gl.x; S[j][1] *= gl.y; S[j][2] *= gl.x; S[j][3] *= gl.y;
+#pragma unroll
+      for (int k = 0; k < 2; ++k) {
+        const float* kd = R + RL::KD + (k * 8 + 2 * t) * RL::LK + d0 + 8 * j + g;
+        mma_split<V_EXACT>(S[j], uh[k], ul[k], kd[0], kd[RL::LK]);
+      }
+    }
+    __syncthreads();
+    if (tid == 0 && ci + STAGES < n_ch) {
+      mbar_expect_tx(&full[buf], REC * 4);
+      bulk_load(sm + buf * REC, rec + (ci + STAGES) * rec_step, REC * 4, &full[buf]);
+    }
+  }
+  if (*s_abort) {
+    bounded_delay_ns(2000000);
+    return;
+  }
+#pragma unroll
+  for (int j = 0; j < ND; ++j)
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int r = d0 + 8 * j + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
+      if (r < p.d && c < p.dv) st[(long long)r * p.dv + c] = S[j][e];
+    }
+}
+
 // ------------------------------------------------------------------ one token per sequence
 // One CTA per (head, sequence): operands from the projected rows (convolution, unit norms, gates), one state update with
 // the state tile in registers between its two passes, read-out, per-head norm and output gate.
@@ -524,7 +759,7 @@ struct StepParams {
 
 template <typename A, bool DELTA, int VEC, int NR>
 __global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1) recur_step_kernel(const StepParams p) {
-  extern __shared__ __align__(16) float sm[];
+  extern __shared__ __align__(128) float sm[];
   float* sq = sm;             // [d]
   float* sk = sq + p.d;       // [d]
   float* sg = sk + p.d;       // [d]
@@ -700,10 +935,17 @@ static void fill_delta(DeltaParams* p, const SxDeltaArgs* a) {
   p->rv = view(&a->ragged);
   p->T = a->T; p->H = a->H; p->G = a->G; p->d = a->d; p->dv = a->dv; p->taps = a->taps;
 }
-static int pad_rows(int d) { return d <= 16 ? 16 : d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
+static int pad_rows(int d) { return d <= 32 ? 32 : d <= 64 ? 64 : d <= 128 ? 128 : 256; }
 
 // Floats of scratch that the records of one (chunk, head) take.
-extern "C" int sx_recur_record(int d, int delta) { return rec_floats(pad_rows(d), delta != 0); }
+extern "C" int sx_recur_record(int d, int delta) {
+  switch (pad_rows(d)) {
+    case 32: return delta ? Rec<32, true>::FLOATS : Rec<32, false>::FLOATS;
+    case 64: return delta ? Rec<64, true>::FLOATS : Rec<64, false>::FLOATS;
+    case 128: return delta ? Rec<128, true>::FLOATS : Rec<128, false>::FLOATS;
+    default: return delta ? Rec<256, true>::FLOATS : Rec<256, false>::FLOATS;
+  }
+}
 
 template <typename K>
 static int allow_smem(K kern, int bytes, bool* done) {
@@ -730,7 +972,6 @@ extern "C" int sx_gate_chunks(const SxGateArgs* a, cudaStream_t st) {
   if (a->d <= 0 || a->d > 256) return -1;
   SX_ACT_DISPATCH(a->f32, {
     switch (pad_rows(a->d)) {
-      case 16: return launch_gate_chunks<A, 16>(a, st);
       case 32: return launch_gate_chunks<A, 32>(a, st);
       case 64: return launch_gate_chunks<A, 64>(a, st);
       case 128: return launch_gate_chunks<A, 128>(a, st);
@@ -762,7 +1003,6 @@ extern "C" int sx_delta_chunks(const SxDeltaArgs* a, const SxChunks* c, float* r
   const ChunkView cv = chunks(c);
   SX_ACT_DISPATCH(a->f32, {
     switch (pad_rows(a->d)) {
-      case 16: return pick_delta_chunks<A, 16>(p, rec, cv, st);
       case 32: return pick_delta_chunks<A, 32>(p, rec, cv, st);
       case 64: return pick_delta_chunks<A, 64>(p, rec, cv, st);
       case 128: return pick_delta_chunks<A, 128>(p, rec, cv, st);
@@ -788,7 +1028,6 @@ static int pick_scan(const ScanParams& p, cudaStream_t st) {
   const bool wide = (long long)((p.dv + ct1 - 1) / ct1) * p.H * p.rv.n > 2 * 148;
 #define SX_SCAN(L) return wide ? launch_scan<A, DELTA, L, 2>(p, st) : launch_scan<A, DELTA, L, 1>(p, st)
   switch (lanes) {
-    case 1: SX_SCAN(1);
     case 2: SX_SCAN(2);
     case 4: SX_SCAN(4);
     case 8: SX_SCAN(8);
@@ -797,7 +1036,31 @@ static int pick_scan(const ScanParams& p, cudaStream_t st) {
 #undef SX_SCAN
 }
 
-// delta != 0: gated delta rule; else the gated write. Portions are independent of each other.
+template <typename A, bool DELTA, int DP, bool SPLITD>
+static int launch_scan_tc(const ScanParams& p, cudaStream_t st) {
+  using Cfg = TcScanCfg<DELTA, DP, SPLITD>;
+  static bool set = false;
+  if (int rc = allow_smem(recur_scan_tc_kernel<A, DELTA, DP, SPLITD>, Cfg::SMEM, &set)) return rc;
+  dim3 grid((p.dv + Cfg::COLS - 1) / Cfg::COLS, p.H, p.rv.n);
+  recur_scan_tc_kernel<A, DELTA, DP, SPLITD><<<grid, 128, Cfg::SMEM, st>>>(p);
+  return last_rc();
+}
+template <bool DELTA>
+static int pick_scan_tc(const ScanParams& p, cudaStream_t st) {
+  using A = __nv_bfloat16;
+  const bool many = (long long)((p.dv + 63) / 64) * p.H * p.rv.n >= 148;   // 64 columns per CTA already fill the machine
+#define SX_SCAN_TC(D) return many ? launch_scan_tc<A, DELTA, D, false>(p, st) : launch_scan_tc<A, DELTA, D, true>(p, st)
+  switch (pad_rows(p.d)) {
+    case 32: SX_SCAN_TC(32);
+    case 64: SX_SCAN_TC(64);
+    case 128: SX_SCAN_TC(128);
+    default: SX_SCAN_TC(256);
+  }
+#undef SX_SCAN_TC
+}
+
+// delta != 0: gated delta rule; else the gated write. Portions are independent of each other. 32-bit runs take the SIMT
+// kernel, bf16 runs the tensor-core kernel.
 extern "C" int sx_recur_scan(const SxScanArgs* a, cudaStream_t st) {
   if (a->ragged.n <= 0) return 0;
   if (a->d <= 0 || a->d > 256 || a->dv <= 0) return -1;
@@ -805,8 +1068,8 @@ extern "C" int sx_recur_scan(const SxScanArgs* a, cudaStream_t st) {
   p.rec = a->rec; p.v = a->v; p.v_ld = a->v_ld; p.state = a->state; p.o = a->o; p.status = a->status;
   p.rv = view(&a->ragged); p.cv = chunks(&a->chunks);
   p.H = a->H; p.d = a->d; p.dv = a->dv;
-  SX_ACT_DISPATCH(a->f32, { return a->delta ? pick_scan<A, true>(p, st) : pick_scan<A, false>(p, st); });
-  return 0;
+  if (a->f32) return a->delta ? pick_scan<float, true>(p, st) : pick_scan<float, false>(p, st);
+  return a->delta ? pick_scan_tc<true>(p, st) : pick_scan_tc<false>(p, st);
 }
 
 template <typename A, bool DELTA, int VEC>

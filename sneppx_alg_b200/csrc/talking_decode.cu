@@ -65,7 +65,8 @@ __host__ __device__ inline DecLayout dec_layout(int H, int G, int d, int dv, int
   return L;
 }
 
-template <int KT, int MAXI>
+// QREG: every warp has one QK item of at most 16 k-steps, whose query fragments then stay in registers.
+template <int KT, int MAXI, bool QREG>
 __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p) {
   extern __shared__ __align__(16) uint8_t smem[];
   const DecLayout L = dec_layout(p.H, p.G, p.d, p.dv, KT, p.stages, p.ksplit);
@@ -91,12 +92,18 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     if (tile < n_tiles) {
       __nv_bfloat16* sk = sKV + (tile % p.stages) * L.stage;
       __nv_bfloat16* sv = sk + KT * L.ldk;
-      const int j0 = lo + tile * KT;
-      for (int r = warp; r < KT; r += 8) {
-        const int j = min(j0 + r, hi - 1);          // rows past the end repeat the last key and are masked
-        const long long e = (long long)table[j / p.block_size - base] * p.block_size + j % p.block_size;
-        const __nv_bfloat16* kr = p.k + e * Gd;
-        const __nv_bfloat16* vr = p.v + e * Gv;
+      // rows past the end repeat the last key and are masked; lane i finds the entry of the warp's i-th row
+      int e = 0;
+      if (lane < KT / 8) {
+        const int j = min(lo + tile * KT + warp + 8 * lane, hi - 1), b = j / p.block_size;
+        e = table[b - base] * p.block_size + j - b * p.block_size;
+      }
+#pragma unroll
+      for (int i = 0; i < KT / 8; ++i) {
+        const long long er = __shfl_sync(0xffffffffu, e, i);
+        const int r = warp + 8 * i;
+        const __nv_bfloat16* kr = p.k + er * Gd;
+        const __nv_bfloat16* vr = p.v + er * Gv;
         for (int c = lane; c < Gd / 8; c += 32) dec_cp16(sk + r * L.ldk + c * 8, kr + c * 8);
         for (int c = lane; c < Gv / 8; c += 32) dec_cp16(sv + r * L.ldv + c * 8, vr + c * 8);
       }
@@ -128,65 +135,131 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
   for (int i = 0; i < MAXI; ++i) O[i][0] = O[i][1] = O[i][2] = O[i][3] = 0.f;
   const int nt8 = p.dv / 8, items = G * nt8, units = (KT / 8) * (L.HP / 16), ksteps = L.D16 / 16;
 
-  for (int tile = 0; tile < n_tiles; ++tile) {
-    if (p.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
-    else asm volatile("cp.async.wait_group 1;" ::: "memory");
+  // scores of a tile: (8 keys x 16 heads) units, each cut along k into ksplit parts
+  uint32_t qf[QREG ? 16 : 1][4];
+  if constexpr (QREG) {
+    const int unit = warp % units, ks = warp / units, m0 = unit / (KT / 8) * 16, k0 = ksteps * ks / p.ksplit;
     __syncthreads();
-    fetch(tile + p.stages - 1);
+#pragma unroll
+    for (int kk = 0; kk < 16; ++kk) {
+      qf[kk][0] = qf[kk][1] = qf[kk][2] = qf[kk][3] = 0;
+      if (ks < p.ksplit && k0 + kk < ksteps * (ks + 1) / p.ksplit)
+        ldsm4(qf[kk], sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8 + (k0 + kk) * 16);
+    }
+  }
+  auto scores = [&](int tile) {
     const __nv_bfloat16* sk = sKV + (tile % p.stages) * L.stage;
-    const __nv_bfloat16* sv = sk + KT * L.ldk;
     for (int it = warp; it < units * p.ksplit; it += 8) {
       const int unit = it % units, ks = it / units, n0 = (unit % (KT / 8)) * 8, m0 = unit / (KT / 8) * 16;
       const int k0 = ksteps * ks / p.ksplit, k1 = ksteps * (ks + 1) / p.ksplit;
       const __nv_bfloat16* qa = sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8;
-      const __nv_bfloat16* kb = sk + (n0 + (lane & 7)) * L.ldk + ((lane >> 3) & 1) * 8;
       float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-      int kk = k0;
-      for (; kk + 1 < k1; kk += 2) {
-        uint32_t a[4], b[2], a2[4], b2[2];
-        ldsm4(a, qa + kk * 16);
-        ldsm2(b, kb + kk * 16);
-        ldsm4(a2, qa + kk * 16 + 16);
-        ldsm2(b2, kb + kk * 16 + 16);
-        mma16816(c0, a, b);
-        mma16816(c1, a2, b2);
-      }
-      if (kk < k1) {
-        uint32_t a[4], b[2];
-        ldsm4(a, qa + kk * 16);
-        ldsm2(b, kb + kk * 16);
-        mma16816(c0, a, b);
+      const __nv_bfloat16* kb = sk + (n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8;   // four 8-wide k pieces per load
+      if constexpr (QREG) {
+#pragma unroll
+        for (int kk = 0; kk < 16; kk += 2) {
+          if (k0 + kk + 1 < k1) {
+            uint32_t b[4];
+            ldsm4(b, kb + (k0 + kk) * 16);
+            const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+            mma16816(c0, qf[kk], b0);
+            mma16816(c1, qf[kk + 1], b1);
+          } else if (k0 + kk < k1) {
+            uint32_t b[2];
+            ldsm2(b, kb + (k0 + kk) * 16);
+            mma16816(c0, qf[kk], b);
+          }
+        }
+      } else {
+        int kk = k0;
+#pragma unroll 4
+        for (; kk + 1 < k1; kk += 2) {
+          uint32_t a[4], a2[4], b[4];
+          ldsm4(a, qa + kk * 16);
+          ldsm4(a2, qa + kk * 16 + 16);
+          ldsm4(b, kb + kk * 16);
+          const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+          mma16816(c0, a, b0);
+          mma16816(c1, a2, b1);
+        }
+        if (kk < k1) {
+          uint32_t a[4], b[2];
+          ldsm4(a, qa + kk * 16);
+          ldsm2(b, kb + kk * 16);
+          mma16816(c0, a, b);
+        }
       }
       float* s = sS + (ks * L.HP + m0 + (lane >> 2)) * L.lds + n0 + (lane & 3) * 2;
       *reinterpret_cast<float2*>(s) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
       *reinterpret_cast<float2*>(s + 8 * L.lds) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
+  };
+  auto arrived = [&]() {
+    if (p.stages == 2) asm volatile("cp.async.wait_group 0;" ::: "memory");
+    else asm volatile("cp.async.wait_group 1;" ::: "memory");
     __syncthreads();
+  };
+  if (n_tiles > 0) {
+    arrived();
+    scores(0);
+  }
+  for (int tile = 0; tile < n_tiles; ++tile) {
+    __syncthreads();          // scores of this tile are complete, and nobody reads the stage refilled next
+    fetch(tile + p.stages - 1);
     const int nk = min(KT, hi - lo - tile * KT);
-    for (int h = warp; h < H; h += 8) {
-      float s = -INFINITY;
-      if (lane < nk) {
-        s = 0.f;
-        for (int ks = 0; ks < p.ksplit; ++ks) s += sS[(ks * L.HP + h) * L.lds + lane];
-        s *= p.scale;
+    // two heads at a time, so that their reductions overlap
+    for (int h0 = warp; h0 < H; h0 += 16) {
+      const bool two = h0 + 8 < H;
+      float s[2], m_old[2], m[2], l[2];
+      __nv_bfloat16 e[2];
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        const int h = two ? h0 + 8 * x : h0;
+        s[x] = -INFINITY;
+        if (lane < nk) {
+          s[x] = 0.f;
+          for (int ks = 0; ks < p.ksplit; ++ks) s[x] += sS[(ks * L.HP + h) * L.lds + lane];
+          s[x] *= p.scale;
+        }
+        m_old[x] = sM[h];
+        m[x] = s[x];
       }
-      const float m_old = sM[h], m = fmaxf(m_old, warp_max(s));
-      const __nv_bfloat16 e = __float2bfloat16_rn(exp2f((s - m) * 1.4426950408889634f));
-      const float l = warp_sum(__bfloat162float(e));
-      if (lane < KT) sP[h * L.ldp + lane] = e;
-      if (lane == 0) {
-        const float c = exp2f((m_old - m) * 1.4426950408889634f);
-        sC[h] = c;
-        sM[h] = m;
-        sL[h] = sL[h] * c + l;
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) m[x] = fmaxf(m[x], __shfl_xor_sync(0xffffffffu, m[x], o));
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        m[x] = fmaxf(m_old[x], m[x]);
+        e[x] = __float2bfloat16_rn(exp2f((s[x] - m[x]) * 1.4426950408889634f));
+        l[x] = __bfloat162float(e[x]);
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int x = 0; x < 2; ++x) l[x] += __shfl_xor_sync(0xffffffffu, l[x], o);
+      __syncwarp();
+#pragma unroll
+      for (int x = 0; x < 2; ++x) {
+        if (x && !two) break;
+        const int h = h0 + 8 * x;
+        if (lane < KT) sP[h * L.ldp + lane] = e[x];
+        if (lane == 0) {
+          const float c = exp2f((m_old[x] - m[x]) * 1.4426950408889634f);
+          sC[h] = c;
+          sM[h] = m[x];
+          sL[h] = sL[h] * c + l[x];
+        }
       }
     }
-    __syncthreads();
+    if (tile + 1 < n_tiles) arrived();      // also: probabilities are visible
+    else __syncthreads();
+    const __nv_bfloat16* sv = sKV + (tile % p.stages) * L.stage + KT * L.ldk;
 #pragma unroll
     for (int i = 0; i < MAXI; ++i) {
       const int it = warp + i * 8;
       if (it >= items) break;
-      const int j = it / nt8, c = j * p.dv + (it % nt8) * 8, r = lane >> 2;
+      const int j = it / nt8, c = j * p.dv + (it - j * nt8) * 8, r = lane >> 2;
       const float f0 = r < grp ? sC[j * grp + r] : 0.f, f1 = r + 8 < grp ? sC[j * grp + r + 8] : 0.f;
       O[i][0] *= f0; O[i][1] *= f0; O[i][2] *= f1; O[i][3] *= f1;
 #pragma unroll
@@ -197,6 +270,7 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
         mma16816(O[i], a, b);
       }
     }
+    if (tile + 1 < n_tiles) scores(tile + 1);
   }
   __syncthreads();
 #pragma unroll
@@ -248,14 +322,14 @@ using namespace sx;
 // 1 when sx_talk_decode takes these sizes.
 extern "C" int sx_talk_decode_ok(int H, int G, int d, int dv) { return dec_plan(H, G, d, dv).kt > 0; }
 
-template <int KT, int MAXI>
+template <int KT, int MAXI, bool QREG>
 static int launch_dec(const TalkDecParams& p, int n, int smem, cudaStream_t st) {
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(talk_decode_kernel<KT, MAXI>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -10;
+    if (cudaFuncSetAttribute(talk_decode_kernel<KT, MAXI, QREG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -10;
     set = true;
   }
-  talk_decode_kernel<KT, MAXI><<<dim3(n, p.splits), 256, smem, st>>>(p);
+  talk_decode_kernel<KT, MAXI, QREG><<<dim3(n, p.splits), 256, smem, st>>>(p);
   return last_rc();
 }
 
@@ -274,8 +348,11 @@ extern "C" int sx_talk_decode(const SxTalkArgs* a, const void* qmix, int q_ld, c
   p.scale = a->scale; p.mul = a->mul;
   const int smem = dec_layout(a->H, a->G, a->d, a->dv, pl.kt, pl.stages, pl.ksplit).bytes;
   int rc;
-  if (pl.kt == 32) rc = pl.maxi == 8 ? launch_dec<32, 8>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<32, 16>(p, a->T, smem, st) : launch_dec<32, 32>(p, a->T, smem, st);
-  else rc = pl.maxi == 8 ? launch_dec<16, 8>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<16, 16>(p, a->T, smem, st) : launch_dec<16, 32>(p, a->T, smem, st);
+  const int units = (pl.kt / 8) * ((a->H + 15) / 16), ksteps = (a->G * a->d + 15) / 16;
+  const bool qreg = pl.kt == 32 && pl.maxi == 8 && units * pl.ksplit <= 8 && (ksteps + pl.ksplit - 1) / pl.ksplit <= 16;
+  if (qreg) rc = launch_dec<32, 8, true>(p, a->T, smem, st);
+  else if (pl.kt == 32) rc = pl.maxi == 8 ? launch_dec<32, 8, false>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<32, 16, false>(p, a->T, smem, st) : launch_dec<32, 32, false>(p, a->T, smem, st);
+  else rc = pl.maxi == 8 ? launch_dec<16, 8, false>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<16, 16, false>(p, a->T, smem, st) : launch_dec<16, 32, false>(p, a->T, smem, st);
   if (rc == 0 && a->splits > 1) rc = sx_talk_merge(a, st);
   return rc;
 }
