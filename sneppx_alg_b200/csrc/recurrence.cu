@@ -547,6 +547,15 @@ __device__ __forceinline__ void split_frag(const float (&c)[4], uint32_t (&hi)[4
   split_tf32(c[1], hi[2], lo[2]);
   split_tf32(c[3], hi[3], lo[3]);
 }
+// The three products of a split pair in accumulators of their own (short dependency chains), summed by the caller.
+__device__ __forceinline__ void mma_split3(float (&c)[3][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], float b0, float b1) {
+  uint32_t h0, l0, h1, l1;
+  split_tf32(b0, h0, l0);
+  split_tf32(b1, h1, l1);
+  mma_tf32(c[0], ah, h0, h1);
+  mma_tf32(c[1], ah, l0, l1);
+  mma_tf32(c[2], al, h0, h1);
+}
 template <bool A_EXACT>
 __device__ __forceinline__ void mma_split(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], float b0, float b1) {
   uint32_t h0, l0, h1, l1;
@@ -564,7 +573,8 @@ struct TcScanCfg {
   static constexpr int REC = Rec<DP, DELTA>::FLOATS;
   static constexpr int XCH = SPLITD ? 2 * 4 * (1 + DELTA) * 8 * 32 : 0;   // [2][warp][quantity][8 values][lane]
   static constexpr int FIT = (227 * 256 - 16 - XCH) / REC;
-  static constexpr int STAGES = FIT < (SPLITD ? 5 : 3) ? FIT : (SPLITD ? 5 : 3);   // a copy takes longer than a chunk
+  static constexpr int WANT = SPLITD ? 4 : (DELTA ? 2 : 3);   // the larger records leave room for more CTAs with two
+  static constexpr int STAGES = FIT < WANT ? FIT : WANT;
   static constexpr int SMEM = (STAGES * REC + XCH) * 4 + 64;
   static_assert(STAGES >= 2 && SMEM <= 227 * 1024, "shared memory");
 };
@@ -607,16 +617,18 @@ __global__ void __launch_bounds__(128) recur_scan_tc_kernel(const ScanParams p) 
     }
   // values of a chunk in accumulator layout: token 8 n + 2 t + (e & 1), column g + 8 (e >> 1)
   const A* vp = reinterpret_cast<const A*>(p.v) + (long long)h * p.dv;
-  auto load_v = [&](int t0, float (&v)[2][4]) {
+  // (kept as loaded until the next chunk converts them: a conversion here would wait for the load)
+  auto load_v = [&](int t0, A (&v)[2][4]) {
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
         const int tok = t0 + 8 * n + 2 * t + (e & 1), c = c0 + g + (e >> 1) * 8;
-        v[n][e] = (tok < len && c < p.dv) ? to_f(vp[(long long)(row0 + tok) * p.v_ld + c]) : 0.f;
+        v[n][e] = from_f<A>(0.f);
+        if (tok < len && c < p.dv) v[n][e] = vp[(long long)(row0 + tok) * p.v_ld + c];
       }
   };
-  float vn[2][4];
+  A vn[2][4];
   load_v(0, vn);
   __syncthreads();
   for (int ci = 0; ci < n_ch; ++ci) {
@@ -625,29 +637,41 @@ __global__ void __launch_bounds__(128) recur_scan_tc_kernel(const ScanParams p) 
 #pragma unroll
     for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) v[n][e] = vn[n][e];
+      for (int e = 0; e < 4; ++e) v[n][e] = to_f(vn[n][e]);
     if (ci + 1 < n_ch) load_v(t0 + RC, vn);
     if (!mbar_wait_warp(&full[buf], (ci / STAGES) & 1, s_abort, p.status, ST_TIMEOUT_PRODUCER)) break;
     const float* R = sm + buf * REC;
     float q[2][4], w[2][4];
+    {
+      float q3[2][3][4], w3[2][3][4];
 #pragma unroll
-    for (int n = 0; n < 2; ++n)
+      for (int n = 0; n < 2; ++n)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) q[n][e] = w[n][e] = 0.f;
+        for (int x = 0; x < 3; ++x)
 #pragma unroll
-    for (int j = 0; j < ND; ++j) {
-      uint32_t ah[4], al[4];
-      split_frag(S[j], ah, al);
-      const float* base = R + g * RL::LQ + d0 + 8 * j + 2 * t;
+          for (int e = 0; e < 4; ++e) q3[n][x][e] = w3[n][x][e] = 0.f;
 #pragma unroll
-      for (int n = 0; n < 2; ++n) {
-        if constexpr (DELTA) {
-          const float2 b = *reinterpret_cast<const float2*>(base + RL::GK + n * 8 * RL::LQ);
-          mma_split<false>(w[n], ah, al, b.x, b.y);
+      for (int j = 0; j < ND; ++j) {
+        uint32_t ah[4], al[4];
+        split_frag(S[j], ah, al);
+        const float* base = R + g * RL::LQ + d0 + 8 * j + 2 * t;
+#pragma unroll
+        for (int n = 0; n < 2; ++n) {
+          if constexpr (DELTA) {
+            const float2 b = *reinterpret_cast<const float2*>(base + RL::GK + n * 8 * RL::LQ);
+            mma_split3(w3[n], ah, al, b.x, b.y);
+          }
+          const float2 b = *reinterpret_cast<const float2*>(base + n * 8 * RL::LQ);
+          mma_split3(q3[n], ah, al, b.x, b.y);
         }
-        const float2 b = *reinterpret_cast<const float2*>(base + n * 8 * RL::LQ);
-        mma_split<false>(q[n], ah, al, b.x, b.y);
       }
+#pragma unroll
+      for (int n = 0; n < 2; ++n)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          q[n][e] = q3[n][0][e] + (q3[n][1][e] + q3[n][2][e]);
+          w[n][e] = w3[n][0][e] + (w3[n][1][e] + w3[n][2][e]);
+        }
     }
     if constexpr (SPLITD) {
       float* x = xch + (ci & 1) * 4 * (1 + DELTA) * 256;

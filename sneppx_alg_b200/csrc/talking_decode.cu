@@ -45,7 +45,7 @@ __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], 
 
 struct DecLayout {
   int HP, D16, ldq, ldk, ldv, ldp, lds, stage;   // elements (stage: bf16 elements of one K + V tile)
-  int off_k, off_s, off_p, off_m, bytes;         // bytes
+  int off_k, off_s, off_p, off_m, off_i, bytes;         // bytes
 };
 __host__ __device__ inline DecLayout dec_layout(int H, int G, int d, int dv, int KT, int stages, int ksplit) {
   DecLayout L;
@@ -61,7 +61,8 @@ __host__ __device__ inline DecLayout dec_layout(int H, int G, int d, int dv, int
   L.off_s = L.off_k + stages * L.stage * 2;
   L.off_p = L.off_s + ksplit * L.HP * L.lds * 4;
   L.off_m = L.off_p + (L.HP + 16) * L.ldp * 2;
-  L.bytes = L.off_m + 3 * L.HP * 4;
+  L.off_i = L.off_m + 3 * L.HP * 4;
+  L.bytes = L.off_i + G * (dv / 8) * 8;
   return L;
 }
 
@@ -77,6 +78,7 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
   float* sM = reinterpret_cast<float*>(smem + L.off_m);
   float* sL = sM + L.HP;
   float* sC = sL + L.HP;
+  int2* sI = reinterpret_cast<int2*>(smem + L.off_i);   // P V items: first head of the group, value column
   const int n = blockIdx.x, split = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   if (p.rv.slot[n] < 0) return;            // padding row of a captured launch
   const int t = p.rv.cu[n], pos = p.rv.pos0[n];
@@ -88,10 +90,11 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
 
   const int base = p.block_base[n];
   const int* table = p.block_table + (long long)n * p.table_ld;
-  auto fetch = [&](int tile) {
+  const int kc = Gd / 8, vc = Gv / 8;      // 16-byte pieces of a key / value row
+  auto fetch = [&](int tile, int stage) {
     if (tile < n_tiles) {
-      __nv_bfloat16* sk = sKV + (tile % p.stages) * L.stage;
-      __nv_bfloat16* sv = sk + KT * L.ldk;
+      __nv_bfloat16* sk = sKV + stage * L.stage + warp * L.ldk + lane * 8;
+      __nv_bfloat16* sv = sKV + stage * L.stage + KT * L.ldk + warp * L.ldv + lane * 8;
       // rows past the end repeat the last key and are masked; lane i finds the entry of the warp's i-th row
       int e = 0;
       if (lane < KT / 8) {
@@ -101,16 +104,21 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
 #pragma unroll
       for (int i = 0; i < KT / 8; ++i) {
         const long long er = __shfl_sync(0xffffffffu, e, i);
-        const int r = warp + 8 * i;
-        const __nv_bfloat16* kr = p.k + er * Gd;
-        const __nv_bfloat16* vr = p.v + er * Gv;
-        for (int c = lane; c < Gd / 8; c += 32) dec_cp16(sk + r * L.ldk + c * 8, kr + c * 8);
-        for (int c = lane; c < Gv / 8; c += 32) dec_cp16(sv + r * L.ldv + c * 8, vr + c * 8);
+        const __nv_bfloat16* kr = p.k + er * Gd + lane * 8;
+        const __nv_bfloat16* vr = p.v + er * Gv + lane * 8;
+#pragma unroll 4
+        for (int c = 0; c < kc; c += 32)
+          if (c + lane < kc) dec_cp16(sk + c * 8, kr + c * 8);
+#pragma unroll 4
+        for (int c = 0; c < vc; c += 32)
+          if (c + lane < vc) dec_cp16(sv + c * 8, vr + c * 8);
+        sk += 8 * L.ldk;
+        sv += 8 * L.ldv;
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  for (int s = 0; s < p.stages - 1; ++s) fetch(s);
+  for (int s = 0; s < p.stages - 1; ++s) fetch(s, s);
   // queries, zero padding
   const __nv_bfloat16* q = p.qmix + (long long)t * H * p.q_ld;
   for (int i = tid; i < L.HP * (L.D16 / 8); i += 256) {
@@ -130,10 +138,11 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     sL[i] = 0.f;
     sC[i] = 1.f;
   }
+  const int nt8 = p.dv / 8, items = G * nt8, units = (KT / 8) * (L.HP / 16), ksteps = L.D16 / 16;
+  for (int i = tid; i < items; i += 256) sI[i] = make_int2(i / nt8 * grp, i / nt8 * p.dv + i % nt8 * 8);
   float O[MAXI][4];
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) O[i][0] = O[i][1] = O[i][2] = O[i][3] = 0.f;
-  const int nt8 = p.dv / 8, items = G * nt8, units = (KT / 8) * (L.HP / 16), ksteps = L.D16 / 16;
 
   // scores of a tile: (8 keys x 16 heads) units, each cut along k into ksplit parts
   uint32_t qf[QREG ? 16 : 1][4];
@@ -147,30 +156,41 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
         ldsm4(qf[kk], sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8 + (k0 + kk) * 16);
     }
   }
-  auto scores = [&](int tile) {
-    const __nv_bfloat16* sk = sKV + (tile % p.stages) * L.stage;
-    for (int it = warp; it < units * p.ksplit; it += 8) {
-      const int unit = it % units, ks = it / units, n0 = (unit % (KT / 8)) * 8, m0 = unit / (KT / 8) * 16;
-      const int k0 = ksteps * ks / p.ksplit, k1 = ksteps * (ks + 1) / p.ksplit;
-      const __nv_bfloat16* qa = sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8;
+  // item geometry of this warp's first (and with QREG only) item
+  const int it_unit = warp % units, it_ks = warp / units;
+  const int it_n0 = (it_unit % (KT / 8)) * 8, it_m0 = it_unit / (KT / 8) * 16;
+  const int it_k0 = ksteps * it_ks / p.ksplit, it_k1 = ksteps * (it_ks + 1) / p.ksplit, it_nk = it_k1 - it_k0;
+  const int kb_off = (it_n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8 + it_k0 * 16;   // four 8-wide k pieces per load
+  float* s_out = sS + (it_ks * L.HP + it_m0 + (lane >> 2)) * L.lds + it_n0 + (lane & 3) * 2;
+  auto scores = [&](int stage) {
+    const __nv_bfloat16* sk = sKV + stage * L.stage;
+    if constexpr (QREG) {
+      if (it_ks >= p.ksplit) return;
       float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-      const __nv_bfloat16* kb = sk + (n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8;   // four 8-wide k pieces per load
-      if constexpr (QREG) {
+      const __nv_bfloat16* kb = sk + kb_off;
 #pragma unroll
-        for (int kk = 0; kk < 16; kk += 2) {
-          if (k0 + kk + 1 < k1) {
-            uint32_t b[4];
-            ldsm4(b, kb + (k0 + kk) * 16);
-            const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
-            mma16816(c0, qf[kk], b0);
-            mma16816(c1, qf[kk + 1], b1);
-          } else if (k0 + kk < k1) {
-            uint32_t b[2];
-            ldsm2(b, kb + (k0 + kk) * 16);
-            mma16816(c0, qf[kk], b);
-          }
+      for (int kk = 0; kk < 16; kk += 2) {
+        if (kk + 1 < it_nk) {
+          uint32_t b[4];
+          ldsm4(b, kb + kk * 16);
+          const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+          mma16816(c0, qf[kk], b0);
+          mma16816(c1, qf[kk + 1], b1);
+        } else if (kk < it_nk) {
+          uint32_t b[2];
+          ldsm2(b, kb + kk * 16);
+          mma16816(c0, qf[kk], b);
         }
-      } else {
+      }
+      *reinterpret_cast<float2*>(s_out) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+      *reinterpret_cast<float2*>(s_out + 8 * L.lds) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+    } else {
+      for (int it = warp; it < units * p.ksplit; it += 8) {
+        const int unit = it % units, ks = it / units, n0 = (unit % (KT / 8)) * 8, m0 = unit / (KT / 8) * 16;
+        const int k0 = ksteps * ks / p.ksplit, k1 = ksteps * (ks + 1) / p.ksplit;
+        const __nv_bfloat16* qa = sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8;
+        const __nv_bfloat16* kb = sk + (n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8;
+        float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
         int kk = k0;
 #pragma unroll 4
         for (; kk + 1 < k1; kk += 2) {
@@ -188,10 +208,10 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
           ldsm2(b, kb + kk * 16);
           mma16816(c0, a, b);
         }
+        float* s = sS + (ks * L.HP + m0 + (lane >> 2)) * L.lds + n0 + (lane & 3) * 2;
+        *reinterpret_cast<float2*>(s) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
+        *reinterpret_cast<float2*>(s + 8 * L.lds) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
       }
-      float* s = sS + (ks * L.HP + m0 + (lane >> 2)) * L.lds + n0 + (lane & 3) * 2;
-      *reinterpret_cast<float2*>(s) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
-      *reinterpret_cast<float2*>(s + 8 * L.lds) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
     }
   };
   auto arrived = [&]() {
@@ -203,9 +223,12 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     arrived();
     scores(0);
   }
+  int stage = 0, refill = p.stages - 1;
+  const int pv_a = (lane & 15) * L.ldp + (lane >> 4) * 8, pv_b = (lane & 15) * L.ldv, pr = lane >> 2;
   for (int tile = 0; tile < n_tiles; ++tile) {
     __syncthreads();          // scores of this tile are complete, and nobody reads the stage refilled next
-    fetch(tile + p.stages - 1);
+    fetch(tile + p.stages - 1, refill);
+    const int next = stage + 1 == p.stages ? 0 : stage + 1;
     const int nk = min(KT, hi - lo - tile * KT);
     // two heads at a time, so that their reductions overlap
     for (int h0 = warp; h0 < H; h0 += 16) {
@@ -254,23 +277,30 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     }
     if (tile + 1 < n_tiles) arrived();      // also: probabilities are visible
     else __syncthreads();
-    const __nv_bfloat16* sv = sKV + (tile % p.stages) * L.stage + KT * L.ldk;
+    const __nv_bfloat16* sv = sKV + stage * L.stage + KT * L.ldk + pv_b;
 #pragma unroll
     for (int i = 0; i < MAXI; ++i) {
-      const int it = warp + i * 8;
-      if (it >= items) break;
-      const int j = it / nt8, c = j * p.dv + (it - j * nt8) * 8, r = lane >> 2;
-      const float f0 = r < grp ? sC[j * grp + r] : 0.f, f1 = r + 8 < grp ? sC[j * grp + r + 8] : 0.f;
-      O[i][0] *= f0; O[i][1] *= f0; O[i][2] *= f1; O[i][3] *= f1;
+      if (warp + i * 8 >= items) break;
+      const int2 w = sI[warp + i * 8];
+      const float f0 = pr < grp ? sC[w.x + pr] : 0.f;
+      O[i][0] *= f0; O[i][1] *= f0;
+      if (grp > 8) {
+        const float f1 = pr + 8 < grp ? sC[w.x + pr + 8] : 0.f;
+        O[i][2] *= f1; O[i][3] *= f1;
+      }
+      const __nv_bfloat16* pa = sP + w.x * L.ldp + pv_a;
+      const __nv_bfloat16* pb = sv + w.y;
 #pragma unroll
       for (int kk = 0; kk < KT / 16; ++kk) {
         uint32_t a[4], b[2];
-        ldsm4(a, sP + (j * grp + (lane & 15)) * L.ldp + kk * 16 + (lane >> 4) * 8);
-        ldsm2t(b, sv + (kk * 16 + (lane & 15)) * L.ldv + c);
+        ldsm4(a, pa + kk * 16);
+        ldsm2t(b, pb + kk * 16 * L.ldv);
         mma16816(O[i], a, b);
       }
     }
-    if (tile + 1 < n_tiles) scores(tile + 1);
+    if (tile + 1 < n_tiles) scores(next);
+    refill = stage;
+    stage = next;
   }
   __syncthreads();
 #pragma unroll
