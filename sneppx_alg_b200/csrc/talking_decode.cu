@@ -25,23 +25,26 @@ struct TalkDecParams {
   float scale, mul;
 };
 
-__device__ __forceinline__ void dec_cp16(void* dst, const void* src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(dst)), "l"(src) : "memory");
+// shared-memory operands are 32-bit addresses: the inner loops then need no 64-bit address arithmetic
+__device__ __forceinline__ void dec_cp16(uint32_t dst, const void* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory");
 }
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], const void* p) {
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t p) {
   asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(smem_u32(p)) : "memory");
+               : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(p) : "memory");
 }
-__device__ __forceinline__ void ldsm2(uint32_t (&r)[2], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)) : "memory");
+__device__ __forceinline__ void ldsm2(uint32_t (&r)[2], uint32_t p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(p) : "memory");
 }
-__device__ __forceinline__ void ldsm2t(uint32_t (&r)[2], const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(smem_u32(p)) : "memory");
+__device__ __forceinline__ void ldsm2t(uint32_t (&r)[2], uint32_t p) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0, %1}, [%2];" : "=r"(r[0]), "=r"(r[1]) : "r"(p) : "memory");
 }
 __device__ __forceinline__ void mma16816(float (&c)[4], const uint32_t (&a)[4], const uint32_t (&b)[2]) {
   asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
                : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b[0]), "r"(b[1]));
 }
+
+constexpr int DW = 16, DT = DW * 32;     // warps and threads of a CTA
 
 struct DecLayout {
   int HP, D16, ldq, ldk, ldv, ldp, lds, stage;   // elements (stage: bf16 elements of one K + V tile)
@@ -66,9 +69,9 @@ __host__ __device__ inline DecLayout dec_layout(int H, int G, int d, int dv, int
   return L;
 }
 
-// QREG: every warp has one QK item of at most 16 k-steps, whose query fragments then stay in registers.
+// QREG: every warp has one QK item of at most 8 k-steps, whose query fragments then stay in registers.
 template <int KT, int MAXI, bool QREG>
-__global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p) {
+__global__ void __launch_bounds__(DT) talk_decode_kernel(const TalkDecParams p) {
   extern __shared__ __align__(16) uint8_t smem[];
   const DecLayout L = dec_layout(p.H, p.G, p.d, p.dv, KT, p.stages, p.ksplit);
   __nv_bfloat16* sQ = reinterpret_cast<__nv_bfloat16*>(smem);
@@ -91,121 +94,139 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
   const int base = p.block_base[n];
   const int* table = p.block_table + (long long)n * p.table_ld;
   const int kc = Gd / 8, vc = Gv / 8;      // 16-byte pieces of a key / value row
-  auto fetch = [&](int tile, int stage) {
+  const uint32_t a_kv = smem_u32(sKV), stage_bytes = L.stage * 2, ldk_b = L.ldk * 2, ldv_b = L.ldv * 2;
+  const uint32_t a_v = a_kv + KT * ldk_b;
+  // rows past the end repeat the last key and are masked; lane i finds the entry of the warp's i-th row
+  auto entry_of = [&](int tile) -> int {
+    if (lane >= KT / DW || tile >= n_tiles) return 0;
+    const int j = min(lo + tile * KT + warp + DW * lane, hi - 1), b = j / p.block_size;
+    return table[b - base] * p.block_size + j - b * p.block_size;
+  };
+  auto fetch = [&](int tile, int stage, int e) {
     if (tile < n_tiles) {
-      __nv_bfloat16* sk = sKV + stage * L.stage + warp * L.ldk + lane * 8;
-      __nv_bfloat16* sv = sKV + stage * L.stage + KT * L.ldk + warp * L.ldv + lane * 8;
-      // rows past the end repeat the last key and are masked; lane i finds the entry of the warp's i-th row
-      int e = 0;
-      if (lane < KT / 8) {
-        const int j = min(lo + tile * KT + warp + 8 * lane, hi - 1), b = j / p.block_size;
-        e = table[b - base] * p.block_size + j - b * p.block_size;
-      }
+      uint32_t dk = a_kv + stage * stage_bytes + warp * ldk_b + lane * 16, dv = a_v + stage * stage_bytes + warp * ldv_b + lane * 16;
 #pragma unroll
-      for (int i = 0; i < KT / 8; ++i) {
+      for (int i = 0; i < KT / DW; ++i) {
         const long long er = __shfl_sync(0xffffffffu, e, i);
         const __nv_bfloat16* kr = p.k + er * Gd + lane * 8;
         const __nv_bfloat16* vr = p.v + er * Gv + lane * 8;
-#pragma unroll 4
-        for (int c = 0; c < kc; c += 32)
-          if (c + lane < kc) dec_cp16(sk + c * 8, kr + c * 8);
-#pragma unroll 4
-        for (int c = 0; c < vc; c += 32)
-          if (c + lane < vc) dec_cp16(sv + c * 8, vr + c * 8);
-        sk += 8 * L.ldk;
-        sv += 8 * L.ldv;
+        for (int c = 0; c < kc; c += 64) {
+          if (c + lane < kc) dec_cp16(dk + c * 16, kr + c * 8);
+          if (c + 32 + lane < kc) dec_cp16(dk + c * 16 + 512, kr + c * 8 + 256);
+        }
+        for (int c = 0; c < vc; c += 64) {
+          if (c + lane < vc) dec_cp16(dv + c * 16, vr + c * 8);
+          if (c + 32 + lane < vc) dec_cp16(dv + c * 16 + 512, vr + c * 8 + 256);
+        }
+        dk += DW * ldk_b;
+        dv += DW * ldv_b;
       }
     }
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
-  for (int s = 0; s < p.stages - 1; ++s) fetch(s, s);
+  for (int s = 0; s < p.stages - 1; ++s) fetch(s, s, entry_of(s));
+  int e_next = entry_of(p.stages - 1);       // one tile ahead of its use
   // queries, zero padding
   const __nv_bfloat16* q = p.qmix + (long long)t * H * p.q_ld;
-  for (int i = tid; i < L.HP * (L.D16 / 8); i += 256) {
+  for (int i = tid; i < L.HP * (L.D16 / 8); i += DT) {
     const int h = i / (L.D16 / 8), c = i % (L.D16 / 8) * 8;
     uint4 x = make_uint4(0, 0, 0, 0);
     if (h < H) x = *reinterpret_cast<const uint4*>(q + (long long)h * p.q_ld + c);
     *reinterpret_cast<uint4*>(sQ + h * L.ldq + c) = x;
   }
   if (Gd < L.D16)
-    for (int i = tid; i < p.stages * KT * (L.D16 - Gd); i += 256) {
+    for (int i = tid; i < p.stages * KT * (L.D16 - Gd); i += DT) {
       const int w = L.D16 - Gd, s = i / (KT * w), r = i / w % KT;
       sKV[s * L.stage + r * L.ldk + Gd + i % w] = __float2bfloat16_rn(0.f);
     }
-  for (int i = tid; i < (L.HP + 16) * L.ldp; i += 256) sP[i] = __float2bfloat16_rn(0.f);
-  for (int i = tid; i < L.HP; i += 256) {
+  for (int i = tid; i < (L.HP + 16) * L.ldp; i += DT) sP[i] = __float2bfloat16_rn(0.f);
+  for (int i = tid; i < L.HP; i += DT) {
     sM[i] = -INFINITY;
     sL[i] = 0.f;
     sC[i] = 1.f;
   }
   const int nt8 = p.dv / 8, items = G * nt8, units = (KT / 8) * (L.HP / 16), ksteps = L.D16 / 16;
-  for (int i = tid; i < items; i += 256) sI[i] = make_int2(i / nt8 * grp, i / nt8 * p.dv + i % nt8 * 8);
+  for (int i = tid; i < items; i += DT) sI[i] = make_int2(i / nt8 * grp, i / nt8 * p.dv + i % nt8 * 8);
   float O[MAXI][4];
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) O[i][0] = O[i][1] = O[i][2] = O[i][3] = 0.f;
 
   // scores of a tile: (8 keys x 16 heads) units, each cut along k into ksplit parts
-  uint32_t qf[QREG ? 16 : 1][4];
+  uint32_t qf[QREG ? 8 : 1][4];
   if constexpr (QREG) {
     const int unit = warp % units, ks = warp / units, m0 = unit / (KT / 8) * 16, k0 = ksteps * ks / p.ksplit;
     __syncthreads();
 #pragma unroll
-    for (int kk = 0; kk < 16; ++kk) {
+    for (int kk = 0; kk < 8; ++kk) {
       qf[kk][0] = qf[kk][1] = qf[kk][2] = qf[kk][3] = 0;
       if (ks < p.ksplit && k0 + kk < ksteps * (ks + 1) / p.ksplit)
-        ldsm4(qf[kk], sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8 + (k0 + kk) * 16);
+        ldsm4(qf[kk], smem_u32(sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8 + (k0 + kk) * 16));
     }
   }
   // item geometry of this warp's first (and with QREG only) item
   const int it_unit = warp % units, it_ks = warp / units;
   const int it_n0 = (it_unit % (KT / 8)) * 8, it_m0 = it_unit / (KT / 8) * 16;
   const int it_k0 = ksteps * it_ks / p.ksplit, it_k1 = ksteps * (it_ks + 1) / p.ksplit, it_nk = it_k1 - it_k0;
-  const int kb_off = (it_n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8 + it_k0 * 16;   // four 8-wide k pieces per load
+  const uint32_t a_kb = a_kv + ((it_n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8 + it_k0 * 16) * 2;   // four 8-wide k pieces per load
   float* s_out = sS + (it_ks * L.HP + it_m0 + (lane >> 2)) * L.lds + it_n0 + (lane & 3) * 2;
   auto scores = [&](int stage) {
-    const __nv_bfloat16* sk = sKV + stage * L.stage;
     if constexpr (QREG) {
       if (it_ks >= p.ksplit) return;
-      float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
-      const __nv_bfloat16* kb = sk + kb_off;
+      float c[4][4];
 #pragma unroll
-      for (int kk = 0; kk < 16; kk += 2) {
-        if (kk + 1 < it_nk) {
-          uint32_t b[4];
-          ldsm4(b, kb + kk * 16);
-          const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
-          mma16816(c0, qf[kk], b0);
-          mma16816(c1, qf[kk + 1], b1);
-        } else if (kk < it_nk) {
-          uint32_t b[2];
-          ldsm2(b, kb + kk * 16);
-          mma16816(c0, qf[kk], b);
+      for (int i = 0; i < 4; ++i) c[i][0] = c[i][1] = c[i][2] = c[i][3] = 0.f;
+      const uint32_t kb = a_kb + stage * stage_bytes;
+      if (it_nk == 8) {
+        uint32_t b[4][4];                              // loads of all k-steps in flight together
+#pragma unroll
+        for (int i = 0; i < 4; ++i) ldsm4(b[i], kb + i * 64);
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const uint32_t b0[2] = {b[i][0], b[i][1]}, b1[2] = {b[i][2], b[i][3]};
+          mma16816(c[i & 1], qf[2 * i], b0);
+          mma16816(c[2 + (i & 1)], qf[2 * i + 1], b1);
+        }
+      } else {
+#pragma unroll
+        for (int kk = 0; kk < 8; kk += 2) {
+          if (kk + 1 < it_nk) {
+            uint32_t b[4];
+            ldsm4(b, kb + kk * 32);
+            const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
+            mma16816(c[0], qf[kk], b0);
+            mma16816(c[1], qf[kk + 1], b1);
+          } else if (kk < it_nk) {
+            uint32_t b[2];
+            ldsm2(b, kb + kk * 32);
+            mma16816(c[0], qf[kk], b);
+          }
         }
       }
-      *reinterpret_cast<float2*>(s_out) = make_float2(c0[0] + c1[0], c0[1] + c1[1]);
-      *reinterpret_cast<float2*>(s_out + 8 * L.lds) = make_float2(c0[2] + c1[2], c0[3] + c1[3]);
+      *reinterpret_cast<float2*>(s_out) = make_float2((c[0][0] + c[1][0]) + (c[2][0] + c[3][0]), (c[0][1] + c[1][1]) + (c[2][1] + c[3][1]));
+      *reinterpret_cast<float2*>(s_out + 8 * L.lds) =
+          make_float2((c[0][2] + c[1][2]) + (c[2][2] + c[3][2]), (c[0][3] + c[1][3]) + (c[2][3] + c[3][3]));
     } else {
-      for (int it = warp; it < units * p.ksplit; it += 8) {
+      for (int it = warp; it < units * p.ksplit; it += DW) {
         const int unit = it % units, ks = it / units, n0 = (unit % (KT / 8)) * 8, m0 = unit / (KT / 8) * 16;
         const int k0 = ksteps * ks / p.ksplit, k1 = ksteps * (ks + 1) / p.ksplit;
-        const __nv_bfloat16* qa = sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8;
-        const __nv_bfloat16* kb = sk + (n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8;
+        const uint32_t qa = smem_u32(sQ + (m0 + (lane & 15)) * L.ldq + (lane >> 4) * 8);
+        const uint32_t kb = a_kv + stage * stage_bytes + ((n0 + (lane & 7)) * L.ldk + (lane >> 3) * 8) * 2;
         float c0[4] = {0.f, 0.f, 0.f, 0.f}, c1[4] = {0.f, 0.f, 0.f, 0.f};
         int kk = k0;
 #pragma unroll 4
         for (; kk + 1 < k1; kk += 2) {
           uint32_t a[4], a2[4], b[4];
-          ldsm4(a, qa + kk * 16);
-          ldsm4(a2, qa + kk * 16 + 16);
-          ldsm4(b, kb + kk * 16);
+          ldsm4(a, qa + kk * 32);
+          ldsm4(a2, qa + kk * 32 + 32);
+          ldsm4(b, kb + kk * 32);
           const uint32_t b0[2] = {b[0], b[1]}, b1[2] = {b[2], b[3]};
           mma16816(c0, a, b0);
           mma16816(c1, a2, b1);
         }
         if (kk < k1) {
           uint32_t a[4], b[2];
-          ldsm4(a, qa + kk * 16);
-          ldsm2(b, kb + kk * 16);
+          ldsm4(a, qa + kk * 32);
+          ldsm2(b, kb + kk * 32);
           mma16816(c0, a, b);
         }
         float* s = sS + (ks * L.HP + m0 + (lane >> 2)) * L.lds + n0 + (lane & 3) * 2;
@@ -224,20 +245,22 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     scores(0);
   }
   int stage = 0, refill = p.stages - 1;
-  const int pv_a = (lane & 15) * L.ldp + (lane >> 4) * 8, pv_b = (lane & 15) * L.ldv, pr = lane >> 2;
+  const uint32_t pv_a = smem_u32(sP + (lane & 15) * L.ldp + (lane >> 4) * 8), pv_b = a_v + (lane & 15) * ldv_b, ldp_b = L.ldp * 2;
+  const int pr = lane >> 2;
   for (int tile = 0; tile < n_tiles; ++tile) {
     __syncthreads();          // scores of this tile are complete, and nobody reads the stage refilled next
-    fetch(tile + p.stages - 1, refill);
+    fetch(tile + p.stages - 1, refill, e_next);
+    e_next = entry_of(tile + p.stages);
     const int next = stage + 1 == p.stages ? 0 : stage + 1;
     const int nk = min(KT, hi - lo - tile * KT);
     // two heads at a time, so that their reductions overlap
-    for (int h0 = warp; h0 < H; h0 += 16) {
-      const bool two = h0 + 8 < H;
+    for (int h0 = warp; h0 < H; h0 += 2 * DW) {
+      const bool two = h0 + DW < H;
       float s[2], m_old[2], m[2], l[2];
       __nv_bfloat16 e[2];
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
-        const int h = two ? h0 + 8 * x : h0;
+        const int h = two ? h0 + DW * x : h0;
         s[x] = -INFINITY;
         if (lane < nk) {
           s[x] = 0.f;
@@ -265,7 +288,7 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
 #pragma unroll
       for (int x = 0; x < 2; ++x) {
         if (x && !two) break;
-        const int h = h0 + 8 * x;
+        const int h = h0 + DW * x;
         if (lane < KT) sP[h * L.ldp + lane] = e[x];
         if (lane == 0) {
           const float c = exp2f((m_old[x] - m[x]) * 1.4426950408889634f);
@@ -277,25 +300,32 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     }
     if (tile + 1 < n_tiles) arrived();      // also: probabilities are visible
     else __syncthreads();
-    const __nv_bfloat16* sv = sKV + stage * L.stage + KT * L.ldk + pv_b;
+    const uint32_t sv = pv_b + stage * stage_bytes;
 #pragma unroll
-    for (int i = 0; i < MAXI; ++i) {
-      if (warp + i * 8 >= items) break;
-      const int2 w = sI[warp + i * 8];
-      const float f0 = pr < grp ? sC[w.x + pr] : 0.f;
-      O[i][0] *= f0; O[i][1] *= f0;
-      if (grp > 8) {
-        const float f1 = pr + 8 < grp ? sC[w.x + pr + 8] : 0.f;
-        O[i][2] *= f1; O[i][3] *= f1;
-      }
-      const __nv_bfloat16* pa = sP + w.x * L.ldp + pv_a;
-      const __nv_bfloat16* pb = sv + w.y;
+    for (int i0 = 0; i0 < MAXI; i0 += 4) {            // four items together: their loads overlap
+      if (warp + i0 * DW >= items) break;
+      uint32_t a[4][KT / 16][4], b[4][KT / 16][2];
+      int2 w[4];
 #pragma unroll
-      for (int kk = 0; kk < KT / 16; ++kk) {
-        uint32_t a[4], b[2];
-        ldsm4(a, pa + kk * 16);
-        ldsm2t(b, pb + kk * 16 * L.ldv);
-        mma16816(O[i], a, b);
+      for (int i = 0; i < 4; ++i) w[i] = sI[min(warp + (i0 + i) * DW, items - 1)];
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int kk = 0; kk < KT / 16; ++kk) {
+          ldsm4(a[i][kk], pv_a + w[i].x * ldp_b + kk * 32);
+          ldsm2t(b[i][kk], sv + w[i].y * 2 + kk * 16 * ldv_b);
+        }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        if (warp + (i0 + i) * DW >= items) break;
+        const float f0 = pr < grp ? sC[w[i].x + pr] : 0.f;
+        O[i0 + i][0] *= f0; O[i0 + i][1] *= f0;
+        if (grp > 8) {
+          const float f1 = pr + 8 < grp ? sC[w[i].x + pr + 8] : 0.f;
+          O[i0 + i][2] *= f1; O[i0 + i][3] *= f1;
+        }
+#pragma unroll
+        for (int kk = 0; kk < KT / 16; ++kk) mma16816(O[i0 + i], a[i][kk], b[i][kk]);
       }
     }
     if (tile + 1 < n_tiles) scores(next);
@@ -305,7 +335,7 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
   __syncthreads();
 #pragma unroll
   for (int i = 0; i < MAXI; ++i) {
-    const int it = warp + i * 8;
+    const int it = warp + i * DW;
     if (it >= items) break;
     const int j = it / nt8, c = (it % nt8) * 8 + (lane & 3) * 2;
 #pragma unroll
@@ -325,7 +355,7 @@ __global__ void __launch_bounds__(256) talk_decode_kernel(const TalkDecParams p)
     }
   }
   if (p.splits > 1)
-    for (int h = tid; h < H; h += 256) {
+    for (int h = tid; h < H; h += DT) {
       float* o = p.part + (((long long)n * p.splits + split) * H + h) * (p.dv + 2);
       o[0] = sM[h];
       o[1] = sL[h];
@@ -336,12 +366,12 @@ struct DecPlan { int kt, stages, ksplit, maxi; };
 static DecPlan dec_plan(int H, int G, int d, int dv) {
   DecPlan pl{0, 0, 0, 0};
   if (H <= 0 || G <= 0 || H % G || H / G > 16 || (G * d) % 8 || (d % 2) || dv % 8) return pl;
-  const int per_warp = (G * (dv / 8) + 7) / 8;
-  if (per_warp > 32) return pl;
+  const int per_warp = (G * (dv / 8) + DW - 1) / DW;
+  if (per_warp > 16) return pl;
   for (int kt = 32; kt >= 16; kt -= 16)
     for (int stages = 3; stages >= 2; --stages) {
-      const int units = (kt / 8) * ((H + 15) / 16), ks = units >= 8 ? 1 : (units >= 4 ? 2 : 4);
-      if (dec_layout(H, G, d, dv, kt, stages, ks).bytes <= 227 * 1024) return DecPlan{kt, stages, ks, per_warp <= 8 ? 8 : per_warp <= 16 ? 16 : 32};
+      const int units = (kt / 8) * ((H + 15) / 16), ks = units >= 16 ? 1 : (units >= 8 ? 2 : (units >= 4 ? 4 : 8));
+      if (dec_layout(H, G, d, dv, kt, stages, ks).bytes <= 227 * 1024) return DecPlan{kt, stages, ks, per_warp <= 4 ? 4 : per_warp <= 8 ? 8 : 16};
     }
   return pl;
 }
@@ -359,7 +389,7 @@ static int launch_dec(const TalkDecParams& p, int n, int smem, cudaStream_t st) 
     if (cudaFuncSetAttribute(talk_decode_kernel<KT, MAXI, QREG>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -10;
     set = true;
   }
-  talk_decode_kernel<KT, MAXI, QREG><<<dim3(n, p.splits), 256, smem, st>>>(p);
+  talk_decode_kernel<KT, MAXI, QREG><<<dim3(n, p.splits), DT, smem, st>>>(p);
   return last_rc();
 }
 
@@ -379,10 +409,11 @@ extern "C" int sx_talk_decode(const SxTalkArgs* a, const void* qmix, int q_ld, c
   const int smem = dec_layout(a->H, a->G, a->d, a->dv, pl.kt, pl.stages, pl.ksplit).bytes;
   int rc;
   const int units = (pl.kt / 8) * ((a->H + 15) / 16), ksteps = (a->G * a->d + 15) / 16;
-  const bool qreg = pl.kt == 32 && pl.maxi == 8 && units * pl.ksplit <= 8 && (ksteps + pl.ksplit - 1) / pl.ksplit <= 16;
-  if (qreg) rc = launch_dec<32, 8, true>(p, a->T, smem, st);
-  else if (pl.kt == 32) rc = pl.maxi == 8 ? launch_dec<32, 8, false>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<32, 16, false>(p, a->T, smem, st) : launch_dec<32, 32, false>(p, a->T, smem, st);
-  else rc = pl.maxi == 8 ? launch_dec<16, 8, false>(p, a->T, smem, st) : pl.maxi == 16 ? launch_dec<16, 16, false>(p, a->T, smem, st) : launch_dec<16, 32, false>(p, a->T, smem, st);
+  const bool qreg = pl.kt == 32 && pl.maxi == 4 && units * pl.ksplit <= DW && (ksteps + pl.ksplit - 1) / pl.ksplit <= 8;
+  const int n = a->T;
+  if (qreg) rc = launch_dec<32, 4, true>(p, n, smem, st);
+  else if (pl.kt == 32) rc = pl.maxi == 4 ? launch_dec<32, 4, false>(p, n, smem, st) : pl.maxi == 8 ? launch_dec<32, 8, false>(p, n, smem, st) : launch_dec<32, 16, false>(p, n, smem, st);
+  else rc = pl.maxi == 4 ? launch_dec<16, 4, false>(p, n, smem, st) : pl.maxi == 8 ? launch_dec<16, 8, false>(p, n, smem, st) : launch_dec<16, 16, false>(p, n, smem, st);
   if (rc == 0 && a->splits > 1) rc = sx_talk_merge(a, st);
   return rc;
 }
