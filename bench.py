@@ -7,6 +7,7 @@ seq 4096, micro-batch 1 per GPU, AdamW beta 0.9/0.95 wd 0.1), synthetic token id
     python bench.py --impl library ...                      # PyTorch library ops + NCCL only, overlapped like FSDP
     python bench.py --model deepseek-v2-lite --ep --micro-batch 2      # SER MoE, expert parallel + ZeRO-1
     python bench.py --model mamba2-2.7b --seq 8192 --tp 2              # Mamba-2, tensor parallel x data parallel
+    python bench.py --serve-hybrid                                     # serving: Rilenex beside Llama and Mamba-2 at equal size
 
 Rank 0 prints one JSON line. ``value`` is whole-job tokens/s from CUDA-event timing (max over ranks);
 ``e2e`` repeats the measurement through the public engine API with the per-step host->device copy of the
@@ -46,6 +47,8 @@ def parse():
                     "fp8 (e4m3 data, 1x128 activation and 128x128 weight scales); backward stays bf16")
     ap.add_argument("--tp", type=int, default=1, help="tensor-parallel size (Mamba-2 models): ranks form world/tp "
                     "data-parallel replicas of tp consecutive ranks; ignored on one GPU")
+    ap.add_argument("--serve-hybrid", action="store_true", help="instead of the training step: prefill and decode throughput of "
+                    "the Rilenex design beside the closest existing models at equal size, and its kernels beside theirs")
     return ap.parse_args()
 
 
@@ -279,12 +282,26 @@ def run_library(args):
     return 0
 
 
+def run_serve_hybrid(args):
+    """One GPU: a JSON line per measurement, then one with all of them and the clocks seen meanwhile."""
+    from sneppx_alg_b200.benchmarks import hybrid_serving
+    from sneppx_alg_b200.ops import _lib
+    clocks = ClockSampler(int(os.environ.get("LOCAL_RANK", "0")))
+    clocks.start()
+    out = hybrid_serving.main(["--steps", str(max(args.steps, 3))])
+    print(json.dumps({"metric": "serving throughput, Rilenex beside existing models", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
+                      "gpu_launches": _lib.launch_count, "clocks": clocks.stop(), **out}))
+    return 0
+
+
 def main():
     args = parse()
     if args.impl == "reference":
         return run_reference(args)
     if args.impl == "library":
         return run_library(args)
+    if args.serve_hybrid:
+        return run_serve_hybrid(args)
 
     import torch
     import torch.distributed as dist
