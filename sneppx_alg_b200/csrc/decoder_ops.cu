@@ -164,10 +164,12 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(const QkvParams p) {
   const A* u = reinterpret_cast<const A*>(p.u) + (long long)row0 * p.u_ld;
   A* ring = reinterpret_cast<A*>(p.ring) + (long long)slot * p.taps * C;
   for (int i = tid; i < NT * (p.rot / 2); i += 256) {
-    double a = (double)(pos + i / (p.rot / 2)) * p.inv_freq[i % (p.rot / 2)];
+    const int t = i / (p.rot / 2);
+    double a = (double)(pos + t) * p.inv_freq[i - t * (p.rot / 2)];
     a -= 6.283185307179586476925286766559 * rint(a * 0.15915494309189533576888376337251);
     float s, c;
-    sincosf((float)a, &s, &c);
+    if (sizeof(A) == 4) sincosf((float)a, &s, &c);
+    else __sincosf((float)a, &s, &c);       // |a| <= pi: within 2^-21 there
     cs[i] = c;
     sn[i] = s;
   }
@@ -197,8 +199,11 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(const QkvParams p) {
   }
   __syncthreads();
   // one warp per head row: RMS norm and rotation of the pairs (2i, 2i + 1)
-  for (int it = warp; it < NT * nh; it += 8) {
-    const int t = it / nh, hh = it % nh;
+  for (int t = 0, hh = warp; t < nt; hh += 8) {
+    while (hh >= nh) {
+      hh -= nh;
+      ++t;
+    }
     if (t >= nt) break;
     float* x = sh + t * nqk + hh * d;
     float ss = 0.f;
@@ -236,6 +241,33 @@ __global__ void __launch_bounds__(256) qkv_prep_kernel(const QkvParams p) {
   __syncthreads();
   A* out = reinterpret_cast<A*>(p.qmix_out) + (long long)row0 * p.H * p.qmix_ld;
   const int half = d / 2;
+  if (NT >= 4 && grp == 4 && half <= 256 && 256 % half == 0) {
+    // a thread keeps one pair of channels of up to four tokens: the mix weights of a head are read once for all of them
+    const int e = tid % half, step = 256 / half;
+    for (int t0 = tid / half; t0 < nt; t0 += 4 * step) {
+      float2 q[4][4];
+#pragma unroll
+      for (int x = 0; x < 4; ++x)
+#pragma unroll
+        for (int g = 0; g < 4; ++g) {
+          const int t = t0 + x * step;
+          q[x][g] = t < nt ? *reinterpret_cast<const float2*>(sh + t * nqk + g * d + 2 * e) : make_float2(0.f, 0.f);
+        }
+      A* o = out + (long long)t0 * p.H * p.qmix_ld + j * d + 2 * e;
+      const long long tstep = (long long)step * p.H * p.qmix_ld;
+      const bool all = t0 + 3 * step < nt;
+#pragma unroll 2
+      for (int h = 0; h < p.H; ++h, o += p.qmix_ld) {
+        const float w0 = st[h * 4], w1 = st[h * 4 + 1], w2 = st[h * 4 + 2], w3 = st[h * 4 + 3];
+#pragma unroll
+        for (int x = 0; x < 4; ++x) {
+          const float a = fmaf(w0, q[x][0].x, fmaf(w1, q[x][1].x, fmaf(w2, q[x][2].x, w3 * q[x][3].x)));
+          const float b = fmaf(w0, q[x][0].y, fmaf(w1, q[x][1].y, fmaf(w2, q[x][2].y, w3 * q[x][3].y)));
+          if (all || t0 + x * step < nt) store2(o + x * tstep, a, b);
+        }
+      }
+    }
+  } else
   for (int i = tid; i < nt * half; i += 256) {
     const int t = i / half, e = i % half;
     const float* x = sh + t * nqk + 2 * e;

@@ -52,18 +52,27 @@ __device__ __forceinline__ void conv_walk(const A* __restrict__ u, long long ld,
   float x[NT + MT - 1], wb[MT];
 #pragma unroll
   for (int b = 0; b < MT; ++b) wb[b] = b < taps ? w[(long long)(taps - 1 - b) * C + ch] : 0.f;
-  const int ph = pos % taps;
+  if (NT > 1 && s0 >= MT - 1 && nt == NT) {     // inside a portion: every row is there
+    const A* r = u + ch - (MT - 1) * ld;
+    A raw[NT + MT - 1];
 #pragma unroll
-  for (int i = 0; i < NT + MT - 1; ++i) {
-    const int t = i - (MT - 1);          // token relative to the first one
-    x[i] = 0.f;
-    if (t < 0) {
-      if (-t < taps) {
-        if (s0 + t >= 0) x[i] = to_f(u[(long long)t * ld + ch]);
-        else if (pos + t >= 0) x[i] = to_f(ring[(long long)(ph + t >= 0 ? ph + t : ph + t + taps) * C + ch]);
+    for (int i = 0; i < NT + MT - 1; ++i, r += ld) raw[i] = *r;
+#pragma unroll
+    for (int i = 0; i < NT + MT - 1; ++i) x[i] = to_f(raw[i]);
+  } else {
+    const int ph = pos % taps;
+#pragma unroll
+    for (int i = 0; i < NT + MT - 1; ++i) {
+      const int t = i - (MT - 1);          // token relative to the first one
+      x[i] = 0.f;
+      if (t < 0) {
+        if (-t < taps) {
+          if (s0 + t >= 0) x[i] = to_f(u[(long long)t * ld + ch]);
+          else if (pos + t >= 0) x[i] = to_f(ring[(long long)(ph + t >= 0 ? ph + t : ph + t + taps) * C + ch]);
+        }
+      } else if (t < nt) {
+        x[i] = to_f(u[(long long)t * ld + ch]);
       }
-    } else if (t < nt) {
-      x[i] = to_f(u[(long long)t * ld + ch]);
     }
   }
 #pragma unroll
