@@ -148,7 +148,7 @@ struct QkvParams {
 // One CTA: NT rows of one portion (a chunk of a prompt, or the one row of a decode step) for one key head with its query
 // heads and value head. A thread walks a channel through the rows; heads are then normed and rotated in shared memory.
 template <typename A, int NT, int MT>
-__global__ void __launch_bounds__(256) qkv_prep_kernel(const QkvParams p) {
+__global__ void __launch_bounds__(256, MT <= 4 ? 3 : 1) qkv_prep_kernel(const QkvParams p) {
   extern __shared__ __align__(16) float sm[];
   const int grp = p.H / p.G, nh = grp + 1, d = p.d, j = blockIdx.y;
   float* cs = sm;                    // [NT, rot/2] cos

@@ -8,6 +8,7 @@ import hashlib
 from collections import OrderedDict
 from typing import Dict, List, Optional, Tuple
 
+import numpy as np
 import torch
 
 
@@ -242,22 +243,19 @@ class ChunkedKVCache(PagedKVCache):
             base += 1
         if not table:
             base = max(base, new_base)
-        entries = []
-        for p in range(n, end):
-            if p < keep:
-                entries.append(-1)
-                continue
-            bi = p // self.block_size - base
-            if bi == len(table):
-                table.append(self.pool.allocate())
-            entries.append(table[bi] * self.block_size + p % self.block_size)
+        while base + len(table) <= (end - 1) // self.block_size:
+            table.append(self.pool.allocate())
         self.base[seq_id], self.lens[seq_id] = base, end
-        return entries
+        first = max(n, keep)
+        return [-1] * (first - n) + self.entries(seq_id, first, end)
 
     def entries(self, seq_id: int, lo: int, hi: int) -> List[int]:
         """Entries of the stored positions [lo, hi)."""
         table, base, bs = self.tables[seq_id], self.base[seq_id], self.block_size
-        return [table[p // bs - base] * bs + p % bs for p in range(lo, hi)]
+        if hi - lo == 1:
+            return [table[lo // bs - base] * bs + lo % bs]
+        p = np.arange(lo, hi)
+        return (np.asarray(table, dtype=np.int64)[p // bs - base] * bs + p % bs).tolist() if hi > lo else []
 
     def fork(self, src_id: int, dst_id: int) -> None:
         raise NotImplementedError("a chunked cache does not share blocks between sequences")

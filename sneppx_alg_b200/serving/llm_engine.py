@@ -465,9 +465,10 @@ class LLMEngine:
             self.running.pop(req.req_id, None)
             self.finished[req.req_id] = req
 
-    def _admit_same_length(self, first: "Request", budget: int) -> List["Request"]:
+    def _admit_same_pass(self, first: "Request", budget: int) -> List["Request"]:
         """Pops the waiting requests that can join ``first``'s prefill pass: they are next in queue order, have a
-        prompt of the same length (any length when the runner packs ragged prompts), hit no cached prefix, fit the batch, the token budget and the block pool."""
+        prompt of the same length (any length when the runner packs ragged prompts), hit no cached prefix, fit the batch,
+        the token budget and the block pool."""
         out, T = [], len(first.prompt)
         ragged = getattr(self.runner, "ragged_prefill", False)
         reserved = self._blocks_needed(first)
@@ -509,7 +510,7 @@ class LLMEngine:
             group = [req]
             if cached == 0 and hasattr(self.runner, "prefill_batch"):
                 # requests behind it with a prompt of the same length (and nothing cached) share the pass
-                group += self._admit_same_length(req, budget - len(req.prompt))
+                group += self._admit_same_pass(req, budget - len(req.prompt))
             if len(group) > 1:
                 logits = self.runner.prefill_batch([g.req_id for g in group], [g.prompt for g in group])
                 picks = logits.argmax(dim=-1).tolist() if any(self._plain_greedy(g) for g in group) else None
