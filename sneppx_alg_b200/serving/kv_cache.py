@@ -243,10 +243,10 @@ class ChunkedKVCache(PagedKVCache):
             base += 1
         if not table:
             base = max(base, new_base)
-        while base + len(table) <= (end - 1) // self.block_size:
+        first = max(n, keep)
+        while first < end and base + len(table) <= (end - 1) // self.block_size:   # first == end: no layer keeps keys
             table.append(self.pool.allocate())
         self.base[seq_id], self.lens[seq_id] = base, end
-        first = max(n, keep)
         return [-1] * (first - n) + self.entries(seq_id, first, end)
 
     def entries(self, seq_id: int, lo: int, hi: int) -> List[int]:

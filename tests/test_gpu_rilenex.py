@@ -374,6 +374,25 @@ def test_long_decoding(name, dtype):
     assert len(r.cache.tables[0]) <= r.cache.table_width
 
 
+@pytest.mark.parametrize("dtype", [F32, BF16])
+def test_model_of_recurrent_layers_only(dtype):
+    cfg = config(56, 70, [hgrn2(2, 24, 16, 48), hgrn2(4, 16, 10, None)])
+    W = make_weights(cfg, 4)
+    model = make_model(cfg, W, dtype, "cuda")
+    seqs = [toks(n, 70, seed=n) for n in (45, 20)]
+    want = [oracle.forward(cfg, W, s) for s in seqs]
+    r = new_runner(model, n=2, graphs=True)
+    for i in range(2):
+        r.cache.add_sequence(i)
+    close(r.step([(i, seqs[i][:17], range(17)) for i in range(2)]), torch.cat([w[:17] for w in want]), dtype)
+    for k in range(17, 20):
+        close(r.step([(i, [seqs[i][k]], (0,)) for i in range(2)]), torch.stack([w[k] for w in want]), dtype)
+    prompt = seqs[1][:5]
+    eng = LLMEngine(model, max_batch_size=2)
+    got = eng.generate([prompt, prompt], SamplingParams(max_new_tokens=4))
+    assert got[0] == got[1] and (dtype == BF16 or got[0] == greedy(cfg, W, prompt, 4))
+
+
 def test_results_do_not_depend_on_company_or_place():
     """Same sequence alone, in a batch, in another slot and other blocks: differences are rounding only."""
     model, _ = model_of("tensor", F32)

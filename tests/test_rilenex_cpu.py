@@ -127,6 +127,15 @@ def test_chunked_cache_keeps_exactly_the_visible_positions(sizes, bs):
     assert cache.pool.num_free == 64
 
 
+def test_cache_without_attention_layers_uses_no_blocks():
+    cache = ChunkedKVCache([], [], 1, 16, dtype=torch.float32, device="cpu")
+    for seq in range(3):
+        cache.add_sequence(seq)
+        for n in (1, 15, 16, 40, 1):
+            assert cache.reserve(seq, n) == [-1] * n
+    assert cache.pool.num_free == 1 and cache.table_width == 0 and cache.blocks_for(100) == 0
+
+
 def test_slots_are_handed_back():
     model = make_model(ODD, make_weights(ODD))
     cache = model.init_cache(2)
