@@ -35,12 +35,12 @@ NVCC_FLAGS = [
 ]
 # Sources whose arithmetic follows IEEE single precision (no approximate division / square root / exponential, no
 # flush of denormals): recurrent state and the paths that also run models in 32-bit.
-PRECISE_SOURCES = {"decoder_ops.cu", "recurrence.cu", "talking_attn.cu"}
+PRECISE_SOURCES = {"decoder_ops.cu", "recurrence.cu", "ssd_serve.cu", "talking_attn.cu", "window_attn.cu"}
 
 # Named subsets of the sources for programs that need only part of the library; each is linked on its own.
 CUDA_SUBSETS = {
     "hybrid": ("decoder_ops.cu", "recurrence.cu", "talking_attn.cu", "talking_attn_tc.cu", "talking_decode.cu",
-               "gemm_tc.cu", "gemm_skinny.cu"),
+               "ssd_serve.cu", "ssd_scan.cu", "window_attn.cu", "window_attn_tc.cu", "window_decode.cu", "gemm_tc.cu", "gemm_skinny.cu"),
 }
 
 CXX_FLAGS = ["-O2", "-std=c++17", "-fPIC", "-pthread", "-Wall", "-Wno-unused-function"]

@@ -143,7 +143,7 @@ def bench_kernels(steps, B=8, T=2048, NB=64, ctx=2000):
     ug, up = torch.randn(rows, gate.in_proj.shape[0], **bf), torch.randn(rows, par.in_proj.shape[0], **bf)
     y = torch.empty(rows, par.out_proj.shape[1], **bf)
     with torch.no_grad():
-        add("rmsnorm, fp32 residual in", _time(lambda: hybrid.rmsnorm_f32(x, model.norm, 1e-5, torch.bfloat16), it), rows * w * 6)
+        add("rmsnorm, fp32 residual in", _time(lambda: hybrid.rmsnorm_f32(x, model.norm.weight, 1e-5, torch.bfloat16), it), rows * w * 6)
         xb, wb = torch.randn(rows, w, **bf), torch.ones(w, **bf)
         add("like: rmsnorm + residual (bf16)", _time(lambda: F.rmsnorm(xb, wb, 1e-5, residual=xb), it), rows * w * 8)
 

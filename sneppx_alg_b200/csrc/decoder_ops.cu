@@ -12,10 +12,10 @@ namespace sx {
 
 // ------------------------------------------------------------------ embedding
 template <typename A>
-__global__ void embed_f32_kernel(const A* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x, int width) {
+__global__ void embed_f32_kernel(const A* __restrict__ table, const int* __restrict__ ids, float* __restrict__ x, int width, float scale) {
   const A* src = table + (long long)ids[blockIdx.x] * width;
   float* dst = x + (long long)blockIdx.x * width;
-  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = to_f(src[i]);
+  for (int i = threadIdx.x; i < width; i += blockDim.x) dst[i] = to_f(src[i]) * scale;
 }
 
 // ------------------------------------------------------------------ RMSNorm of fp32 rows
@@ -65,6 +65,114 @@ __global__ void __launch_bounds__(256) rmsnorm_f32_kernel(const float* __restric
     ss = block_sum(ss, red);
     const float r = 1.f / sqrtf(ss / width + eps);
     for (int i = threadIdx.x; i < width; i += 256) yr[i] = from_f<A>(xr[i] * r * w[i]);
+  }
+}
+
+// ------------------------------------------------------------------ layer norm of fp32 rows
+// y = (x - mean) / sqrt(mean of squared deviations + eps) * w + b. Rows as in the RMSNorm; up to 4096 entries of a row stay in
+// registers between the passes.
+template <typename A>
+__global__ void __launch_bounds__(256) layernorm_f32_kernel(const float* __restrict__ x, const float* __restrict__ w,
+                                                            const float* __restrict__ b, const int* __restrict__ rows,
+                                                            A* __restrict__ y, int width, float eps) {
+  __shared__ float red[40];
+  const long long src = rows ? rows[blockIdx.x] : blockIdx.x;
+  const float* xr = x + src * width;
+  A* yr = y + (long long)blockIdx.x * width;
+  if ((width & 3) == 0) {
+    const float4* x4 = reinterpret_cast<const float4*>(xr);
+    const float4* w4 = reinterpret_cast<const float4*>(w);
+    const float4* b4 = reinterpret_cast<const float4*>(b);
+    const int n4 = width / 4;
+    float4 keep[4];
+    float s = 0.f;
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = threadIdx.x + k * 256;
+      keep[k] = i < n4 ? x4[i] : make_float4(0.f, 0.f, 0.f, 0.f);
+      s += (keep[k].x + keep[k].y) + (keep[k].z + keep[k].w);
+    }
+    for (int i = threadIdx.x + 1024; i < n4; i += 256) {
+      const float4 v = x4[i];
+      s += (v.x + v.y) + (v.z + v.w);
+    }
+    const float m = block_sum(s, red) / width;
+    float ss = 0.f;
+    auto dev = [&](const float4& v) {
+      const float a = v.x - m, c = v.y - m, d = v.z - m, e = v.w - m;
+      ss += (a * a + c * c) + (d * d + e * e);
+    };
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (threadIdx.x + k * 256 < n4) dev(keep[k]);
+    for (int i = threadIdx.x + 1024; i < n4; i += 256) dev(x4[i]);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / width + eps);
+    auto put = [&](int i, const float4& v) {
+      const float4 g = w4[i], o = b4[i];
+      store4(yr + 4 * i, fmaf((v.x - m) * r, g.x, o.x), fmaf((v.y - m) * r, g.y, o.y), fmaf((v.z - m) * r, g.z, o.z),
+             fmaf((v.w - m) * r, g.w, o.w));
+    };
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (threadIdx.x + k * 256 < n4) put(threadIdx.x + k * 256, keep[k]);
+    for (int i = threadIdx.x + 1024; i < n4; i += 256) put(i, x4[i]);
+  } else {
+    float s = 0.f, ss = 0.f;
+    for (int i = threadIdx.x; i < width; i += 256) s += xr[i];
+    const float m = block_sum(s, red) / width;
+    for (int i = threadIdx.x; i < width; i += 256) ss += (xr[i] - m) * (xr[i] - m);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / width + eps);
+    for (int i = threadIdx.x; i < width; i += 256) yr[i] = from_f<A>(fmaf((xr[i] - m) * r, w[i], b[i]));
+  }
+}
+
+// ------------------------------------------------------------------ RMSNorm of equal parts of activation rows, in place
+// One CTA per (row, part). VEC: parts, pitch and base allow 16-byte pieces; up to 4 pieces per thread stay in registers.
+template <typename A, bool VEC>
+__global__ void __launch_bounds__(256) part_rmsnorm_kernel(A* __restrict__ y, long long ld, const float* __restrict__ w, int part, float eps) {
+  __shared__ float red[40];
+  A* yr = y + (long long)blockIdx.x * ld + (long long)blockIdx.y * part;
+  const float* wr = w + (long long)blockIdx.y * part;
+  const int n = blockDim.x;
+  float ss = 0.f;
+  if constexpr (VEC) {
+    constexpr int E = 16 / sizeof(A);
+    const int pieces = part / E;
+    uint4 keep[4];
+    auto sum = [&](const uint4& v) {
+      const A* a = reinterpret_cast<const A*>(&v);
+#pragma unroll
+      for (int e = 0; e < E; ++e) ss = fmaf(to_f(a[e]), to_f(a[e]), ss);
+    };
+#pragma unroll
+    for (int k = 0; k < 4; ++k) {
+      const int i = threadIdx.x + k * n;
+      if (i < pieces) {
+        keep[k] = reinterpret_cast<const uint4*>(yr)[i];
+        sum(keep[k]);
+      }
+    }
+    for (int i = threadIdx.x + 4 * n; i < pieces; i += n) sum(reinterpret_cast<const uint4*>(yr)[i]);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / part + eps);
+    auto put = [&](int i, const uint4& v) {
+      const A* a = reinterpret_cast<const A*>(&v);
+#pragma unroll
+      for (int e = 0; e < E; e += 4) {
+        const float4 g = *reinterpret_cast<const float4*>(wr + i * E + e);
+        store4(yr + i * E + e, to_f(a[e]) * r * g.x, to_f(a[e + 1]) * r * g.y, to_f(a[e + 2]) * r * g.z, to_f(a[e + 3]) * r * g.w);
+      }
+    };
+#pragma unroll
+    for (int k = 0; k < 4; ++k)
+      if (threadIdx.x + k * n < pieces) put(threadIdx.x + k * n, keep[k]);
+    for (int i = threadIdx.x + 4 * n; i < pieces; i += n) {
+      const uint4 v = reinterpret_cast<const uint4*>(yr)[i];
+      put(i, v);
+    }
+  } else {
+    for (int i = threadIdx.x; i < part; i += n) ss = fmaf(to_f(yr[i]), to_f(yr[i]), ss);
+    const float r = 1.f / sqrtf(block_sum(ss, red) / part + eps);
+    for (int i = threadIdx.x; i < part; i += n) yr[i] = from_f<A>(to_f(yr[i]) * r * wr[i]);
   }
 }
 
@@ -319,15 +427,34 @@ __global__ void kv_gather_kernel(const A* __restrict__ cache, const int* __restr
 using namespace sx;
 
 
-extern "C" int sx_embed_f32(const void* table, const int* ids, float* x, int T, int width, int f32, cudaStream_t st) {
+extern "C" int sx_embed_f32(const void* table, const int* ids, float* x, int T, int width, float scale, int f32, cudaStream_t st) {
   if (T <= 0) return 0;
-  SX_ACT_DISPATCH(f32, (embed_f32_kernel<A><<<T, 256, 0, st>>>((const A*)table, ids, x, width)));
+  SX_ACT_DISPATCH(f32, (embed_f32_kernel<A><<<T, 256, 0, st>>>((const A*)table, ids, x, width, scale)));
   return last_rc();
 }
 extern "C" int sx_rmsnorm_f32(const float* x, const float* w, const int* rows, void* y, int T, int width, float eps, int f32,
                               cudaStream_t st) {
   if (T <= 0) return 0;
   SX_ACT_DISPATCH(f32, (rmsnorm_f32_kernel<A><<<T, 256, 0, st>>>(x, w, rows, (A*)y, width, eps)));
+  return last_rc();
+}
+extern "C" int sx_layernorm_f32(const float* x, const float* w, const float* b, const int* rows, void* y, int T, int width, float eps,
+                                int f32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  SX_ACT_DISPATCH(f32, (layernorm_f32_kernel<A><<<T, 256, 0, st>>>(x, w, b, rows, (A*)y, width, eps)));
+  return last_rc();
+}
+extern "C" int sx_part_rmsnorm(void* y, long long ld, const float* w, int T, int width, int parts, float eps, int f32, cudaStream_t st) {
+  if (T <= 0) return 0;
+  if (parts <= 0 || parts > 65535 || width % parts) return -1;
+  const int part = width / parts, E = f32 ? 4 : 8;
+  const bool vec = part % E == 0 && ld % E == 0 && (reinterpret_cast<uintptr_t>(y) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
+  const int threads = part >= 2048 ? 256 : part >= 512 ? 128 : 32;
+  const dim3 grid(T, parts);
+  SX_ACT_DISPATCH(f32, {
+    if (vec) part_rmsnorm_kernel<A, true><<<grid, threads, 0, st>>>((A*)y, ld, w, part, eps);
+    else part_rmsnorm_kernel<A, false><<<grid, threads, 0, st>>>((A*)y, ld, w, part, eps);
+  });
   return last_rc();
 }
 extern "C" int sx_head_norm_gate(const float* o, const float* w, const void* gate, long long gate_ld, float mul, void* y,

@@ -75,6 +75,8 @@ __device__ __forceinline__ float skinny_epilogue(float v, const SkinnyParams& p,
   else if (p.act == 2) v = silu(v);
   else if (p.act == 3) v = fmaxf(v, 0.f);
   else if (p.act == 4) v = xielu(v, p.act_a, p.act_b);
+  else if (p.act == 5) v = squared_relu(v);
+  else if (p.act == 6) v = softcap(v, p.act_a, p.act_b);
   return v;
 }
 __device__ __forceinline__ void skinny_store(const SkinnyParams& p, int m, int n, float v) {

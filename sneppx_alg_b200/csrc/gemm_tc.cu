@@ -521,6 +521,12 @@ __global__ void __launch_bounds__(GEMM_THREADS, 1) gemm_tc_kernel(const __grid_c
         } else if (p.act == 4) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = xielu(v[j], p.act_a, p.act_b);
+        } else if (p.act == 5) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = squared_relu(v[j]);
+        } else if (p.act == 6) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = softcap(v[j], p.act_a, p.act_b);
         }
         if (COMM == 2) {
           // this lane's 64 bytes of the row go to the warp's slab: 16-byte chunk index XOR row keeps both the writes
@@ -928,6 +934,12 @@ __global__ void __cluster_dims__(2, 1, 1) __launch_bounds__(GEMM_THREADS, 1)
         } else if (p.act == 4) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) v[j] = xielu(v[j], p.act_a, p.act_b);
+        } else if (p.act == 5) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = squared_relu(v[j]);
+        } else if (p.act == 6) {
+#pragma unroll
+          for (int j = 0; j < 32; ++j) v[j] = softcap(v[j], p.act_a, p.act_b);
         }
         if (p.out_fp32) {
           float* dp = reinterpret_cast<float*>(p.D) + drow + col0;

@@ -1,5 +1,7 @@
 // Gated linear recurrences with an fp32 state per head, S [d, dv]:
 //   gated write   S <- f S + (1 - f) v^T                               o = S^T q        (decay f per row)
+//   SSD           S <- a S + dt B x^T                                  o = S^T C        (one decay a per head; prompts of
+//                                                                       32-bit runs, the other forms are in ssd_serve.cu)
 //   gated delta   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;     o = S^T q        (decay g per row)
 // Operand preparation, the scan over a portion of a prompt, and the one-token step of decoding. The state stays in fp32
 // and every term that enters it is computed in fp32; a portion may start from any stored state, so a prompt can be cut
@@ -173,6 +175,37 @@ __global__ void __launch_bounds__(256) gate_chunk_kernel(const A* __restrict__ q
     sq[i] = q;
     sg[i] = f;
     sk[i] = 1.f - f;       // 0 on padding
+  }
+  __syncthreads();
+  write_record<DP, false>(sq, sk, sg, nullptr, nullptr, rec + ((long long)ch * H + h) * Rec<DP, false>::FLOATS, nt);
+}
+
+// SSD records from the operands of sx_ssd_operands: q = C, k = dt B, one decay for all rows of a head's state.
+template <typename A, int DP>
+__global__ void __launch_bounds__(256) ssd_chunk_kernel(const A* __restrict__ b, const A* __restrict__ c, const float* __restrict__ dt,
+                                                        const float* __restrict__ la, float* __restrict__ rec, const RaggedView rv,
+                                                        const ChunkView cv, int H, int G, int N, int np) {
+  extern __shared__ __align__(128) float sm[];
+  float* sq = sm;
+  float* sk = sq + RC * DP;
+  float* sg = sk + RC * DP;
+  const int ch = blockIdx.x, h = blockIdx.y, seq = cv.seq[ch], s0 = cv.start[ch];
+  const int row0 = rv.cu[seq] + s0, nt = min(RC, rv.cu[seq + 1] - row0), g = h / (H / G);
+  for (int i = threadIdx.x; i < RC * DP; i += 256) {
+    const int t = i / DP, n = i % DP;
+    float q = 0.f, k = 0.f, f = 1.f;
+    if (t < nt) {
+      const long long th = (long long)(row0 + t) * H + h;
+      f = expf(la[th]);
+      if (n < N) {
+        const long long o = ((long long)(row0 + t) * G + g) * np + n;
+        q = to_f(c[o]);
+        k = to_f(b[o]) * dt[th];
+      }
+    }
+    sq[i] = q;
+    sk[i] = k;
+    sg[i] = f;
   }
   __syncthreads();
   write_record<DP, false>(sq, sk, sg, nullptr, nullptr, rec + ((long long)ch * H + h) * Rec<DP, false>::FLOATS, nt);
@@ -1000,6 +1033,31 @@ extern "C" int sx_gate_chunks(const SxGateArgs* a, cudaStream_t st) {
       case 64: return launch_gate_chunks<A, 64>(a, st);
       case 128: return launch_gate_chunks<A, 128>(a, st);
       default: return launch_gate_chunks<A, 256>(a, st);
+    }
+  });
+  return 0;
+}
+
+template <typename A, int DP>
+static int launch_ssd_chunks(const SxSsdArgs* a, float* rec, cudaStream_t st) {
+  static bool set = false;
+  const int smem = 3 * RC * DP * 4;
+  if (int rc = allow_smem(ssd_chunk_kernel<A, DP>, smem, &set)) return rc;
+  ssd_chunk_kernel<A, DP><<<dim3(a->chunks.n, a->H), 256, smem, st>>>((const A*)a->b, (const A*)a->c, a->dt, a->la, rec, view(&a->ragged),
+                                                                      chunks(&a->chunks), a->H, a->G, a->N, a->np);
+  return last_rc();
+}
+
+// Records of the SSD recurrence from its operands.
+extern "C" int sx_ssd_chunks(const SxSsdArgs* a, float* rec, cudaStream_t st) {
+  if (a->chunks.n <= 0) return 0;
+  if (a->N <= 0 || a->N > 256 || a->G <= 0 || a->H % a->G) return -1;
+  SX_ACT_DISPATCH(a->f32, {
+    switch (pad_rows(a->N)) {
+      case 32: return launch_ssd_chunks<A, 32>(a, rec, st);
+      case 64: return launch_ssd_chunks<A, 64>(a, rec, st);
+      case 128: return launch_ssd_chunks<A, 128>(a, rec, st);
+      default: return launch_ssd_chunks<A, 256>(a, rec, st);
     }
   });
   return 0;

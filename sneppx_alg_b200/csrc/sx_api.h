@@ -22,7 +22,8 @@ typedef struct SxGemmArgs {
   long long strideA, strideB, strideD, strideC;  // batch strides in elements (0: operand shared)
   int a_mn, b_mn;
   int out_fp32, c_fp32;
-  int act;  // 0 none, 1 gelu(tanh), 2 silu, 3 relu, 4 xIELU with coefficients act_a (z > 0) and act_b (z <= 0)
+  int act;  // 0 none, 1 gelu(tanh), 2 silu, 3 relu, 4 xIELU with coefficients act_a (z > 0) and act_b (z <= 0),
+            // 5 squared relu, 6 act_a * tanh(z * act_b)
   float alpha, beta;
   const int* tile_group;  // grouped GEMM: per 128-row block of A, index of the B matrix (-1 skips the block)
   int num_groups;         // number of B matrices when tile_group is set
@@ -237,8 +238,12 @@ typedef struct SxChunks {
   int n;
 } SxChunks;
 // f32: 1 for 32-bit activations, 0 for bf16. Norm weights, convolution weights and biases are fp32.
-int sx_embed_f32(const void* table, const int* ids, float* x, int T, int width, int f32, cudaStream_t stream);
+int sx_embed_f32(const void* table, const int* ids, float* x, int T, int width, float scale, int f32, cudaStream_t stream);
 int sx_rmsnorm_f32(const float* x, const float* w, const int* rows, void* y, int T, int width, float eps, int f32, cudaStream_t stream);
+int sx_layernorm_f32(const float* x, const float* w, const float* b, const int* rows, void* y, int T, int width, float eps, int f32,
+                     cudaStream_t stream);
+// RMSNorm of `parts` equal parts of every activation row, in place: y [T, width], row pitch ld, w [width].
+int sx_part_rmsnorm(void* y, long long ld, const float* w, int T, int width, int parts, float eps, int f32, cudaStream_t stream);
 int sx_head_norm_gate(const float* o, const float* w, const void* gate, long long gate_ld, float mul, void* y, long long y_ld,
                       int T, int H, int dv, float eps, int f32, cudaStream_t stream);
 // Stores the last min(length, taps - 1) projected rows of every portion: ring [slots, taps, C], position p in entry p % taps.
@@ -353,6 +358,73 @@ typedef struct SxTalkTcArgs {
 } SxTalkTcArgs;
 int sx_talk_attn_tc_ok(int H, int G, int d, int dv);
 int sx_talk_attn_tc(const SxTalkTcArgs* args, cudaStream_t stream);
+// SSD (Mamba-2) recurrence with an fp32 state [slots, H, N, P] per head: S <- a S + dt B x^T, y = (S^T C + D x) silu(z), from
+// projected rows u = z [H P] | x [H P] | B [G N] | C [G N] | dt [H]. x, B and C pass a causal convolution with bias and silu.
+typedef struct SxSsdArgs {
+  const void* u; long long u_ld;
+  const float* wconv; const float* bconv; void* ring;   // [taps, C], [C], [slots, taps, C], C = H P + 2 G N
+  const float* dt_bias; const float* a_log; const float* D;   // [H]
+  void* x; void* b; void* c;      // operands of the prompt forms: [T, H, xp], [T, G, np] (zeros past P and N)
+  float* dt; float* la;           // [T, H] step size and logarithm of the decay
+  float* state;
+  void* y; long long y_ld;        // [T, H P]
+  SxRagged ragged;
+  SxChunks chunks;
+  int* status;
+  int T, H, P, N, G, taps, xp, np, f32;
+} SxSsdArgs;
+int sx_ssd_operands(const SxSsdArgs* args, cudaStream_t stream);   // u -> x, b, c, dt, la
+int sx_ssd_chunks(const SxSsdArgs* args, float* rec, cudaStream_t stream);   // records for sx_recur_scan (d = N, dv = P)
+int sx_ssd_gate(const SxSsdArgs* args, const float* o, cudaStream_t stream); // y from the read-outs o [T, H, P] of the scan
+int sx_ssd_step(const SxSsdArgs* args, cudaStream_t stream);       // one token per sequence, from u to y
+int sx_ssd_scan_ok(int P, int N);
+int sx_ssd_scan(const SxSsdArgs* args, cudaStream_t stream);       // prompt form on tensor cores (bf16): operands -> state, y
+// Operands of window attention over tokens and averaged blocks, from projected rows u = q [H d] | k [G d] | v [G dv]: bias,
+// rotation of the first `rot` entries of query and key heads, rotation of whole value heads, cache append.
+typedef struct SxWinPrepArgs {
+  const void* u; long long u_ld;
+  const float* bias;                                     // [H d + G d + G dv] or null
+  const double* freq; const double* vfreq;               // [rot / 2], [dv / 2] angle per position
+  const float* temp;                                     // [H] factor on the queries, or null
+  float* q32; void* q; int q_ld;                         // [T, H, d] fp32 or [T, H, q_ld] activations (zeros past d)
+  void* k_out; void* v_out; long long k_ld, v_ld; int dp, dvp;   // packed rows, head j at column j dp / j dvp; or null
+  const int* kv_row;
+  void* k_cache; void* v_cache; const int* cache_entry;  // [entries, G, d], [entries, G, dv]; -1: not stored
+  float* turn;                                           // [T, dv / 2, 2] cos and sin of the value angles
+  SxRagged ragged;
+  // decoding: average of the block of `pool` positions that this token completes (entry -1: none)
+  const int* pool_entry; const int* block_table; const int* block_base; int table_ld, block_size, pool;
+  int T, H, G, d, dv, rot, interleaved, f32;
+  float rot_mul;                                         // factor on cos and sin of the query / key rotation
+} SxWinPrepArgs;
+int sx_win_prep(const SxWinPrepArgs* args, cudaStream_t stream);
+// Averages of the blocks completed by a prompt batch: `pool` packed rows from src[i] on -> packed row row[i], cache entry[i].
+int sx_pool_blocks(void* rows, long long ld, int wp, void* cache, int G, int w, const int* src, const int* row, const int* entry, int n,
+                   int pool, int f32, cudaStream_t stream);
+// Attention of each query to the last `size` positions and to the averages of whole earlier blocks of `pool` positions in one
+// softmax whose denominator also holds exp(sink[h]). Output: values turned back by the position's angles, times
+// sigmoid(gate). Queries carry the temperature. Keys are packed rows (pool_base / kv_base) or cache entries (tables).
+typedef struct SxWinAttnArgs {
+  const float* q32; const void* q; int q_ld;
+  const void* k; const void* v; long long k_ld, v_ld, kv_rows; int dp, dvp;
+  const int* kv_base; const int* pool_base;              // packed: row of position 0, row of block 0 of each sequence
+  const int* tiles; int n_tiles;
+  const int* block_table; const int* block_base; const int* pool_table; int table_ld, pool_ld, block_size;   // paged
+  const float* sink; const float* turn;
+  const void* gate; long long gate_ld;                   // [T, H dv]
+  void* y; long long y_ld;
+  SxRagged ragged;
+  float scale;
+  int T, H, G, d, dv, size, pool, interleaved, f32;
+  float* part; int splits;                               // [T, splits, H, dv + 2]
+  int* status;
+} SxWinAttnArgs;
+int sx_win_attn(const SxWinAttnArgs* args, cudaStream_t stream);          // any sizes; q32
+int sx_win_attn_tc_ok(int H, int G, int d, int dv);
+int sx_win_attn_tc(const SxWinAttnArgs* args, cudaStream_t stream);       // prompts on tensor cores (bf16)
+int sx_win_decode_ok(int H, int G, int d, int dv);
+int sx_win_decode(const SxWinAttnArgs* args, cudaStream_t stream);        // decoding on tensor cores (bf16)
+int sx_win_merge(const SxWinAttnArgs* args, cudaStream_t stream);         // key slices -> y
 
 #ifdef __cplusplus
 }

@@ -270,5 +270,13 @@ __device__ __forceinline__ float xielu(float z, float a, float b) {
   return z > 0.f ? fmaf(a * z, z, 0.5f * z) : fmaf(b, expm1f(z) - z, 0.5f * z);
 }
 __device__ __forceinline__ float silu(float x) { return x / (1.f + __expf(-x)); }
+__device__ __forceinline__ float squared_relu(float z) {
+  const float r = fmaxf(z, 0.f);
+  return r * r;
+}
+// cap * tanh(z / cap) with inv = 1 / cap; tanh x = 1 - 2 / (e^2x + 1) keeps an absolute error of a few 2^-24 everywhere
+__device__ __forceinline__ float softcap(float z, float cap, float inv) {
+  return cap * (1.f - __fdividef(2.f, __expf(fminf(2.f * z * inv, 80.f)) + 1.f));
+}
 
 }  // namespace sx

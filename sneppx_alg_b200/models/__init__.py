@@ -18,15 +18,24 @@ def build_model(cfg, dtype=None, device=None):
     if arch == "deepseek_moe":
         from .deepseek import DeepSeekV2ForCausalLM
         return DeepSeekV2ForCausalLM(cfg, dtype=dtype, device=device)
+    hybrid = _hybrid_class(arch)
+    if hybrid is not None:
+        return hybrid(cfg, dtype=dtype, device=device)
+    raise ValueError(f"unknown architecture '{arch}'")
+
+
+def _hybrid_class(arch):
+    """Class of a hybrid decoder family, None for other architectures."""
     if arch == "rilenex":
         from .rilenex import RilenexForCausalLM
-        return RilenexForCausalLM(cfg, dtype=dtype, device=device)
-    raise ValueError(f"unknown architecture '{arch}'")
+        return RilenexForCausalLM
+    if arch == "tibalorn":
+        from .tibalorn import TibalornForCausalLM
+        return TibalornForCausalLM
+    return None
 
 
 def complete_config(cfg, tensors):
     """Fill in the sizes that a checkpoint gives only through its tensors' shapes (a no-op for most families)."""
-    if cfg.architecture == "rilenex":
-        from .rilenex import RilenexForCausalLM
-        return RilenexForCausalLM.config_from_tensors(cfg, tensors)
-    return cfg
+    hybrid = _hybrid_class(cfg.architecture)
+    return hybrid.config_from_tensors(cfg, tensors) if hybrid is not None else cfg

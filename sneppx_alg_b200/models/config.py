@@ -21,6 +21,18 @@ def _rilenex_fields(d: Dict[str, Any]) -> Dict[str, Any]:
     return out
 
 
+def _tibalorn_fields(d: Dict[str, Any]) -> Dict[str, Any]:
+    """The keys of a Tibalorn ``config.json`` under this schema's names; other keys pass through."""
+    out = {k: v for k, v in d.items() if k not in ("layers", "vocab", "width", "norm", "embedding")}
+    out.update(architecture="tibalorn", layer_specs=d["layers"], vocab_size=d["vocab"], hidden_size=d["width"],
+               layer_norm_eps=d["norm"]["eps"], num_hidden_layers=len(d["layers"]), embedding_scale=d["embedding"]["scale"],
+               tie_word_embeddings=True, use_rms_norm=False)
+    return out
+
+
+_FIELD_READERS = {"rilenex": _rilenex_fields, "tibalorn": _tibalorn_fields}
+
+
 @dataclass
 class ModelConfig:
     # identity
@@ -31,7 +43,7 @@ class ModelConfig:
     license: str = ""
     repository: str = ""
     homepage: str = ""
-    architecture: str = "transformer"   # transformer | mamba2 | hss_ser | deepseek_moe | rilenex | bert | gpt | t5 | vit
+    architecture: str = "transformer"   # transformer | mamba2 | hss_ser | deepseek_moe | rilenex | tibalorn | bert | gpt | t5 | vit
     model_type: str = "causal-lm"
     framework: str = "sneppx"
     # shape
@@ -108,6 +120,8 @@ class ModelConfig:
     ssm_chunk_size: int = 256
     # per-layer specifications of hybrid decoders: {"type", "mixer": {sizes}, "mlp": {sizes} or None}
     layer_specs: List[dict] = field(default_factory=list)
+    embedding_scale: float = 1.0     # factor on the embedding rows as they enter the residual stream
+    logit_softcap: float = 0.0       # logits <- cap * tanh(logits / cap); 0: none
     custom: Dict[str, Any] = field(default_factory=dict)
 
     def __post_init__(self):
@@ -137,8 +151,9 @@ class ModelConfig:
 
     @classmethod
     def from_dict(cls, d: Dict[str, Any]) -> "ModelConfig":
-        if str(d.get("architecture", "")).lower() == "rilenex" and "layers" in d:
-            d = _rilenex_fields(d)
+        reader = _FIELD_READERS.get(str(d.get("architecture", "")).lower())
+        if reader is not None and "layers" in d:
+            d = reader(d)
         names = {f.name for f in dataclasses.fields(cls)}
         known = {k: v for k, v in d.items() if k in names}
         extra = {k: v for k, v in d.items() if k not in names}
@@ -171,6 +186,8 @@ class ModelConfig:
         d, L, V = self.hidden_size, self.num_hidden_layers, self.vocab_size
         if self.architecture == "rilenex":
             return _rilenex_parameters(self)
+        if self.architecture == "tibalorn":
+            return _tibalorn_parameters(self)
         hd = self.head_dim or 0
         attn = d * (self.num_attention_heads + 2 * self.num_key_value_heads) * hd + self.num_attention_heads * hd * d
         ffn = (3 if self.gated_ffn else 2) * d * self.intermediate_size
@@ -206,6 +223,22 @@ def _rilenex_parameters(cfg: ModelConfig) -> int:
             total += d * (c + H + ra + rg + H * v) + r["conv"] * c + ra * H * k + rg * H * v + H * (k + 1) + v + d
         if s.get("mlp") is not None:
             total += 2 * d * s["mlp"]["ff"] + d + 2
+    return total
+
+
+def _tibalorn_parameters(cfg: ModelConfig) -> int:
+    d, total = cfg.hidden_size, (cfg.vocab_size + 2) * cfg.hidden_size
+    for s in cfg.layer_specs:
+        m = s["mixer"]
+        total += 2 * d
+        if s["type"] == "mamba2":
+            inner, c = m["heads"] * m["vdim"], m["heads"] * m["vdim"] + 2 * m["groups"] * m["state"]
+            total += d * (2 * inner + c + m["heads"]) + (m["conv"] + 1) * c + 3 * m["heads"] + inner
+        else:
+            q, k, v, o = m["heads"] * m["dim"], m["kv_heads"] * m["dim"], m["kv_heads"] * m["vdim"], m["heads"] * m["vdim"]
+            total += (d + 1) * (q + k + v) + 2 * d * o + 2 * m["heads"]
+        if s.get("mlp") is not None:
+            total += 2 * d * s["mlp"]["ff"] + 2 * d
     return total
 
 
@@ -312,6 +345,31 @@ _MODEL_REGISTRY["rilenex"] = {
                    dict(heads=32, kv_heads=32, dim=128, vdim=128, conv=4, decay_rank=128, gate_rank=128)),
 }
 
+def _tibalorn(width, ff, vocab, groups, mamba, attention, max_len=131072):
+    """Layer pattern of the presets: ``groups`` times three recurrent layers followed by one attention layer."""
+    m = {"type": "mamba2", "mixer": mamba, "mlp": None}
+    a = {"type": "attention", "mixer": attention, "mlp": {"kind": "dense", "ff": ff}}
+    return dict(architecture="tibalorn", hidden_size=width, vocab_size=vocab, layer_specs=[m, m, m, a] * groups,
+                num_hidden_layers=4 * groups, max_position_embeddings=max_len, layer_norm_eps=1e-5, use_rms_norm=False,
+                embedding_scale=width ** 0.5, logit_softcap=30.0, tie_word_embeddings=True)
+
+
+def _yarn(base, dims, original, factor):
+    return {"base": base, "dims": dims, "scaling": {"factor": factor, "original": original, "fast": 32.0, "slow": 1.0}}
+
+
+_MODEL_REGISTRY["tibalorn"] = {
+    "tiny": _tibalorn(128, 192, 512, 1, dict(heads=4, vdim=32, state=16, groups=2, conv=4, norm_groups=2),
+                      dict(heads=4, kv_heads=2, dim=32, vdim=24, mask={"size": 40, "pool": 8}, rot=_yarn(1e4, 16, 128, 8.0), scale=0.2),
+                      max_len=4096),
+    "1B": _tibalorn(2048, 8192, 32000, 7, dict(heads=64, vdim=64, state=128, groups=1, conv=4, norm_groups=1),
+                    dict(heads=16, kv_heads=4, dim=128, vdim=128, mask={"size": 2048, "pool": 16}, rot=_yarn(5e5, 128, 8192, 16.0),
+                         scale=128 ** -0.5)),
+    "7B": _tibalorn(4096, 14336, 32000, 9, dict(heads=128, vdim=64, state=128, groups=8, conv=4, norm_groups=8),
+                    dict(heads=32, kv_heads=8, dim=128, vdim=128, mask={"size": 4096, "pool": 16}, rot=_yarn(5e5, 128, 8192, 16.0),
+                         scale=128 ** -0.5)),
+}
+
 _ALIASES = {"llama": "llama2", "llama-2": "llama2", "llama-3": "llama3", "deepseek": "deepseek_v2",
             "deepseek-v2": "deepseek_v2", "mamba-2": "mamba2", "hss": "hss_ser"}
 
@@ -334,11 +392,11 @@ def get_model_config(family: str, size: str) -> dict:
 
 
 def config_from_name(name: str) -> ModelConfig:
-    """'llama3-8b', 'meta-llama/Llama-3-8B', 'mistral-7b', 'deepseek-v2-lite', 'mamba2-2.7b', 'hss-ser-tiny', 'rilenex-1b' ..."""
+    """'llama3-8b', 'meta-llama/Llama-3-8B', 'mistral-7b', 'deepseek-v2-lite', 'mamba2-2.7b', 'hss-ser-tiny', 'rilenex-1b', 'tibalorn-1b' ..."""
     n = name.lower().split("/")[-1].replace("_", "-")
     table = [("llama-3", "llama3"), ("llama3", "llama3"), ("llama-2", "llama2"), ("llama2", "llama2"),
              ("llama", "llama2"), ("mistral", "mistral"), ("qwen2", "qwen2"), ("deepseek", "deepseek_v2"),
-             ("mamba", "mamba2"), ("hss", "hss_ser"), ("rilenex", "rilenex")]
+             ("mamba", "mamba2"), ("hss", "hss_ser"), ("rilenex", "rilenex"), ("tibalorn", "tibalorn")]
     for pat, fam in table:
         if pat in n:
             for size in _MODEL_REGISTRY[fam]:

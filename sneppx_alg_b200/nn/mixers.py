@@ -1,6 +1,6 @@
 """Token mixers of the hybrid decoders, built from branches that share one layer input.
 
-A branch (``GatedWriteBranch``, ``DeltaBranch``, ``TalkingAttentionBranch``) names the projections it reads, the state it
+A branch (``GatedWriteBranch``, ``DeltaBranch``, ``SSDBranch``, ``TalkingAttentionBranch``, ``PooledAttentionBranch``) names the projections it reads, the state it
 keeps per sequence and the columns it produces; ``FusedMixer`` runs any number of branches side by side: one GEMM projects
 the layer input for all of them, every branch writes its read-outs (norm, gate and branch scale applied in fp32) into its
 columns of one buffer, and one GEMM multiplies those with the joined output weights and adds the result to the fp32
@@ -10,6 +10,7 @@ Tensor names are those of the checkpoint, relative to the mixer (``tensors()``);
 """
 from __future__ import annotations
 
+import math
 from collections import OrderedDict
 from typing import Dict, List, Tuple
 
@@ -42,7 +43,7 @@ class Branch(Module):
     out_width: int
 
     def kv_spec(self):
-        """(kv heads, key size, value size, chunk length) of the cached keys, or None."""
+        """(kv heads, key size, value size, mask) of the cached keys, or None; a chunk length stands for its mask."""
         return None
 
     def state_spec(self, act_dtype) -> Dict[str, Tuple[tuple, torch.dtype]]:
@@ -135,6 +136,122 @@ class DeltaBranch(Branch):
         hybrid.conv_ring(qkv, state["ring"], batch, self.channels, self.taps)
         o = hybrid.recur_scan(rec, v, state["S"], batch, H, d, dv, delta=True)
         hybrid.head_norm_gate(o, self.norm, y, self.eps, gate=gate, mul=scale)
+
+
+class SSDBranch(Branch):
+    """Mamba-2 recurrence (state-space duality): one projection z | x | B | C | dt, a short convolution with bias and silu on x,
+    B and C, one decay per head, B and C shared by the heads of a group, output gate silu(z), then an RMS norm in equal
+    parts."""
+
+    def __init__(self, heads, vdim, state, groups, taps, norm_parts, eps, dtype=None, device=None):
+        super().__init__()
+        if heads % groups or (heads * vdim) % norm_parts:
+            raise ValueError(f"{heads} heads of size {vdim} do not divide into {groups} groups and {norm_parts} norm parts")
+        self.H, self.P, self.N, self.G, self.taps, self.parts, self.eps = heads, vdim, state, groups, taps, norm_parts, eps
+        inner = heads * vdim
+        self.channels = inner + 2 * groups * state
+        self.segments = OrderedDict([("in", inner + self.channels + heads)])
+        self.out_width = inner
+        f32 = dict(dtype=torch.float32, device=device)
+        self.conv = _param(taps, self.channels, fill=1.0 / taps, **f32)
+        self.conv_bias = _param(self.channels, **f32)
+        self.dt_bias = _param(heads, fill=-2.0, **f32)
+        self.a_log = _param(heads, **f32)
+        self.skip = _param(heads, fill=1.0, **f32)
+        self.norm = _param(inner, fill=1.0, **f32)
+
+    def state_spec(self, act_dtype):
+        return {"S": ((self.H, self.N, self.P), torch.float32), "ring": ((self.taps, self.channels), act_dtype)}
+
+    def tensors(self):
+        return [("conv", self.conv.data.t()), ("conv.b", self.conv_bias), ("dt_bias", self.dt_bias), ("A_log", self.a_log), ("D", self.skip),
+                ("norm", self.norm)]
+
+    def run(self, u, y, batch, state, kv, scale):
+        if scale != 1.0:
+            raise NotImplementedError("the norm of this branch takes no scale")
+        fn = hybrid.ssd_step if batch.decode else hybrid.ssd_prompt
+        fn(u["in"], self.conv, self.conv_bias, state["ring"], self.dt_bias, self.a_log, self.skip, state["S"], y, batch, self.H, self.P, self.N,
+           self.G, self.taps)
+        hybrid.part_rmsnorm_(y, self.norm, self.parts, self.eps)
+
+
+def rotary_frequencies(dims, base, scaling=None):
+    """Angles per position of the ``dims / 2`` rotation pairs (float64) and the factor on cos and sin. ``scaling`` (YaRN:
+    factor, original, fast, slow) divides the slow pairs by the factor, leaves the fast ones, and blends in between."""
+    i = torch.arange(dims // 2, dtype=torch.float64)
+    f = float(base) ** (-2.0 * i / max(dims, 1))
+    if not scaling:
+        return f, 1.0
+
+    def pair_of(turns):       # pair that turns this often over the original length
+        return dims * math.log(scaling["original"] / (2 * math.pi * turns)) / (2 * math.log(base))
+
+    lo, hi = max(math.floor(pair_of(scaling["fast"])), 0), min(math.ceil(pair_of(scaling["slow"])), dims - 1)
+    ramp = ((i - lo) / max(hi - lo, 0.001)).clamp(0, 1)
+    return f * (ramp / scaling["factor"] + (1 - ramp)), 0.1 * math.log(scaling["factor"]) + 1
+
+
+class PooledAttentionBranch(Branch):
+    """Grouped-query attention to a window of tokens and to averages of older blocks (``window``), with projection biases,
+    rotated queries and keys, values rotated by their position and turned back by the query's, a temperature per head, a sink
+    in the softmax and an elementwise output gate. ``interleaved``: rotation pairs are neighbours instead of halves."""
+
+    def __init__(self, heads, kv_heads, dim, vdim, window, rot_dims, rot_base, scale, scaling=None, interleaved=False, dtype=None, device=None):
+        super().__init__()
+        if vdim % 2 or rot_dims % 2 or rot_dims > dim:
+            raise ValueError(f"rotation of {rot_dims} of {dim} key entries and {vdim} value entries")
+        if window.size < 1 or window.pool < 1:
+            raise ValueError(f"window of {window.size} tokens with blocks of {window.pool}")
+        self.H, self.G, self.d, self.dv, self.window, self.scale, self.interleaved = heads, kv_heads, dim, vdim, window, scale, interleaved
+        self.segments = OrderedDict(q=heads * dim, k=kv_heads * dim, v=kv_heads * vdim, g=heads * vdim)
+        self.tight = ("q", "k", "v")
+        self.out_width = heads * vdim
+        f32 = dict(dtype=torch.float32, device=device)
+        self.bias = _param(heads * dim + kv_heads * (dim + vdim), **f32)
+        self.temp = _param(heads, fill=1.0, **f32)
+        self.sink = _param(heads, **f32)
+        freq, self.rot_mul = rotary_frequencies(rot_dims, rot_base, scaling)
+        self._freq = (freq, rotary_frequencies(vdim, rot_base)[0])
+
+    def freqs(self, device):
+        if self._freq[0].device != device:
+            self._freq = tuple(f.to(device) for f in self._freq)
+        return self._freq
+
+    def kv_spec(self):
+        return self.G, self.d, self.dv, self.window
+
+    def tensors(self):
+        a, b = self.H * self.d, (self.H + self.G) * self.d
+        c = self.bias.data
+        return [("q.b", c[:a]), ("k.b", c[a:b]), ("v.b", c[b:]), ("temp", self.temp), ("sink", self.sink)]
+
+    def run(self, u, y, batch, state, kv, scale):
+        if scale != 1.0:
+            raise NotImplementedError("the gate of this branch takes no scale")
+        H, G, d, dv, win = self.H, self.G, self.d, self.dv, self.window
+        k_cache, v_cache = kv
+        qkv, gate = u["q"], u["g"]
+        dev, act = qkv.device, qkv.dtype
+        prep = (qkv, self.bias, *self.freqs(dev), self.rot_mul, self.temp, batch, k_cache, v_cache, H, G, d, dv, self.interleaved)
+        tc = (hybrid.window_decode_tc if batch.decode else hybrid.window_tc)(act, H, G, d, dv)
+        q = dict(q=torch.empty(batch.T, H, _up(d, 16 if batch.decode else 64), dtype=act, device=dev)) if tc else             dict(q32=torch.empty(batch.T, H, d, dtype=torch.float32, device=dev))
+        if batch.decode:
+            turn = hybrid.win_prep(*prep, **q, pool=win.pool)
+            hybrid.window_decode(k_cache, v_cache, self.sink, turn, gate, y, batch, self.scale, H, G, d, dv, win, self.interleaved, **q)
+            return
+        view = batch.views[win]
+        dp, dvp = _up(d), _up(dv)
+        k = (torch.empty if dp == d else torch.zeros)(view.rows, G * dp, dtype=act, device=dev)
+        v = (torch.empty if dvp == dv else torch.zeros)(view.rows, G * dvp, dtype=act, device=dev)
+        # before the append: the append may reuse blocks that earlier positions still occupy
+        hybrid.kv_gather(k_cache, view.gather_entry, view.gather_row, k, G, d, dp)
+        hybrid.kv_gather(v_cache, view.gather_entry, view.gather_row, v, G, dv, dvp)
+        turn = hybrid.win_prep(*prep, **q, k_out=k, v_out=v, dp=dp, dvp=dvp, kv_row=view.kv_row)
+        hybrid.pool_blocks(k, dp, k_cache, view, G, d, win.pool)
+        hybrid.pool_blocks(v, dvp, v_cache, view, G, dv, win.pool)
+        hybrid.window_attention(k, v, dp, dvp, self.sink, turn, gate, y, batch, view, self.scale, H, G, d, dv, win, self.interleaved, **q)
 
 
 class TalkingAttentionBranch(Branch):

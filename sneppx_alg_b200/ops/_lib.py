@@ -119,6 +119,38 @@ class SxTalkTcArgs(C.Structure):
     ]
 
 
+class SxSsdArgs(C.Structure):
+    _fields_ = [
+        ("u", c_void_p), ("u_ld", c_ll), ("wconv", c_void_p), ("bconv", c_void_p), ("ring", c_void_p), ("dt_bias", c_void_p),
+        ("a_log", c_void_p), ("D", c_void_p), ("x", c_void_p), ("b", c_void_p), ("c", c_void_p), ("dt", c_void_p), ("la", c_void_p),
+        ("state", c_void_p), ("y", c_void_p), ("y_ld", c_ll), ("ragged", SxRagged), ("chunks", SxChunks), ("status", c_void_p),
+        ("T", c_int), ("H", c_int), ("P", c_int), ("N", c_int), ("G", c_int), ("taps", c_int), ("xp", c_int), ("np", c_int), ("f32", c_int),
+    ]
+
+
+class SxWinPrepArgs(C.Structure):
+    _fields_ = [
+        ("u", c_void_p), ("u_ld", c_ll), ("bias", c_void_p), ("freq", c_void_p), ("vfreq", c_void_p), ("temp", c_void_p),
+        ("q32", c_void_p), ("q", c_void_p), ("q_ld", c_int), ("k_out", c_void_p), ("v_out", c_void_p), ("k_ld", c_ll), ("v_ld", c_ll),
+        ("dp", c_int), ("dvp", c_int), ("kv_row", c_void_p), ("k_cache", c_void_p), ("v_cache", c_void_p), ("cache_entry", c_void_p),
+        ("turn", c_void_p), ("ragged", SxRagged), ("pool_entry", c_void_p), ("block_table", c_void_p), ("block_base", c_void_p),
+        ("table_ld", c_int), ("block_size", c_int), ("pool", c_int), ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int), ("dv", c_int),
+        ("rot", c_int), ("interleaved", c_int), ("f32", c_int), ("rot_mul", c_float),
+    ]
+
+
+class SxWinAttnArgs(C.Structure):
+    _fields_ = [
+        ("q32", c_void_p), ("q", c_void_p), ("q_ld", c_int), ("k", c_void_p), ("v", c_void_p), ("k_ld", c_ll), ("v_ld", c_ll),
+        ("kv_rows", c_ll), ("dp", c_int), ("dvp", c_int), ("kv_base", c_void_p), ("pool_base", c_void_p), ("tiles", c_void_p),
+        ("n_tiles", c_int), ("block_table", c_void_p), ("block_base", c_void_p), ("pool_table", c_void_p), ("table_ld", c_int),
+        ("pool_ld", c_int), ("block_size", c_int), ("sink", c_void_p), ("turn", c_void_p), ("gate", c_void_p), ("gate_ld", c_ll),
+        ("y", c_void_p), ("y_ld", c_ll), ("ragged", SxRagged), ("scale", c_float), ("T", c_int), ("H", c_int), ("G", c_int), ("d", c_int),
+        ("dv", c_int), ("size", c_int), ("pool", c_int), ("interleaved", c_int), ("f32", c_int), ("part", c_void_p), ("splits", c_int),
+        ("status", c_void_p),
+    ]
+
+
 _lock = threading.Lock()
 _lib = None
 _status = {}

@@ -16,7 +16,7 @@ import torch
 
 from . import _lib
 
-ACT = {None: 0, "none": 0, "gelu": 1, "silu": 2, "relu": 3}
+ACT = {None: 0, "none": 0, "gelu": 1, "silu": 2, "relu": 3, "relu2": 5}
 
 
 class XIELU:
@@ -34,9 +34,23 @@ class XIELU:
         return torch.where(z > 0, self.a * z * z, self.b * (torch.expm1(zn) - zn)) + 0.5 * z
 
 
+class SoftCap:
+    """Activation object for ``gemm(act=...)``: cap * tanh(z / cap)."""
+
+    code = 6
+
+    def __init__(self, cap: float):
+        self.a, self.b = float(cap), 1.0 / float(cap)
+
+    def __call__(self, z):
+        return self.a * torch.tanh(z / self.a)
+
+
 def _act_ref(x, act):
-    if isinstance(act, XIELU):
+    if isinstance(act, (XIELU, SoftCap)):
         return act(x)
+    if act in ("relu2", 5):
+        return torch.relu(x) ** 2
     if act in (None, "none", 0):
         return x
     if act in ("gelu", 1):
@@ -213,7 +227,7 @@ def gemm(a, b, *, a_mn=False, b_mn=False, out=None, out_dtype=None, c=None, beta
     args.a_mn, args.b_mn = int(a_mn), int(b_mn)
     args.out_fp32 = int(out.dtype == torch.float32)
     args.c_fp32 = int(c is not None and c.dtype == torch.float32)
-    if isinstance(act, XIELU):
+    if isinstance(act, (XIELU, SoftCap)):
         args.act, args.act_a, args.act_b = act.code, act.a, act.b
     else:
         args.act = ACT[act] if not isinstance(act, int) else act

@@ -1,6 +1,7 @@
-"""Front-ends of the hybrid-decoder kernels: fp32-residual norms, the gated recurrences (``csrc/recurrence.cu``), and
-chunked attention with a head mix before the softmax (``csrc/talking_attn.cu``). They run on CUDA tensors only; activations
-are bf16 or fp32, everything that the recurrences and the softmax work on is fp32 inside."""
+"""Front-ends of the hybrid-decoder kernels: fp32-residual norms, the gated recurrences (``csrc/recurrence.cu``), the SSD
+recurrence (``csrc/ssd_serve.cu``), chunked attention with a head mix before the softmax (``csrc/talking_attn.cu``), and window
+attention over tokens and averaged blocks (``csrc/window_attn.cu``). They run on CUDA tensors only; activations are bf16 or
+fp32, everything that the recurrences and the softmax work on is fp32 inside."""
 from __future__ import annotations
 
 import ctypes as C
@@ -26,11 +27,12 @@ def _need_cuda(t):
     _lib.lib()
 
 
-def embed_f32(table, ids):
-    """fp32 rows of the embedding table."""
+def embed_f32(table, ids, scale=1.0):
+    """fp32 rows of the embedding table, times ``scale``."""
     _need_cuda(table)
     x = torch.empty(ids.numel(), table.shape[1], dtype=torch.float32, device=table.device)
-    _lib.call("sx_embed_f32", ptr(table), ptr(ids), ptr(x), c_int(ids.numel()), c_int(table.shape[1]), c_int(_f32(table)), stream())
+    _lib.call("sx_embed_f32", ptr(table), ptr(ids), ptr(x), c_int(ids.numel()), c_int(table.shape[1]), c_float(scale),
+              c_int(_f32(table)), stream())
     return x
 
 
@@ -41,6 +43,22 @@ def rmsnorm_f32(x, w, eps, out_dtype, rows=None):
     y = torch.empty(n, x.shape[1], dtype=out_dtype, device=x.device)
     _lib.call("sx_rmsnorm_f32", ptr(x), ptr(w), ptr(rows), ptr(y), c_int(n), c_int(x.shape[1]), c_float(eps), c_int(_f32(y)), stream())
     return y
+
+
+def layernorm_f32(x, w, b, eps, out_dtype, rows=None):
+    """Layer norm with weight and bias of fp32 rows (all of them, or the listed ones) into activations."""
+    _need_cuda(x)
+    n = x.shape[0] if rows is None else rows.numel()
+    y = torch.empty(n, x.shape[1], dtype=out_dtype, device=x.device)
+    _lib.call("sx_layernorm_f32", ptr(x), ptr(w), ptr(b), ptr(rows), ptr(y), c_int(n), c_int(x.shape[1]), c_float(eps), c_int(_f32(y)),
+              stream())
+    return y
+
+
+def part_rmsnorm_(y, w, parts, eps):
+    """RMS norm of ``parts`` equal parts of every row of y (a column slice will do), in place."""
+    _lib.call("sx_part_rmsnorm", ptr(y), c_ll(y.stride(0)), ptr(w), c_int(y.shape[0]), c_int(y.shape[1]), c_int(parts), c_float(eps),
+              c_int(_f32(y)), stream())
 
 
 def head_norm_gate(o, w, y, eps, gate=None, mul=1.0):
@@ -138,6 +156,55 @@ def delta_step(u, wconv, ring, b, a, a_log, dt_bias, state, norm, y, batch: Ragg
     _lib.call("sx_recur_step", C.byref(s), stream())
 
 
+# ----------------------------------------------------------------------------- SSD recurrence
+def _ssd_args(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch, H, P, N, G, taps):
+    a = _lib.SxSsdArgs()
+    a.u, a.u_ld, a.wconv, a.bconv, a.ring = u.data_ptr(), u.stride(0), wconv.data_ptr(), bconv.data_ptr(), ring.data_ptr()
+    a.dt_bias, a.a_log, a.D, a.state, a.y, a.y_ld = (dt_bias.data_ptr(), a_log.data_ptr(), D.data_ptr(), state.data_ptr(), y.data_ptr(),
+                                                     y.stride(0))
+    a.ragged = batch.struct()
+    if not batch.decode:
+        a.chunks = batch.chunks()
+    a.status = _lib.status_word(u.device).data_ptr()
+    a.T, a.H, a.P, a.N, a.G, a.taps, a.xp, a.np, a.f32 = batch.T, H, P, N, G, taps, P, N, _f32(u)
+    return a
+
+
+def ssd_scan_tc(act_dtype, P, N) -> bool:
+    """Whether the tensor-core prompt kernel takes these sizes."""
+    return act_dtype == torch.bfloat16 and bool(_lib.lib().sx_ssd_scan_ok(c_int(P), c_int(N)))
+
+
+def ssd_prompt(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch: RaggedBatch, H, P, N, G, taps):
+    """Portions through the SSD recurrence, from projected rows (z | x | B | C | dt) to gated read-outs in y."""
+    _need_cuda(u)
+    T, dev = batch.T, u.device
+    tc = ssd_scan_tc(u.dtype, P, N)
+    a = _ssd_args(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch, H, P, N, G, taps)
+    if tc:
+        a.xp, a.np = (P + 7) // 8 * 8, (N + 7) // 8 * 8
+    x = torch.empty(T, H * a.xp, dtype=u.dtype, device=dev)
+    b, c = torch.empty(2, T, G * a.np, dtype=u.dtype, device=dev)
+    dt, la = torch.empty(2, T, H, dtype=torch.float32, device=dev)
+    a.x, a.b, a.c, a.dt, a.la = x.data_ptr(), b.data_ptr(), c.data_ptr(), dt.data_ptr(), la.data_ptr()
+    _lib.call("sx_ssd_operands", C.byref(a), stream())
+    conv_ring(u[:, H * P:], ring, batch, H * P + 2 * G * N, taps)
+    if tc:
+        _lib.call("sx_ssd_scan", C.byref(a), stream())
+        return
+    rec = _records(batch, H, N, False, dev)
+    _lib.call("sx_ssd_chunks", C.byref(a), ptr(rec), stream())
+    o = recur_scan(rec, x, state, batch, H, N, P, delta=False)
+    _lib.call("sx_ssd_gate", C.byref(a), ptr(o), stream())
+
+
+def ssd_step(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch: RaggedBatch, H, P, N, G, taps):
+    """One token of every sequence through the SSD recurrence, from projected rows to gated read-outs in y."""
+    _need_cuda(u)
+    a = _ssd_args(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch, H, P, N, G, taps)
+    _lib.call("sx_ssd_step", C.byref(a), stream())
+
+
 # ----------------------------------------------------------------------------- attention with a head mix
 def qkv_prep(u, wconv, ring, qn, kn, inv_freq, batch: RaggedBatch, k_cache, v_cache, H, G, d, dv, taps, eps, q_out=None,
              qmix_out=None, talk=None, k_out=None, v_out=None, dvp=0, kv_row=None):
@@ -230,3 +297,92 @@ def talking_decode(q, k_cache, v_cache, talk, gate, y, batch: RaggedBatch, scale
         _lib.call("sx_talk_decode", C.byref(a), ptr(qmix), c_int(qmix.shape[-1]), stream())
     else:
         _lib.call("sx_talk_attn", C.byref(a), stream())
+
+
+# ----------------------------------------------------------------------------- window attention over tokens and averaged blocks
+def win_prep(u, bias, freq, vfreq, rot_mul, temp, batch: RaggedBatch, k_cache, v_cache, H, G, d, dv, interleaved=False, q32=None, q=None,
+             k_out=None, v_out=None, dp=0, dvp=0, kv_row=None, pool=0):
+    """Bias, rotation and cache append of attention operands (see ``SxWinPrepArgs``); returns the table of value angles. In
+    decoding also averages the blocks of ``pool`` positions that the tokens complete."""
+    _need_cuda(u)
+    turn = torch.empty(batch.T, dv // 2, 2, dtype=torch.float32, device=u.device)
+    a = _lib.SxWinPrepArgs()
+    a.u, a.u_ld, a.freq, a.vfreq = u.data_ptr(), u.stride(0), freq.data_ptr(), vfreq.data_ptr()
+    for name, t in (("bias", bias), ("temp", temp), ("q32", q32), ("q", q), ("k_out", k_out), ("v_out", v_out), ("kv_row", kv_row)):
+        if t is not None:
+            setattr(a, name, t.data_ptr())
+    if q is not None:
+        a.q_ld = q.shape[-1]
+    if k_out is not None:
+        a.k_ld, a.v_ld, a.dp, a.dvp = k_out.stride(0), v_out.stride(0), dp, dvp
+    a.k_cache, a.v_cache, a.cache_entry, a.turn = k_cache.data_ptr(), v_cache.data_ptr(), batch.entry.data_ptr(), turn.data_ptr()
+    a.ragged = batch.struct()
+    if batch.decode and pool:
+        a.pool_entry, a.block_table, a.block_base = batch.pool_entry[pool].data_ptr(), batch.block_table.data_ptr(), batch.block_base.data_ptr()
+        a.table_ld, a.block_size, a.pool = batch.table_width, k_cache.shape[1], pool
+    a.T, a.H, a.G, a.d, a.dv, a.rot, a.interleaved, a.f32 = batch.T, H, G, d, dv, 2 * freq.numel(), int(interleaved), _f32(u)
+    a.rot_mul = rot_mul
+    _lib.call("sx_win_prep", C.byref(a), stream())
+    return turn
+
+
+def pool_blocks(rows, wp, cache, view, G, w, pool):
+    """Averages of the blocks that a prompt batch completes, from its packed rows (head pitch ``wp``) to their packed rows and
+    cache entries."""
+    if view.n_pool:
+        _lib.call("sx_pool_blocks", ptr(rows), c_ll(rows.stride(0)), c_int(wp), ptr(cache), c_int(G), c_int(w), ptr(view.pool_src),
+                  ptr(view.pool_row), ptr(view.pool_entry), c_int(view.n_pool), c_int(pool), c_int(_f32(rows)), stream())
+
+
+def _win_args(sink, turn, gate, y, batch, scale, H, G, d, dv, window, interleaved):
+    a = _lib.SxWinAttnArgs()
+    a.sink, a.turn, a.gate, a.gate_ld, a.y, a.y_ld = (sink.data_ptr(), turn.data_ptr(), gate.data_ptr(), gate.stride(0), y.data_ptr(),
+                                                      y.stride(0))
+    a.ragged = batch.struct()
+    a.scale, a.T, a.H, a.G, a.d, a.dv, a.size, a.pool = scale, batch.T, H, G, d, dv, window.size, window.pool
+    a.interleaved, a.f32, a.splits = int(interleaved), _f32(y), 1
+    a.status = _lib.status_word(y.device).data_ptr()
+    return a
+
+
+def window_tc(act_dtype, H, G, d, dv) -> bool:
+    """Whether the tensor-core prompt kernel takes these sizes."""
+    return act_dtype == torch.bfloat16 and bool(_lib.lib().sx_win_attn_tc_ok(c_int(H), c_int(G), c_int(d), c_int(dv)))
+
+
+def window_attention(k, v, dp, dvp, sink, turn, gate, y, batch: RaggedBatch, view, scale, H, G, d, dv, window, interleaved=False, q32=None,
+                     q=None):
+    """Prompt form over packed keys and values. Either ``q32`` (fp32 [T, H, d], any sizes) or ``q`` (bf16 [T, H, q_ld], the
+    tensor-core kernel)."""
+    a = _win_args(sink, turn, gate, y, batch, scale, H, G, d, dv, window, interleaved)
+    a.k, a.v, a.k_ld, a.v_ld, a.kv_rows, a.dp, a.dvp = k.data_ptr(), v.data_ptr(), k.stride(0), v.stride(0), k.shape[0], dp, dvp
+    a.kv_base, a.pool_base = view.kv_base.data_ptr(), view.pool_base.data_ptr()
+    if q is not None:
+        a.q, a.q_ld, a.tiles, a.n_tiles = q.data_ptr(), q.shape[-1], view.tiles.data_ptr(), view.n_tiles
+        _lib.call("sx_win_attn_tc", C.byref(a), stream())
+    else:
+        a.q32 = q32.data_ptr()
+        _lib.call("sx_win_attn", C.byref(a), stream())
+
+
+def window_decode_tc(act_dtype, H, G, d, dv) -> bool:
+    """Whether the tensor-core decode kernel takes these sizes."""
+    return act_dtype == torch.bfloat16 and bool(_lib.lib().sx_win_decode_ok(c_int(H), c_int(G), c_int(d), c_int(dv)))
+
+
+def window_decode(k_cache, v_cache, sink, turn, gate, y, batch: RaggedBatch, scale, H, G, d, dv, window, interleaved=False, q32=None, q=None):
+    """Decode form: one query per sequence against the block pool; ``q32`` or ``q`` as in the prompt form."""
+    a = _win_args(sink, turn, gate, y, batch, scale, H, G, d, dv, window, interleaved)
+    a.k, a.v, a.k_ld, a.v_ld, a.dp, a.dvp = k_cache.data_ptr(), v_cache.data_ptr(), G * d, G * dv, d, dv
+    a.block_table, a.block_base, a.table_ld, a.block_size = batch.block_table.data_ptr(), batch.block_base.data_ptr(), batch.table_width, k_cache.shape[1]
+    a.pool_table, a.pool_ld = batch.pool_table[window.pool].data_ptr(), batch.pool_width
+    most = window.size + batch.pool_width * a.block_size
+    a.splits = max(1, min((most + 127) // 128, 2 * 148 // max(batch.n * G, 1)))
+    part = torch.empty(batch.n * a.splits * H * (dv + 2), dtype=torch.float32, device=y.device)
+    a.part = part.data_ptr()
+    if q is not None:
+        a.q, a.q_ld = q.data_ptr(), q.shape[-1]
+        _lib.call("sx_win_decode", C.byref(a), stream())
+    else:
+        a.q32 = q32.data_ptr()
+        _lib.call("sx_win_attn", C.byref(a), stream())

@@ -14,10 +14,53 @@ from . import _lib
 RECUR_CHUNK = 16     # tokens per chunk of the recurrence kernels
 
 
+@dataclass(frozen=True)
+class Chunk:
+    """Position p sees the positions of its own chunk of ``size`` up to itself."""
+
+    size: int
+    pool = 0
+
+    def first(self, pos: int) -> int:
+        """Earliest position whose key a token at ``pos`` needs."""
+        return pos // self.size * self.size
+
+    @property
+    def span(self) -> int:
+        """Most positions between ``first(pos)`` and ``pos``, both included."""
+        return self.size
+
+
+@dataclass(frozen=True)
+class PooledWindow:
+    """Position p sees the last ``size`` positions one by one and, before them, whole blocks of ``pool`` positions as one
+    averaged key and value each. Keys of an unfinished block are kept until its average is formed."""
+
+    size: int
+    pool: int
+
+    def first(self, pos: int) -> int:
+        return max(0, min(pos - self.size + 1, pos // self.pool * self.pool))
+
+    @property
+    def span(self) -> int:
+        return max(self.size, self.pool)
+
+    def blocks_seen(self, pos: int) -> int:
+        """Averaged blocks that a token at ``pos`` sees."""
+        return max(0, pos - self.size + 1) // self.pool
+
+
+def as_mask(m):
+    """A chunk length stands for its ``Chunk``."""
+    return Chunk(m) if isinstance(m, int) else m
+
+
 @dataclass
 class ChunkView:
-    """Packed keys and values of one chunk length: rows of the portion, preceded by the rows of earlier positions that
-    the portion's first tokens still see (copied from the cache: ``gather_entry`` -> ``gather_row``)."""
+    """Packed keys and values of one mask: per sequence the averaged blocks (masks that pool: all complete ones, those that
+    this portion completes last), then the earlier positions that the portion's first tokens still see, then the portion.
+    Rows of earlier work are copied from the cache: ``gather_entry`` -> ``gather_row``."""
 
     rows: int
     kv_row: torch.Tensor        # [T] packed row of each token
@@ -26,6 +69,11 @@ class ChunkView:
     gather_row: torch.Tensor
     tiles: Optional[torch.Tensor] = None   # [n_tiles, 2]: portion, first row of the portion in the tile
     n_tiles: int = 0
+    pool_base: Optional[torch.Tensor] = None     # [n] row of each sequence's first averaged block
+    pool_src: Optional[torch.Tensor] = None      # blocks completed by this batch: row of the first token,
+    pool_row: Optional[torch.Tensor] = None      # row of the average,
+    pool_entry: Optional[torch.Tensor] = None    # cache entry of the average
+    n_pool: int = 0
 
 
 class RaggedBatch:
@@ -50,9 +98,11 @@ class RaggedBatch:
 
     @classmethod
     def prompt(cls, device, tokens: List[List[int]], pos0: List[int], slots: List[int], entries: List[List[int]],
-               earlier: Dict[int, List[List[int]]], want: List[int], tile_rows: int = 128) -> "RaggedBatch":
-        """``earlier[size][i]``: cache entries of the positions before sequence i's portion that lie in the same chunk of
-        that length. ``want``: rows whose logits are asked for."""
+               earlier: Dict[object, List[List[int]]], want: List[int], tile_rows: int = 128, averages=None) -> "RaggedBatch":
+        """``earlier[mask][i]``: cache entries of the positions before sequence i's portion that its first token still
+        needs (a chunk length may stand for its mask). ``averages[mask][i]``: for masks that pool, the cache entries of the
+        averaged blocks complete before the portion and of those that it completes. ``want``: rows whose logits are asked
+        for."""
         b = cls()
         b.n, b.T = len(tokens), sum(len(t) for t in tokens)
         lens = np.array([len(t) for t in tokens], dtype=np.int32)
@@ -72,22 +122,36 @@ class RaggedBatch:
         chunk_seq = np.repeat(np.arange(b.n, dtype=np.int32), per)
         parts += [chunk_seq, (np.arange(first[-1], dtype=np.int32) - first[chunk_seq]) * RECUR_CHUNK, first]
         b.n_chunks = int(first[-1])
-        sizes = sorted(earlier)
-        rows = []
-        for size in sizes:
-            carry = np.array([len(e) for e in earlier[size]], dtype=np.int32)
+        views, none = [], np.zeros(0, np.int32)
+        cat = lambda xs: np.concatenate([np.asarray(x, dtype=np.int32) for x in xs]) if xs else none  # noqa: E731
+        for key in earlier:
+            mask = as_mask(key)
+            carry = np.array([len(e) for e in earlier[key]], dtype=np.int32)
+            done, new = zip(*averages[key]) if mask.pool else ([()] * b.n, [()] * b.n)
+            n_done, n_new = (np.array([len(e) for e in x], dtype=np.int32) for x in (done, new))
             start = np.zeros(b.n + 1, dtype=np.int32)
-            np.cumsum(carry + lens, out=start[1:])
-            row0 = start[:-1] + carry                               # packed row of the portion's first token
-            parts += [row0[seq] + local, row0 - p0,
-                      np.concatenate([np.asarray(e, dtype=np.int32) for e in earlier[size]]) if carry.sum() else np.zeros(0, np.int32),
-                      np.concatenate([start[i] + np.arange(carry[i], dtype=np.int32) for i in range(b.n)])]
-            rows.append(int(start[-1]))
+            np.cumsum(n_done + n_new + carry + lens, out=start[1:])
+            kept = start[:-1] + n_done + n_new                      # packed row of the first earlier position
+            row0 = kept + carry                                     # packed row of the portion's first token
+            parts += [row0[seq] + local, row0 - p0, cat([e for i in range(b.n) for e in (done[i], earlier[key][i])]),
+                      cat([r for i in range(b.n) for r in (start[i] + np.arange(n_done[i]), kept[i] + np.arange(carry[i]))])]
+            if mask.pool:
+                first_new = p0 // mask.pool
+                assert (n_done == first_new).all() and (n_new == (p0 + lens) // mask.pool - first_new).all()
+                parts += [start[:-1],
+                          cat([row0[i] - p0[i] + (first_new[i] + np.arange(n_new[i])) * mask.pool for i in range(b.n)]),
+                          cat([start[i] + n_done[i] + np.arange(n_new[i]) for i in range(b.n)]), cat(list(new))]
+            views.append((key, int(start[-1]), int(n_new.sum())))
         dev = cls._upload(device, parts)
         b.ids, b.cu, b.pos0, b.slot, b.tok_seq, b.tok_pos, b.entry, b.want, tl, b.chunk_seq, b.chunk_start, b.chunk_first = dev[:12]
-        for i, size in enumerate(sizes):
-            r, base, ge, gr = dev[12 + 4 * i: 16 + 4 * i]
-            b.views[size] = ChunkView(rows[i], r, base, ge, gr, tl, len(tiles))
+        at = 12
+        for key, rows, n_pool in views:
+            v = b.views[key] = ChunkView(rows, *dev[at: at + 4], tl, len(tiles))
+            at += 4
+            if as_mask(key).pool:
+                v.pool_base, v.pool_src, v.pool_row, v.pool_entry = dev[at: at + 4]
+                v.n_pool = n_pool
+                at += 4
         if len(want) == b.T:
             b.want = None
         b.n_want = len(want)
@@ -109,10 +173,13 @@ class RaggedBatch:
         return [buf[o:o + len(p)] for p, o in zip(parts, offs)]
 
     @classmethod
-    def decode_layout(cls, n: int, width: int):
-        """Offsets of the decode arrays in one int32 buffer of ``length`` entries: (slices, length)."""
+    def decode_layout(cls, n: int, width: int, pools=(), pool_width: int = 0):
+        """Offsets of the decode arrays in one int32 buffer of ``length`` entries: (slices, length). ``pools``: block
+        lengths of the masks that pool, each with a table of ``pool_width`` cache blocks of averages."""
         names = [("ids", n), ("pos0", n), ("slot", n), ("entry", n), ("block_base", n), ("cu", n + 1), ("tok_seq", n),
                  ("block_table", n * width)]
+        for p in pools:
+            names += [(("pool_entry", p), n), (("pool_table", p), n * pool_width)]
         out, o = {}, 0
         for name, k in names:
             out[name] = slice(o, o + k)
@@ -120,21 +187,27 @@ class RaggedBatch:
         return out, max(o, 1)
 
     @classmethod
-    def decode_views(cls, buf: torch.Tensor, n: int, width: int) -> "RaggedBatch":
+    def decode_views(cls, buf: torch.Tensor, n: int, width: int, pools=(), pool_width: int = 0) -> "RaggedBatch":
         """Decode batch over a device buffer laid out by ``decode_layout``."""
-        lay, _ = cls.decode_layout(n, width)
+        lay, _ = cls.decode_layout(n, width, pools, pool_width)
         b = cls()
         b.n = b.T = b.n_want = n
         b.decode = True
+        b.pool_entry, b.pool_table, b.pool_width = {}, {}, pool_width
         for name, sl in lay.items():
-            setattr(b, name, buf[sl])
+            if isinstance(name, tuple):
+                getattr(b, name[0])[name[1]] = buf[sl]
+            else:
+                setattr(b, name, buf[sl])
         b.tok_pos, b.table_width = b.pos0, width
         return b
 
     @classmethod
-    def fill_decode(cls, hv, n: int, width: int, ids, pos, slots, entries, tables, bases) -> None:
-        """Writes the host side of a decode buffer; rows past the sequences given are padding (slot and entry -1)."""
-        lay, _ = cls.decode_layout(n, width)
+    def fill_decode(cls, hv, n: int, width: int, ids, pos, slots, entries, tables, bases, pools=None, pool_width: int = 0) -> None:
+        """Writes the host side of a decode buffer; rows past the sequences given are padding (slot and entry -1).
+        ``pools[length]``: (cache entry of the average that each token completes or -1, tables of averages)."""
+        pools = pools or {}
+        lay, _ = cls.decode_layout(n, width, tuple(pools), pool_width)
         k = len(ids)
         hv[:] = 0
         hv[lay["slot"]] = -1
@@ -143,7 +216,13 @@ class RaggedBatch:
             hv[lay[name].start: lay[name].start + k] = vals
         hv[lay["cu"]] = np.arange(n + 1, dtype=np.int32)
         hv[lay["tok_seq"]] = np.arange(n, dtype=np.int32)
-        if width:
-            bt = hv[lay["block_table"]].reshape(n, width)
-            for i, t in enumerate(tables):
+        grids = [("block_table", width, tables)] if width else []
+        for p, (done, tabs) in pools.items():
+            e = lay["pool_entry", p]
+            hv[e] = -1
+            hv[e.start: e.start + k] = done
+            grids.append((("pool_table", p), pool_width, tabs))
+        for name, w, rows in grids:
+            bt = hv[lay[name]].reshape(n, w)
+            for i, t in enumerate(rows):
                 bt[i, :len(t)] = t

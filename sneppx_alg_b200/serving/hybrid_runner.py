@@ -1,7 +1,7 @@
-"""Runs a hybrid decoder (recurrent layers and chunked attention, ``models/rilenex.py``) for the engine: prompts of any
-lengths packed into one ragged batch, portions of a prompt from the state earlier portions left, and decode steps that
-replay one CUDA graph per batch bucket. A sequence's memory is one state slot plus the cache blocks of its running chunk
-(``serving.kv_cache.HybridCache``)."""
+"""Runs a hybrid decoder (recurrent layers and attention of bounded reach, ``models/hybrid.py``) for the engine: prompts of
+any lengths packed into one ragged batch, portions of a prompt from the state earlier portions left, and decode steps that
+replay one CUDA graph per batch bucket. A sequence's memory is one state slot plus the cache blocks of the positions that
+its next token needs and of its averaged blocks (``serving.kv_cache.HybridCache``)."""
 from __future__ import annotations
 
 from typing import List, Sequence, Tuple
@@ -34,16 +34,20 @@ class HybridRunner:
             logits = self.decode([s for s, _, _ in entries], [t[0] for _, t, _ in entries])
             keep = [i for i, (_, _, want) in enumerate(entries) for _ in want]
             return logits if keep == list(range(len(entries))) else logits[keep]
-        cache, sizes = self.cache, self.cache.sizes
+        cache = self.cache
         pos0 = [cache.lens[s] for s, _, _ in entries]
-        earlier = {size: [cache.entries(s, p // size * size, p) for (s, _, _), p in zip(entries, pos0)] for size in sizes}
+        earlier = {m: [cache.entries(s, r.first(p), p) for (s, _, _), p in zip(entries, pos0)]
+                   for m, r in zip(cache.masks, cache.rules)}
         slots = [cache.reserve(s, len(t)) for s, t, _ in entries]
+        averages = {m: [(cache.average_entries(s, r.pool, 0, p // r.pool),
+                         cache.average_entries(s, r.pool, p // r.pool, (p + len(t)) // r.pool)) for (s, t, _), p in zip(entries, pos0)]
+                    for m, r in zip(cache.masks, cache.rules) if r.pool}
         want, row = [], 0
         for _, toks, w in entries:
             want += [row + (i if i >= 0 else len(toks) + i) for i in w]
             row += len(toks)
         batch = RaggedBatch.prompt(self.device, [t for _, t, _ in entries], pos0, [cache.slots[s] for s, _, _ in entries], slots,
-                                   earlier, want)
+                                   earlier, want, averages=averages)
         return self.model.step(batch, cache)
 
     def prefill(self, seq_id: int, tokens: List[int], start: int):
@@ -60,7 +64,8 @@ class HybridRunner:
     # ------------------------------------------------------------------ decode
     def enable_graphs(self, max_batch: int, max_len: int = 0):
         """Capture the decode step per batch bucket (1, 2, 4, .. max_batch). All inputs of a step sit in one int32 buffer
-        filled by one host -> device copy; its size depends on the chunk lengths only, not on how long sequences get."""
+        filled by one host -> device copy; its size depends on what the masks reach, not on how long sequences get, except
+        for the tables of averaged blocks, whose width is bucketed too (a graph is captured when one is outgrown)."""
         if self.device.type != "cuda":
             return
         self._buckets, b = [], 1
@@ -74,17 +79,18 @@ class HybridRunner:
         with static_weights():
             return self.model.step(batch, self.cache)
 
-    def _graph_for(self, n):
-        g = self._graphs.get(n)
+    def _graph_for(self, n, pool_width):
+        g = self._graphs.get((n, pool_width))
         if g is not None:
             return g
-        width = self.cache.table_width
-        _, length = RaggedBatch.decode_layout(n, width)
+        width, pools = self.cache.table_width, self.cache.pools
+        _, length = RaggedBatch.decode_layout(n, width, pools, pool_width)
         host = torch.zeros(length, dtype=torch.int32).pin_memory()
         hv = host.numpy()
-        RaggedBatch.fill_decode(hv, n, width, [], [], [], [], [], [])     # padding only: the warm-up writes no state
+        # padding only: the warm-up writes no state
+        RaggedBatch.fill_decode(hv, n, width, [], [], [], [], [], [], {p: ([], []) for p in pools}, pool_width)
         buf = host.to(self.device)
-        batch = RaggedBatch.decode_views(buf, n, width)
+        batch = RaggedBatch.decode_views(buf, n, width, pools, pool_width)
         side = torch.cuda.Stream(device=self.device)
         side.wait_stream(torch.cuda.current_stream())
         with torch.cuda.stream(side):
@@ -95,8 +101,13 @@ class HybridRunner:
         graph = torch.cuda.CUDAGraph()
         with torch.cuda.graph(graph, capture_error_mode="thread_local"):   # other threads (HTTP handlers) may call CUDA
             out = self._body(batch)
-        g = self._graphs[n] = dict(graph=graph, host=host, hv=hv, buf=buf, out=out)
+        g = self._graphs[n, pool_width] = dict(graph=graph, host=host, hv=hv, buf=buf, out=out)
         return g
+
+    def _pool_width(self, seq_ids) -> int:
+        """Blocks of averages per table: the longest table, up to a power of two."""
+        most = max((len(t[s]) for t in self.cache.averages.values() for s in seq_ids), default=0)
+        return max(4, 1 << (most - 1).bit_length()) if self.cache.pools else 0
 
     @torch.no_grad()
     def decode(self, seq_ids: List[int], last_tokens: List[int]):
@@ -104,17 +115,20 @@ class HybridRunner:
         cache, B, width = self.cache, len(seq_ids), self.cache.table_width
         pos = [cache.lens[s] for s in seq_ids]
         entries = [cache.reserve(s, 1)[0] for s in seq_ids]
+        pools = {p: ([cache.average_entries(s, p, q // p, q // p + 1)[0] if (q + 1) % p == 0 else -1 for s, q in zip(seq_ids, pos)],
+                     [cache.averages[p][s] for s in seq_ids]) for p in cache.pools}
+        pw = self._pool_width(seq_ids)
         args = (last_tokens, pos, [cache.slots[s] for s in seq_ids], entries, [cache.tables[s] for s in seq_ids],
-                [cache.base[s] for s in seq_ids])
+                [cache.base[s] for s in seq_ids], pools, pw)
         if self._graphs is not None and B <= self._buckets[-1]:
             n = next(b for b in self._buckets if b >= B)
-            g = self._graph_for(n)
+            g = self._graph_for(n, pw)
             torch.cuda.current_stream().synchronize()      # the previous step's copy has left the pinned buffer
             RaggedBatch.fill_decode(g["hv"], n, width, *args)
             g["buf"].copy_(g["host"], non_blocking=True)
             g["graph"].replay()
             return g["out"][:B].clone()
-        _, length = RaggedBatch.decode_layout(B, width)
+        _, length = RaggedBatch.decode_layout(B, width, cache.pools, pw)
         host = torch.zeros(length, dtype=torch.int32)
         RaggedBatch.fill_decode(host.numpy(), B, width, *args)
-        return self.model.step(RaggedBatch.decode_views(host.to(self.device), B, width), cache)
+        return self.model.step(RaggedBatch.decode_views(host.to(self.device), B, width, cache.pools, pw), cache)

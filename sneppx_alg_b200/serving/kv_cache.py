@@ -11,6 +11,8 @@ from typing import Dict, List, Optional, Tuple
 import numpy as np
 import torch
 
+from ..ops.ragged import as_mask
+
 
 class KVBlockPool:
     """Block id allocator with refcounts (shared prefixes) and copy-on-write."""
@@ -130,6 +132,10 @@ class PagedKVCache:
         """Most blocks a sequence of ``n_tokens`` holds at any time."""
         return (n_tokens + self.block_size - 1) // self.block_size
 
+    def blocks_held(self, seq_id: int) -> int:
+        """Blocks in the tables of a sequence."""
+        return len(self.tables.get(seq_id, ()))
+
     def available_blocks(self) -> int:
         """Free blocks plus those the prefix cache would give back."""
         return self.pool.num_free + (self.prefix.evictable() if self.prefix is not None else 0)
@@ -206,34 +212,54 @@ class PagedKVCache:
 
 
 class ChunkedKVCache(PagedKVCache):
-    """Paged cache of layers in which a position only sees its own chunk of positions (``sizes``: the chunk lengths that
-    occur). Positions behind the last visible one are never stored, and blocks that fall behind it go back to the pool,
-    so a sequence holds a bounded number of blocks however long it grows. Block tables start at block ``base[seq]``."""
+    """Paged cache of layers in which a position sees a bounded stretch of positions (``masks``: the masks that occur, see
+    ``ops.ragged``; an integer stands for chunks of that length). Positions behind the last needed one are never stored, and
+    blocks that fall behind it go back to the pool. Block tables start at block ``base[seq]``. Masks that average older blocks
+    of positions keep one entry per average; these live in blocks of the same pool, listed per block length in ``averages``,
+    and stay as long as the sequence. Without them a sequence holds a bounded number of blocks however long it grows."""
 
-    def __init__(self, layer_shapes, sizes, num_blocks, block_size, dtype=torch.bfloat16, device="cuda"):
+    def __init__(self, layer_shapes, masks, num_blocks, block_size, dtype=torch.bfloat16, device="cuda"):
         super().__init__(len(layer_shapes), num_blocks, block_size, dtype=dtype, device=device, enable_prefix_cache=False,
                          layer_shapes=layer_shapes)
-        self.sizes = sorted(set(sizes))
+        self.masks = list(dict.fromkeys(masks))
+        self.rules = [as_mask(m) for m in self.masks]
+        self.pools = tuple(sorted({m.pool for m in self.rules if m.pool}))
         self.base: Dict[int, int] = {}
+        self.averages: Dict[int, Dict[int, List[int]]] = {p: {} for p in self.pools}
+
+    @property
+    def sizes(self) -> List[int]:
+        """Most positions that each mask reaches back, ascending."""
+        return sorted(m.span for m in self.rules)
 
     @property
     def table_width(self) -> int:
-        """Blocks that the visible positions of one sequence can touch."""
-        return (self.sizes[-1] + self.block_size - 2) // self.block_size + 1 if self.sizes else 0
+        """Blocks that the stored positions of one sequence can touch."""
+        return (self.sizes[-1] + self.block_size - 2) // self.block_size + 1 if self.rules else 0
+
+    def average_blocks(self, n_tokens: int, pool: int) -> int:
+        """Cache blocks that hold the averages of ``n_tokens`` tokens in blocks of ``pool``."""
+        return (n_tokens // pool + self.block_size - 1) // self.block_size
 
     def blocks_for(self, n_tokens: int) -> int:
-        return min(super().blocks_for(n_tokens), self.table_width)
+        return min(super().blocks_for(n_tokens), self.table_width) + sum(self.average_blocks(n_tokens, p) for p in self.pools)
+
+    def blocks_held(self, seq_id: int) -> int:
+        return super().blocks_held(seq_id) + sum(len(t.get(seq_id, ())) for t in self.averages.values())
 
     def first_visible(self, pos: int) -> int:
-        """Earliest position that any layer still sees from ``pos``."""
-        return min(pos // s * s for s in self.sizes) if self.sizes else pos + 1
+        """Earliest position that any layer still needs at ``pos``."""
+        return min(m.first(pos) for m in self.rules) if self.rules else pos + 1
 
     def add_sequence(self, seq_id: int, tokens=None) -> int:
         self.tables[seq_id], self.lens[seq_id], self.base[seq_id] = [], 0, 0
+        for t in self.averages.values():
+            t[seq_id] = []
         return 0
 
     def reserve(self, seq_id: int, n_new: int) -> List[int]:
-        """Cache entries of the next ``n_new`` tokens; -1 for tokens that no later token sees."""
+        """Cache entries of the next ``n_new`` tokens; -1 for tokens that no later token needs. Also makes room for the
+        averages that these tokens complete."""
         n, table, base = self.lens[seq_id], self.tables[seq_id], self.base[seq_id]
         end = n + n_new
         keep = self.first_visible(end - 1)
@@ -246,8 +272,17 @@ class ChunkedKVCache(PagedKVCache):
         first = max(n, keep)
         while first < end and base + len(table) <= (end - 1) // self.block_size:   # first == end: no layer keeps keys
             table.append(self.pool.allocate())
+        for p, t in self.averages.items():
+            while len(t[seq_id]) < self.average_blocks(end, p):
+                t[seq_id].append(self.pool.allocate())
         self.base[seq_id], self.lens[seq_id] = base, end
         return [-1] * (first - n) + self.entries(seq_id, first, end)
+
+    def average_entries(self, seq_id: int, pool: int, lo: int, hi: int) -> List[int]:
+        """Entries of the averages of blocks [lo, hi) of ``pool`` positions."""
+        table, bs = self.averages[pool][seq_id], self.block_size
+        i = np.arange(lo, hi)
+        return (np.asarray(table, dtype=np.int64)[i // bs] * bs + i % bs).tolist() if hi > lo else []
 
     def entries(self, seq_id: int, lo: int, hi: int) -> List[int]:
         """Entries of the stored positions [lo, hi)."""
@@ -262,17 +297,20 @@ class ChunkedKVCache(PagedKVCache):
 
     def free_sequence(self, seq_id: int, tokens=None) -> None:
         self.base.pop(seq_id, None)
+        for t in self.averages.values():
+            for b in t.pop(seq_id, ()):
+                self.pool.release(b)
         super().free_sequence(seq_id)
 
 
 class HybridCache(ChunkedKVCache):
-    """Memory of models that mix recurrent layers and chunked attention: the block pool of the attention layers and one
+    """Memory of models that mix recurrent layers and attention of bounded reach: the block pool of the attention layers and one
     slot of fixed-size state per live sequence (``state_spec``: per layer, name -> (shape, dtype) of one slot). A slot is
     never cleared: the kernels start a sequence's first portion from an empty state whatever the slot holds."""
 
-    def __init__(self, kv_shapes, sizes, state_spec, max_sequences, num_blocks, block_size=16, dtype=torch.bfloat16,
+    def __init__(self, kv_shapes, masks, state_spec, max_sequences, num_blocks, block_size=16, dtype=torch.bfloat16,
                  device="cuda"):
-        super().__init__(kv_shapes, sizes, num_blocks, block_size, dtype, device)
+        super().__init__(kv_shapes, masks, num_blocks, block_size, dtype, device)
         self.free_slots = list(range(max_sequences - 1, -1, -1))
         self.slots: Dict[int, int] = {}
         self.state = [{k: torch.zeros(max_sequences, *shape, dtype=dt, device=device) for k, (shape, dt) in spec.items()}

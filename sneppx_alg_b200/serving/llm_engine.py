@@ -379,8 +379,8 @@ class LLMEngine:
         p = next(model.parameters())
         if runner is None and getattr(cfg, "architecture", "transformer") == "mamba2":
             runner = StatefulRunner(model)   # recurrent-state models: no KV cache, one state slot per sequence
-        if runner is None and getattr(cfg, "architecture", "transformer") == "rilenex":
-            # recurrent layers beside chunked attention: state slots and a block pool
+        if runner is None and hasattr(model, "init_cache"):
+            # hybrid decoders: recurrent layers beside attention of bounded reach, state slots and a block pool
             runner = HybridRunner(model, model.init_cache(max_batch_size, num_blocks, block_size))
         if isinstance(runner, StatefulRunner):
             self.cache = StateCache(max_batch_size, on_free=runner.release)
@@ -428,10 +428,9 @@ class LLMEngine:
     def _committed(self) -> int:
         """Blocks the running sequences may still claim before they finish (admission keeps these in hand, so a
         decode step never finds the pool empty)."""
-        tables = getattr(self.cache, "tables", None)
-        if tables is None:
+        if getattr(self.cache, "tables", None) is None:
             return 0
-        return sum(max(0, self._blocks_needed(r) - len(tables.get(r.req_id, ()))) for r in self.running.values())
+        return sum(max(0, self._blocks_needed(r) - self.cache.blocks_held(r.req_id)) for r in self.running.values())
 
     def _fail(self, req: Request, why: str):
         req.finish_time = time.perf_counter()

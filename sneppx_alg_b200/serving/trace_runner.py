@@ -15,10 +15,12 @@ import json
 import os
 import sys
 
+from ..ops.ragged import as_mask
+
 
 def _cache_size(model, max_tokens: int):
-    """State slots and cache blocks for ``max_tokens`` live tokens: a request holds at least one token and at most one
-    partly visible block more than its tokens fill."""
+    """State slots and cache blocks for ``max_tokens`` live tokens: a request holds at least one token, at most two partly
+    filled blocks of tokens, and for masks that average older blocks at most one partly filled block of averages."""
     slots = max(1, min(max_tokens, 256))
     per_slot = 0
     for layer in model.layers:
@@ -28,7 +30,8 @@ def _cache_size(model, max_tokens: int):
                 n *= s
             per_slot += n
     slots = max(1, min(slots, (8 << 30) // max(per_slot, 1)))
-    return slots, max_tokens // 16 + 2 * slots
+    pools = {as_mask(s[3]).pool for layer in model.layers for s in layer.mixer.kv_specs()} - {0}
+    return slots, max_tokens // 16 + 2 * slots + sum(max_tokens // (16 * p) + slots for p in pools)
 
 
 def main(argv=None) -> int:
