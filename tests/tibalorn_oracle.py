@@ -93,15 +93,16 @@ def block_visible(i, b, pool, size):
     return (b + 1) * pool - 1 <= i - size
 
 
-def pooled_window_attention(q, k, v, scale, temp, sink, size, pool):
+def pooled_window_attention(q, k, v, scale, temp, sink, size, pool, at=None):
     """q [T, H, d], k [T, G, d], v [T, G, dv] -> [T, H, dv]: the last ``size`` tokens one by one, earlier ones as means of
-    whole blocks of ``pool`` tokens, one softmax with exp(sink[h]) added to its denominator."""
+    whole blocks of ``pool`` tokens, one softmax with exp(sink[h]) added to its denominator. ``at``: only these positions (the others stay
+    zero)."""
     T, H, _ = q.shape
     G, NB = k.shape[1], T // pool
     kb = k[:NB * pool].view(NB, pool, *k.shape[1:]).mean(1)
     vb = v[:NB * pool].view(NB, pool, *v.shape[1:]).mean(1)
     out = torch.zeros(T, H, v.shape[2], dtype=q.dtype)
-    for i in range(T):
+    for i in (range(T) if at is None else at):
         js = [j for j in range(max(0, i - size + 1), i + 1) if token_visible(i, j, size)]
         bs = [b for b in range(NB) if block_visible(i, b, pool, size)]
         kk, vv = torch.cat([k[js], kb[bs]]), torch.cat([v[js], vb[bs]])
