@@ -7,7 +7,7 @@ seq 4096, micro-batch 1 per GPU, AdamW beta 0.9/0.95 wd 0.1), synthetic token id
     python bench.py --impl library ...                      # PyTorch library ops + NCCL only, overlapped like FSDP
     python bench.py --model deepseek-v2-lite --ep --micro-batch 2      # SER MoE, expert parallel + ZeRO-1
     python bench.py --model mamba2-2.7b --seq 8192 --tp 2              # Mamba-2, tensor parallel x data parallel
-    python bench.py --serve-hybrid                                     # serving: Rilenex beside Llama and Mamba-2 at equal size
+    python bench.py --serve-hybrid [rilenex|tibalorn]                  # serving: a hybrid decoder beside Llama and Mamba-2 at equal size
 
 Rank 0 prints one JSON line. ``value`` is whole-job tokens/s from CUDA-event timing (max over ranks);
 ``e2e`` repeats the measurement through the public engine API with the per-step host->device copy of the
@@ -47,8 +47,9 @@ def parse():
                     "fp8 (e4m3 data, 1x128 activation and 128x128 weight scales); backward stays bf16")
     ap.add_argument("--tp", type=int, default=1, help="tensor-parallel size (Mamba-2 models): ranks form world/tp "
                     "data-parallel replicas of tp consecutive ranks; ignored on one GPU")
-    ap.add_argument("--serve-hybrid", action="store_true", help="instead of the training step: prefill and decode throughput of "
-                    "the Rilenex design beside the closest existing models at equal size, and its kernels beside theirs")
+    ap.add_argument("--serve-hybrid", nargs="?", const="rilenex", choices=["rilenex", "tibalorn"], help="instead of the training step: "
+                    "prefill and decode throughput of a hybrid decoder beside the closest existing models at equal size, and its kernels "
+                    "beside theirs")
     return ap.parse_args()
 
 
@@ -288,8 +289,8 @@ def run_serve_hybrid(args):
     from sneppx_alg_b200.ops import _lib
     clocks = ClockSampler(int(os.environ.get("LOCAL_RANK", "0")))
     clocks.start()
-    out = hybrid_serving.main(["--steps", str(max(args.steps, 3))])
-    print(json.dumps({"metric": "serving throughput, Rilenex beside existing models", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
+    out = hybrid_serving.main(["--design", args.serve_hybrid, "--steps", str(max(args.steps, 3))])
+    print(json.dumps({"metric": f"serving throughput, {args.serve_hybrid.capitalize()} beside existing models", "dtype": "bf16", "data": "synthetic", "n_gpus": 1,
                       "gpu_launches": _lib.launch_count, "clocks": clocks.stop(), **out}))
     return 0
 

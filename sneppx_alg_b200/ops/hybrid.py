@@ -175,27 +175,40 @@ def ssd_scan_tc(act_dtype, P, N) -> bool:
     return act_dtype == torch.bfloat16 and bool(_lib.lib().sx_ssd_scan_ok(c_int(P), c_int(N)))
 
 
-def ssd_prompt(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch: RaggedBatch, H, P, N, G, taps):
-    """Portions through the SSD recurrence, from projected rows (z | x | B | C | dt) to gated read-outs in y."""
+def ssd_operands(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch: RaggedBatch, H, P, N, G, taps):
+    """Convolved x, B, C, step sizes and decays of the rows of a prompt batch, from projected rows (z | x | B | C | dt). Returns
+    what ``ssd_scan`` takes: the kernels' arguments and the tensors that they point to."""
     _need_cuda(u)
     T, dev = batch.T, u.device
-    tc = ssd_scan_tc(u.dtype, P, N)
     a = _ssd_args(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch, H, P, N, G, taps)
-    if tc:
+    if ssd_scan_tc(u.dtype, P, N):
         a.xp, a.np = (P + 7) // 8 * 8, (N + 7) // 8 * 8
     x = torch.empty(T, H * a.xp, dtype=u.dtype, device=dev)
-    b, c = torch.empty(2, T, G * a.np, dtype=u.dtype, device=dev)
+    b, c = torch.empty(2, T, (G * a.np + 7) // 8 * 8, dtype=u.dtype, device=dev)
     dt, la = torch.empty(2, T, H, dtype=torch.float32, device=dev)
     a.x, a.b, a.c, a.dt, a.la = x.data_ptr(), b.data_ptr(), c.data_ptr(), dt.data_ptr(), la.data_ptr()
     _lib.call("sx_ssd_operands", C.byref(a), stream())
-    conv_ring(u[:, H * P:], ring, batch, H * P + 2 * G * N, taps)
-    if tc:
+    return a, (u, x, b, c, dt, la, state, y, D)
+
+
+def ssd_scan(operands, batch: RaggedBatch):
+    """Walks every portion of the batch from its slot's state (empty at position 0), stores the state back and writes the gated
+    read-outs."""
+    a, (u, x, _, _, _, _, state, _, _) = operands
+    if ssd_scan_tc(u.dtype, a.P, a.N):
         _lib.call("sx_ssd_scan", C.byref(a), stream())
         return
-    rec = _records(batch, H, N, False, dev)
+    rec = _records(batch, a.H, a.N, False, u.device)
     _lib.call("sx_ssd_chunks", C.byref(a), ptr(rec), stream())
-    o = recur_scan(rec, x, state, batch, H, N, P, delta=False)
+    o = recur_scan(rec, x, state, batch, a.H, a.N, a.P, delta=False)
     _lib.call("sx_ssd_gate", C.byref(a), ptr(o), stream())
+
+
+def ssd_prompt(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch: RaggedBatch, H, P, N, G, taps):
+    """Portions through the SSD recurrence, from projected rows to gated read-outs in y."""
+    operands = ssd_operands(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch, H, P, N, G, taps)
+    conv_ring(u[:, H * P:], ring, batch, H * P + 2 * G * N, taps)
+    ssd_scan(operands, batch)
 
 
 def ssd_step(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch: RaggedBatch, H, P, N, G, taps):

@@ -38,7 +38,7 @@ ODD = config(72, 101, [
     attention(3, 3, 17, 22, 7, 16, 16, 0.4, 1e4),
     mamba2(3, 7, 33, 1, 1, 3),
 ], eps=1e-3, scale=1.7, cap=9.0)
-# sizes that the tensor-core kernels take
+# sizes that the tensor-core kernels take; an epsilon at which rows that nearly cancel do not amplify bf16 rounding
 TENSOR = config(128, 160, [
     mamba2(4, 64, 128, 2, 4, 4),
     attention(8, 2, 64, 64, 48, 8, 32, 0.2, 1e5, yarn(8.0, 256, 16.0, 2.0), 96),
@@ -46,7 +46,7 @@ TENSOR = config(128, 160, [
     attention(20, 1, 40, 72, 130, 3, 40, 0.25),
     mamba2(2, 32, 200, 2, 4, 2),
     attention(4, 2, 136, 128, 5, 2, 0, 0.1),
-], scale=0.8)
+], eps=2e-2, scale=0.8)
 CONFIGS = {"odd": ODD, "tensor": TENSOR}
 
 
