@@ -83,7 +83,7 @@ __global__ void __launch_bounds__(256) ssd_gate_kernel(const SsdParams P, const 
 // One CTA per (head, sequence). Threads own VEC columns of the state and walk its rows; the rows of a warp are summed by
 // shuffles, the warps through shared memory.
 template <typename A, int VEC>
-__global__ void __launch_bounds__(256) ssd_step_kernel(const SsdParams P, int lpr) {
+__global__ void __launch_bounds__(256, 3) ssd_step_kernel(const SsdParams P, int lpr) {
   const SxSsdArgs& p = P.a;
   extern __shared__ __align__(16) float sm[];
   const int N = p.N, W = p.P;
@@ -100,9 +100,27 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const SsdParams P, int lp
   A* ring = reinterpret_cast<A*>(p.ring) + (long long)slot * p.taps * C;
   const float dt = softplus_f(to_f(u[inner + C + h]) + p.dt_bias[h]);
   const float decay = pos == 0 ? 0.f : expf(-expf(p.a_log[h]) * dt);
-  // rows of the state that this thread loads first: in flight while the convolutions run
   const int rows = 256 / lpr, r0 = tid / lpr, cv = W / VEC;
   float* st = p.state + ((long long)slot * p.H + h) * N * W;
+  float S[8][VEC];
+  auto load = [&](int c, int n0) {        // up to 8 rows of the state, all loads in flight together
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      const int n = n0 + k * rows;
+#pragma unroll
+      for (int e = 0; e < VEC; ++e) S[k][e] = 0.f;
+      if (c < cv && n < N && pos != 0) {
+        const float* s = st + (long long)n * W + c * VEC;
+        if constexpr (VEC == 4) {
+          const float4 v = __ldcs(reinterpret_cast<const float4*>(s));
+          S[k][0] = v.x; S[k][1] = v.y; S[k][2] = v.z; S[k][3] = v.w;
+        } else {
+          S[k][0] = *s;
+        }
+      }
+    }
+  };
+  load(tid % lpr, r0);                    // arrives while the convolutions run
   for (int i = tid; i < W + 2 * N; i += 256) {
     const int which = i < W ? 0 : (i - W) / N, n = i < W ? i : (i - W) % N;
     const int col = i < W ? h * W + i : inner + (which * p.G + g) * N + n;
@@ -128,22 +146,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const SsdParams P, int lp
       xv[e] = ok ? sx[c * VEC + e] : 0.f;
     }
     for (int n0 = r0; n0 < N; n0 += 8 * rows) {
-      float S[8][VEC];
-#pragma unroll
-      for (int k = 0; k < 8; ++k) {
-        const int n = n0 + k * rows;
-#pragma unroll
-        for (int e = 0; e < VEC; ++e) S[k][e] = 0.f;
-        if (ok && n < N && pos != 0) {
-          const float* s = st + (long long)n * W + c * VEC;
-          if constexpr (VEC == 4) {
-            const float4 v = __ldcs(reinterpret_cast<const float4*>(s));
-            S[k][0] = v.x; S[k][1] = v.y; S[k][2] = v.z; S[k][3] = v.w;
-          } else {
-            S[k][0] = *s;
-          }
-        }
-      }
+      if (cb > 0 || n0 > r0) load(c, n0);
 #pragma unroll
       for (int k = 0; k < 8; ++k) {
         const int n = n0 + k * rows;

@@ -24,6 +24,28 @@ __device__ __forceinline__ int2 pair_at(int m, int n, int interleaved) {
   return interleaved ? make_int2(2 * m, 2 * m + 1) : make_int2(m, m + n);
 }
 
+// Decoding: the block of p.pool positions that the row of sequence `seq` at `pos` completes becomes an average in the cache.
+// All threads of the CTA that appended the row take part.
+template <typename A>
+__device__ __forceinline__ void win_pool_step(const SxWinPrepArgs& p, int seq, int pos) {
+  if (!p.pool_entry) return;
+  const int done = p.pool_entry[seq];
+  if (done < 0) return;
+  __syncthreads();                            // this row's entry is in the cache
+  const int* table = p.block_table + (long long)seq * p.table_ld;
+  const int first = pos - p.pool + 1, b0 = p.block_base[seq], G = p.G, d = p.d, dv = p.dv;
+  for (int i = threadIdx.x; i < G * (d + dv); i += blockDim.x) {
+    const bool is_v = i >= G * d;
+    const int wd = is_v ? G * dv : G * d, c = is_v ? i - G * d : i;
+    A* cache = reinterpret_cast<A*>(is_v ? p.v_cache : p.k_cache);
+    float s = 0.f;
+#pragma unroll 4
+    for (int j = first; j <= pos; ++j)
+      s += to_f(cache[((long long)table[j / p.block_size - b0] * p.block_size + j % p.block_size) * wd + c]);
+    cache[(long long)done * wd + c] = from_f<A>(s / p.pool);
+  }
+}
+
 // ------------------------------------------------------------------ operands: one CTA per row
 template <typename A>
 __global__ void __launch_bounds__(256) win_prep_kernel(const WinPrepParams P) {
@@ -114,21 +136,103 @@ __global__ void __launch_bounds__(256) win_prep_kernel(const WinPrepParams P) {
     const int pad = p.q_ld - d;
     for (int i = tid; i < H * pad; i += 256) q[(i / pad) * p.q_ld + d + i % pad] = from_f<A>(0.f);
   }
-  if (!p.pool_entry) return;
-  const int done = p.pool_entry[seq];
-  if (done < 0) return;
-  __syncthreads();                            // this row's entry is in the cache
-  const int* table = p.block_table + (long long)seq * p.table_ld;
-  const int first = pos - p.pool + 1, b0 = p.block_base[seq];
-  for (int i = tid; i < G * (d + dv); i += 256) {
-    const bool is_v = i >= G * d;
-    const int wd = is_v ? G * dv : G * d, c = is_v ? i - G * d : i;
-    A* cache = reinterpret_cast<A*>(is_v ? p.v_cache : p.k_cache);
-    float s = 0.f;
-    for (int j = first; j <= pos; ++j)
-      s += to_f(cache[((long long)table[j / p.block_size - b0] * p.block_size + j % p.block_size) * wd + c]);
-    cache[(long long)done * wd + c] = from_f<A>(s / p.pool);
+  win_pool_step<A>(p, seq, pos);
+}
+
+// ------------------------------------------------------------------ the same with 16-byte pieces (bf16, halves)
+// One CTA: NT rows. A thread keeps its piece of the row (8 pairs, or 8 entries that pass unchanged) for all of them, so that
+// biases are read once and the loads of all rows are in flight together.
+template <int NT>
+__global__ void __launch_bounds__(256, 3) win_prep_vec_kernel(const WinPrepParams P) {
+  using bf = __nv_bfloat16;
+  const SxWinPrepArgs& p = P.a;
+  extern __shared__ __align__(16) float sm[];
+  const int t0 = blockIdx.x * NT, tid = threadIdx.x, n = blockDim.x, nt = min(NT, p.T - t0);
+  const int d = p.d, dv = p.dv, nr = p.rot / 2, nv = dv / 2, H = p.H, G = p.G;
+  float2* cs = reinterpret_cast<float2*>(sm); // [NT][nr + nv] cos, sin; those of queries and keys with their factor
+  const int wq = nr / 8 + (d - p.rot) / 8, wv = nv / 8, items = (H + G) * wq + G * wv;
+  bf16x8 x[NT], y[NT];
+  bool is_v, pair;
+  int h, a0, a1, base;                        // head, its two pieces' columns, its first column in the row
+  auto load = [&](int i) {
+    is_v = i >= (H + G) * wq;
+    const int j = is_v ? i - (H + G) * wq : i, w = is_v ? wv : wq, e = j % w;
+    h = j / w;
+    pair = is_v || e < nr / 8;
+    a0 = pair ? e * 8 : p.rot + (e - nr / 8) * 8;
+    a1 = a0 + (is_v ? nv : nr);
+    base = is_v ? (H + G) * d + h * dv : h * d;
+    const bf* u = reinterpret_cast<const bf*>(p.u) + (long long)t0 * p.u_ld + base;
+#pragma unroll
+    for (int t = 0; t < NT; ++t)
+      if (t < nt) {
+        x[t] = ld8(u + t * p.u_ld + a0);
+        y[t] = ld8(u + t * p.u_ld + (pair ? a1 : a0));
+      }
+  };
+  if (tid < items) load(tid);                 // arrives while the angles are worked out
+#pragma unroll
+  for (int t = 0; t < NT; ++t) {
+    if (t >= nt) break;
+    const int pos = P.rv.tok_pos[t0 + t];
+    for (int e = tid; e < nr + nv; e += n) {
+      float c, s;
+      turn_angle(e < nr ? p.freq[e] : p.vfreq[e - nr], pos, &c, &s, false);
+      cs[t * (nr + nv) + e] = e < nr ? make_float2(c * p.rot_mul, s * p.rot_mul) : make_float2(c, s);
+      if (e >= nr) reinterpret_cast<float2*>(p.turn)[(long long)(t0 + t) * nv + e - nr] = make_float2(c, s);
+    }
   }
+  __syncthreads();
+  for (int i = tid; i < items; i += n) {
+    if (i != tid) load(i);
+    float bx[8], by[8];
+#pragma unroll
+    for (int k = 0; k < 8; ++k) {
+      bx[k] = p.bias ? p.bias[base + a0 + k] : 0.f;
+      by[k] = p.bias && pair ? p.bias[base + a1 + k] : 0.f;
+    }
+    const float f = !is_v && h < H && p.temp ? p.temp[h] : 1.f;
+#pragma unroll
+    for (int t = 0; t < NT; ++t) {
+      if (t >= nt) break;
+      const int row = t0 + t;
+      if (P.rv.slot[P.rv.tok_seq[row]] < 0) continue;            // padding row of a captured launch
+      float a[8], b[8];
+      unpack8(x[t], a);
+      unpack8(y[t], b);
+      const float2* c = cs + t * (nr + nv) + (is_v ? nr : 0) + a0;
+#pragma unroll
+      for (int k = 0; k < 8; ++k) {
+        const float u0 = a[k] + bx[k], u1 = b[k] + by[k];
+        if (pair) {
+          const float2 q = c[k];
+          a[k] = (u0 * q.x - u1 * q.y) * f;
+          b[k] = (u1 * q.x + u0 * q.y) * f;
+        } else {
+          a[k] = u0 * f;
+        }
+      }
+      const bf16x8 oa = pack8(a), ob = pack8(b);
+      auto put = [&](bf* dst) {
+        st8(dst + a0, oa);
+        if (pair) st8(dst + a1, ob);
+      };
+      if (!is_v && h < H) {
+        put(reinterpret_cast<bf*>(p.q) + ((long long)row * H + h) * p.q_ld);
+      } else {
+        const int g = is_v ? h : h - H, entry = p.cache_entry[row];
+        bf* out = reinterpret_cast<bf*>(is_v ? p.v_out : p.k_out);
+        if (out) put(out + (long long)(p.kv_row ? p.kv_row[row] : row) * (is_v ? p.v_ld : p.k_ld) + g * (is_v ? p.dvp : p.dp));
+        if (entry >= 0) put(reinterpret_cast<bf*>(is_v ? p.v_cache : p.k_cache) + ((long long)entry * G + g) * (is_v ? dv : d));
+      }
+    }
+  }
+  if (p.q_ld > d) {
+    const int pad = (p.q_ld - d) / 8;
+    for (int i = tid; i < nt * H * pad; i += n)
+      *reinterpret_cast<uint4*>(reinterpret_cast<bf*>(p.q) + ((long long)t0 * H + i / pad) * p.q_ld + d + i % pad * 8) = make_uint4(0, 0, 0, 0);
+  }
+  if (NT == 1 && P.rv.slot[P.rv.tok_seq[t0]] >= 0) win_pool_step<bf>(p, P.rv.tok_seq[t0], P.rv.tok_pos[t0]);
 }
 
 // ------------------------------------------------------------------ averages of the blocks that a prompt batch completes
@@ -270,7 +374,18 @@ extern "C" int sx_win_prep(const SxWinPrepArgs* a, cudaStream_t st) {
   if (a->d <= 0 || a->dv <= 0 || a->dv % 2 || a->rot % 2 || a->rot > a->d || a->G <= 0 || a->H % a->G) return -1;
   const WinPrepParams p{*a, view(&a->ragged)};
   const int smem = (a->rot + a->dv) * 4;
-  if (smem > 48 * 1024) return -2;
+  if (smem > 12 * 1024) return -2;
+  const auto al = [](const void* x) { return (reinterpret_cast<uintptr_t>(x) & 15) == 0; };
+  const bool vec = !a->f32 && !a->interleaved && a->q && !a->q32 && a->rot % 16 == 0 && a->d % 8 == 0 && a->dv % 16 == 0 && a->u_ld % 8 == 0 &&
+                   a->q_ld % 8 == 0 && al(a->u) && al(a->q) && al(a->k_cache) && al(a->v_cache) &&
+                   (!a->k_out || (al(a->k_out) && al(a->v_out) && a->k_ld % 8 == 0 && a->v_ld % 8 == 0 && a->dp % 8 == 0 && a->dvp % 8 == 0));
+  if (vec) {
+    const int items = (a->H + a->G) * (a->d - a->rot / 2) / 8 + a->G * a->dv / 16;
+    const int threads = items >= 256 ? 256 : items <= 32 ? 32 : (items + 31) / 32 * 32;
+    if (a->T >= 4 * 148 && !a->pool_entry) win_prep_vec_kernel<4><<<(a->T + 3) / 4, threads, 4 * smem, st>>>(p);
+    else win_prep_vec_kernel<1><<<a->T, threads, smem, st>>>(p);
+    return last_rc();
+  }
   SX_ACT_DISPATCH(a->f32, (win_prep_kernel<A><<<a->T, 256, smem, st>>>(p)));
   return last_rc();
 }

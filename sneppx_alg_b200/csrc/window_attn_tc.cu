@@ -1,11 +1,12 @@
 // Prompt form of window attention over tokens and averaged blocks on tcgen05 (bf16); see window_attn.cu.
 //
-// One CTA serves 128 query rows of one portion for one head. It walks 128-key tiles, first those of the averaged blocks that
-// its last row sees, then those of the tokens from its first row's window on, in two interleaved streams (even and odd
-// tiles), each with its own scores, probabilities and output accumulator in TMEM and its own softmax warpgroup, so the tensor
-// pipe works on one stream while the other does its softmax. The streams and the sink are merged at the end, where the
-// outputs are also turned back by their row's angles and gated.
-//   S_x = Q K^T           over d in slices of 64: K by TMA in a ring of two-slice stages, Q resident in shared memory
+// One CTA serves 128 query rows of one portion. It walks 128-key tiles, first those of the averaged blocks that its last row
+// sees, then those of the tokens from its first row's window on, in two streams, each with its own scores, probabilities and
+// output accumulator in TMEM and its own softmax warpgroup, so the tensor pipe works on one stream while the other does its
+// softmax. PAIR: the streams are two heads of the same key head, which see the same keys, so every K and V tile is loaded once
+// for both. Otherwise (an odd number of heads per key head) they are the even and the odd tiles of one head, merged at the end.
+// The end also adds the sink, turns the outputs back by their row's angles and gates them.
+//   S_x = Q_x K^T         over d in slices of 64: K by TMA in a ring of two-slice stages, Q resident in shared memory
 //   P_x = exp2(S_x - m)   one query row per thread; packed bf16 over the S columns
 //   O_x += P_x V          tcgen05.mma TS, V MN-major
 // Keys are rows of a packed buffer: per sequence its averaged blocks, then its tokens in position order.
@@ -29,13 +30,15 @@ struct WinTcParams {
   float scale_log2;
 };
 
-template <bool INTER>
+// NQ: slices of a query row, 0 when only known at run time.
+template <bool INTER, bool PAIR, int NQ>
 __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_constant__ WinTcParams p) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int stage_bytes = 2 * WT_SLICE;
+  constexpr int stage_bytes = 2 * WT_SLICE;
+  const int nq = NQ ? NQ : p.nq;
   uint8_t* sQ = smem;
-  uint8_t* sR = smem + p.nq * WT_SLICE;
+  uint8_t* sR = smem + (PAIR ? 2 : 1) * nq * WT_SLICE;
   uint64_t* bars = reinterpret_cast<uint64_t*>(sR + p.stages * stage_bytes);
   uint64_t* full = bars;                       // [stages]
   uint64_t* empty = bars + WT_MAX_STAGES;      // [stages]
@@ -49,7 +52,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
 
   const SxWinAttnArgs& a = p.a;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int tile = a.n_tiles - 1 - blockIdx.y, head = blockIdx.x;
+  const int tile = a.n_tiles - 1 - blockIdx.y, head0 = PAIR ? 2 * blockIdx.x : blockIdx.x;
   const int seq = a.tiles[2 * tile], r0 = a.tiles[2 * tile + 1];
   const int cu = p.rv.cu[seq], len = p.rv.cu[seq + 1] - cu, pos0 = p.rv.pos0[seq];
   const int t0 = cu + r0;
@@ -58,7 +61,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
   const int n_blk = (k_last.blocks + WT_BN - 1) / WT_BN;                        // tiles of averaged blocks
   const int n_steps = n_blk + (p_last - k_first.first) / WT_BN + 1;
   const int blk_row = a.pool_base[seq], tok_row = a.kv_base[seq] + k_first.first;
-  const int kvh = head / (a.H / a.G);
+  const int kvh = head0 / (a.H / a.G);
   const int nv = (a.dv + 63) / 64;             // V slices
 
   if (threadIdx.x == 0) {
@@ -84,11 +87,13 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
   tc_fence_after();
   const uint32_t tmem_base = *tmem_slot;
 
-  // order of the ring: K(0), K(1), then V(j), K(j + 2) for j = 0, 1, ..
+  // order of the ring. PAIR: K(0), then V(j), K(j + 1) for j = 0, 1, ..; else K(0), K(1), then V(j), K(j + 2)
+  constexpr int AHEAD = PAIR ? 1 : 2;
   if (warp == 0) {
     if (lane == 0) {
-      mbar_expect_tx(q_full, p.nq * WT_SLICE);
-      for (int c = 0; c < p.nq; ++c) tma_load_2d(sQ + c * WT_SLICE, &p.tmQ, q_full, (head * p.nq + c) * 64, t0);
+      const int n_q = (PAIR ? 2 : 1) * nq;
+      mbar_expect_tx(q_full, n_q * WT_SLICE);
+      for (int c = 0; c < n_q; ++c) tma_load_2d(sQ + c * WT_SLICE, &p.tmQ, q_full, (head0 * nq + c) * 64, t0);
       int it = 0;
       bool ok = true;
       auto slot = [&](int bytes) -> int {      // waits for a free stage and announces `bytes`
@@ -101,21 +106,20 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
       auto row_of = [&](int j) { return j < n_blk ? blk_row + j * WT_BN : tok_row + (j - n_blk) * WT_BN; };
       auto load_k = [&](int j) {
         const int row = row_of(j);
-        for (int c = 0; c < p.nq && ok; c += 2) {
-          const int w = min(2, p.nq - c);
+        for (int c = 0; c < nq && ok; c += 2) {
+          const int w = min(2, nq - c);
           const int s = slot(w * WT_SLICE);
           if (!ok) return;
           for (int e = 0; e < w; ++e) tma_load_2d(sR + s * stage_bytes + e * WT_SLICE, &p.tmK, &full[s], kvh * a.dp + (c + e) * 64, row);
         }
       };
-      load_k(0);
-      if (n_steps > 1 && ok) load_k(1);
+      for (int j = 0; j < AHEAD && j < n_steps && ok; ++j) load_k(j);
       for (int j = 0; j < n_steps && ok; ++j) {
         const int s = slot(nv * WT_SLICE);
         if (!ok) break;
         const int row = row_of(j);
         for (int e = 0; e < nv; ++e) tma_load_2d(sR + s * stage_bytes + e * WT_SLICE, &p.tmV, &full[s], kvh * a.dvp + e * 64, row);
-        if (j + 2 < n_steps) load_k(j + 2);
+        if (j + AHEAD < n_steps) load_k(j + AHEAD);
       }
     }
   } else if (warp == 1) {
@@ -130,42 +134,91 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
         ++it;
         return s;
       };
-      auto issue_qk = [&](int j) {
-        const uint32_t d = tmem_base + (j & 1) * 256;
-        for (int c = 0; c < p.nq; c += 2) {
-          const int s = stage();
-          if (!ok) return;
-          tc_fence_after();
-          const uint32_t b0 = smem_u32(sR + s * stage_bytes), a0 = smem_u32(sQ + c * WT_SLICE);
-          for (int e = 0; e < 2 && c + e < p.nq; ++e)
+      // descriptors: an offset in bytes is added in units of 16 (addresses stay inside the 14-bit field)
+      const uint64_t q_desc = umma_desc_sw128(smem_u32(sQ), 16, 1024), k_desc = umma_desc_sw128(smem_u32(sR), 16, 1024);
+      const uint64_t v_desc = umma_desc_sw128(smem_u32(sR), WT_SLICE, 1024);
+      // scores for stream x: query slices c, c + 1 with the K slices of stage s
+      auto qk = [&](int x, int c, int s) {
+        const uint32_t d = tmem_base + x * 256;
+        const uint64_t qd = q_desc + (((PAIR ? x * nq : 0) + c) * WT_SLICE >> 4), kd = k_desc + (s * stage_bytes >> 4);
 #pragma unroll
-            for (int k = 0; k < 4; ++k)
-              umma_f16_ss(d, umma_desc_sw128(a0 + e * WT_SLICE + k * 32, 16, 1024), umma_desc_sw128(b0 + e * WT_SLICE + k * 32, 16, 1024),
-                          idesc_qk, (c | e | k) ? 1u : 0u);
-          umma_commit(&empty[s]);
+        for (int e = 0; e < 2; ++e) {
+          if (c + e >= nq) break;
+#pragma unroll
+          for (int k = 0; k < 4; ++k)
+            umma_f16_ss(d, qd + ((e * WT_SLICE + k * 32) >> 4), kd + ((e * WT_SLICE + k * 32) >> 4), idesc_qk, (c | e | k) ? 1u : 0u);
         }
-        umma_commit(&s_full[j & 1]);
+      };
+      auto pv = [&](int x, int s, bool first) {
+        const uint32_t dO = tmem_base + x * 256 + 128, aP = tmem_base + x * 256;
+        const uint64_t vd = v_desc + (s * stage_bytes >> 4);
+#pragma unroll
+        for (int k = 0; k < 8; ++k) umma_f16_ts(dO, aP + k * 8, vd + (k * 2048 >> 4), idesc_pv, (!first || k) ? 1u : 0u);
       };
       ok = mbar_wait(q_full, 0, s_abort, a.status, ST_TIMEOUT_MMA);
-      if (ok) {
-        tc_fence_after();
-        issue_qk(0);
-      }
-      if (ok && n_steps > 1) issue_qk(1);
-      for (int j = 0; j < n_steps && ok; ++j) {
-        const int x = j & 1;
-        const int s = stage();
-        if (!ok) break;
-        if (!mbar_wait(&p_full[x], (j >> 1) & 1, s_abort, a.status, ST_TIMEOUT_MMA)) break;
-        tc_fence_after();
-        const uint32_t b0 = smem_u32(sR + s * stage_bytes);
-        const uint32_t dO = tmem_base + x * 256 + 128, aP = tmem_base + x * 256;
-#pragma unroll
-        for (int k = 0; k < 8; ++k)
-          umma_f16_ts(dO, aP + k * 8, umma_desc_sw128(b0 + k * 2048, WT_SLICE, 1024), idesc_pv, (j > 1 || k) ? 1u : 0u);
-        umma_commit(&empty[s]);
-        if (j + 2 >= n_steps) umma_commit(&o_done[x]);   // last step of this stream
-        if (j + 2 < n_steps) issue_qk(j + 2);
+      if (ok) tc_fence_after();
+      if constexpr (PAIR) {
+        int k0 = 0, k1 = 0;                    // stages of the K tile in turn
+        auto k_stages = [&]() {
+          k0 = stage();
+          if (nq > 2 && ok) k1 = stage();
+          if (ok) tc_fence_after();
+        };
+        auto qk_all = [&](int x) {
+          qk(x, 0, k0);
+          if (nq > 2) qk(x, 2, k1);
+          umma_commit(&s_full[x]);
+        };
+        auto k_release = [&]() {
+          umma_commit(&empty[k0]);
+          if (nq > 2) umma_commit(&empty[k1]);
+        };
+        if (ok) k_stages();
+        if (ok) {
+          qk_all(0);
+          qk_all(1);
+          k_release();
+        }
+        for (int j = 0; j < n_steps && ok; ++j) {
+          const bool more = j + 1 < n_steps;
+          const int s = stage();
+          if (ok && more) k_stages();
+          for (int x = 0; x < 2 && ok; ++x) {
+            ok = mbar_wait(&p_full[x], j & 1, s_abort, a.status, ST_TIMEOUT_MMA);
+            if (!ok) break;
+            tc_fence_after();
+            pv(x, s, j == 0);
+            if (more) qk_all(x);
+            else umma_commit(&o_done[x]);
+          }
+          if (!ok) break;
+          umma_commit(&empty[s]);
+          if (more) k_release();
+        }
+      } else {
+        auto issue_qk = [&](int j) {
+          for (int c = 0; c < nq; c += 2) {
+            const int s = stage();
+            if (!ok) return;
+            tc_fence_after();
+            qk(j & 1, c, s);
+            umma_commit(&empty[s]);
+          }
+          umma_commit(&s_full[j & 1]);
+        };
+        if (ok) issue_qk(0);
+        if (ok && n_steps > 1) issue_qk(1);
+        for (int j = 0; j < n_steps && ok; ++j) {
+          const int x = j & 1;
+          const int s = stage();
+          if (!ok) break;
+          if (!mbar_wait(&p_full[x], (j >> 1) & 1, s_abort, a.status, ST_TIMEOUT_MMA)) break;
+          tc_fence_after();
+          pv(x, s, j < 2);
+          umma_commit(&empty[s]);
+          if (j + 2 >= n_steps) umma_commit(&o_done[x]);   // last step of this stream
+          if (j + 2 < n_steps) issue_qk(j + 2);
+        }
       }
     }
   } else {
@@ -179,13 +232,15 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
     const WinKeys mine = win_keys(p_first + row, a.size, a.pool);
     float m_used = -INFINITY, l = 0.f;
     bool ok = true;
-    for (int j = x; j < n_steps; j += 2) {
+    const int head = head0 + (PAIR ? x : 0);
+    int cnt = 0;                            // steps of this stream so far
+    for (int j = PAIR ? 0 : x; j < n_steps; j += PAIR ? 1 : 2, ++cnt) {
       // key index of column 0, the indices that this row sees, and whether some row of the tile misses a column
       const bool is_blk = j < n_blk;
       const int kv0 = is_blk ? j * WT_BN : k_first.first + (j - n_blk) * WT_BN;
       const int lo = is_blk ? 0 : mine.first, hi = row_ok ? (is_blk ? mine.blocks : p_first + row + 1) : INT_MIN;
       const bool need_mask = r0 + WT_BM > len || (is_blk ? kv0 + WT_BN > k_first.blocks : kv0 + WT_BN - 1 > p_first || kv0 < k_last.first);
-      if (!mbar_wait_warp(&s_full[x], (j >> 1) & 1, s_abort, a.status, ST_TIMEOUT_EPILOGUE)) { ok = false; break; }
+      if (!mbar_wait_warp(&s_full[x], cnt & 1, s_abort, a.status, ST_TIMEOUT_EPILOGUE)) { ok = false; break; }
       tc_fence_after();
       uint32_t r[WT_BN];
 #pragma unroll
@@ -224,7 +279,7 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
       }
       l += lsum;
       // s_full(j) was committed after P V of this stream's previous step (in-order pipe): O and the S / P columns are ours
-      if (j > 1 && __any_sync(0xffffffffu, rescale)) {
+      if (cnt > 0 && __any_sync(0xffffffffu, rescale)) {
 #pragma unroll 1
         for (int c = 0; c < (a.dv + 31) / 32; ++c) {
           uint32_t o[32];
@@ -242,16 +297,21 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
       __syncwarp();
       if (lane == 0) mbar_arrive(&p_full[x]);
     }
-    const int n_streams = n_steps > 1 ? 2 : 1;
-    for (int s = 0; s < n_streams && ok; ++s) ok = mbar_wait_warp(&o_done[s], 0, s_abort, a.status, ST_TIMEOUT_EPILOGUE);
-    if (ok) {      // every load has been consumed: the ring is free
-      s_ml[x * 2 * WT_BN + row] = m_used;
-      s_ml[(x * 2 + 1) * WT_BN + row] = l;
+    const int n_streams = !PAIR && n_steps > 1 ? 2 : 1;      // accumulators that make up an output
+    if constexpr (PAIR) {
+      if (ok) ok = mbar_wait_warp(&o_done[x], 0, s_abort, a.status, ST_TIMEOUT_EPILOGUE);
+    } else {
+      for (int s = 0; s < n_streams && ok; ++s) ok = mbar_wait_warp(&o_done[s], 0, s_abort, a.status, ST_TIMEOUT_EPILOGUE);
+      if (ok) {      // every load has been consumed: the ring is free
+        s_ml[x * 2 * WT_BN + row] = m_used;
+        s_ml[(x * 2 + 1) * WT_BN + row] = l;
+      }
+      asm volatile("bar.sync 1, 256;" ::: "memory");      // the eight softmax warps
     }
-    asm volatile("bar.sync 1, 256;" ::: "memory");      // the eight softmax warps
     if (ok) {
       tc_fence_after();
-      const float m0 = s_ml[row], l0 = s_ml[WT_BN + row], m1 = s_ml[2 * WT_BN + row], l1 = s_ml[3 * WT_BN + row];
+      const float m0 = PAIR ? m_used : s_ml[row], l0 = PAIR ? l : s_ml[WT_BN + row];
+      const float m1 = PAIR ? -INFINITY : s_ml[2 * WT_BN + row], l1 = PAIR ? 0.f : s_ml[3 * WT_BN + row];
       const float sk = a.sink[head] * 1.4426950408889634f;
       const float m = fmaxf(sk, fmaxf(m0, m1));
       const float e0 = m0 == -INFINITY ? 0.f : exp2f(m0 - m), e1 = m1 == -INFINITY ? 0.f : exp2f(m1 - m);
@@ -265,9 +325,9 @@ __global__ void __launch_bounds__(WT_THREADS, 1) win_tc_kernel(const __grid_cons
       const float2* turn = reinterpret_cast<const float2*>(a.turn) + t * half;
       const bool vec = half % 16 == 0 && a.y_ld % 8 == 0 && a.gate_ld % 8 == 0 &&
                        ((reinterpret_cast<uintptr_t>(a.y) | reinterpret_cast<uintptr_t>(a.gate) | reinterpret_cast<uintptr_t>(a.turn)) & 15) == 0;
-      const uint32_t tO0 = tmem_base + 128 + lane_addr, tO1 = tO0 + 256;
+      const uint32_t tO0 = PAIR ? tO : tmem_base + 128 + lane_addr, tO1 = tO0 + 256;
 #pragma unroll 1
-      for (int c = x; c < (half + 15) / 16; c += 2) {    // each warpgroup takes every other 16 pairs
+      for (int c = PAIR ? 0 : x; c < (half + 15) / 16; c += PAIR ? 1 : 2) {    // one stream: the warpgroups take turns
         const int ca = INTER ? c * 32 : c * 16, cb = INTER ? ca + 16 : half + c * 16;
         float v[32];
         {
@@ -343,15 +403,19 @@ static int win_rows_map(CUtensorMap* tm, const void* base, long long width, long
   return make_tmap(tm, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, base, dims, strides, box);
 }
 
-template <bool INTER>
+template <bool INTER, bool PAIR, int NQ>
 static int launch_win_tc(const WinTcParams& p, int smem, cudaStream_t st) {
   static bool set = false;
   if (!set) {
-    if (cudaFuncSetAttribute(win_tc_kernel<INTER>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -10;
+    if (cudaFuncSetAttribute(win_tc_kernel<INTER, PAIR, NQ>, cudaFuncAttributeMaxDynamicSharedMemorySize, 227 * 1024) != cudaSuccess) return -10;
     set = true;
   }
-  win_tc_kernel<INTER><<<dim3(p.a.H, p.a.n_tiles), WT_THREADS, smem, st>>>(p);
+  win_tc_kernel<INTER, PAIR, NQ><<<dim3(PAIR ? p.a.H / 2 : p.a.H, p.a.n_tiles), WT_THREADS, smem, st>>>(p);
   return last_rc();
+}
+template <bool INTER, bool PAIR>
+static int pick_win_tc(const WinTcParams& p, int smem, cudaStream_t st) {
+  return p.nq == 1 ? launch_win_tc<INTER, PAIR, 1>(p, smem, st) : p.nq == 2 ? launch_win_tc<INTER, PAIR, 2>(p, smem, st) : launch_win_tc<INTER, PAIR, 0>(p, smem, st);
 }
 
 }  // namespace sx
@@ -375,9 +439,12 @@ extern "C" int sx_win_attn_tc(const SxWinAttnArgs* a, cudaStream_t st) {
   p.a = *a;
   p.rv = view(&a->ragged);
   p.scale_log2 = a->scale * 1.4426950408889634f;
-  const int held = p.nq * WT_SLICE, room = 227 * 1024 - held - 1024 - 256;    // alignment and barriers set aside
+  const bool pair = a->H / a->G % 2 == 0;
+  const int held = (pair ? 2 : 1) * p.nq * WT_SLICE, room = 227 * 1024 - held - 1024 - 256;    // alignment and barriers set aside
   p.stages = room / (2 * WT_SLICE);
   if (p.stages > WT_MAX_STAGES) p.stages = WT_MAX_STAGES;
+  if (p.stages < 1 + (p.nq + 1) / 2) return -4;          // a V tile and the next K tile are in the ring together
   const int smem = held + p.stages * 2 * WT_SLICE + 1024 + 256;
-  return a->interleaved ? launch_win_tc<true>(p, smem, st) : launch_win_tc<false>(p, smem, st);
+  if (pair) return a->interleaved ? pick_win_tc<true, true>(p, smem, st) : pick_win_tc<false, true>(p, smem, st);
+  return a->interleaved ? pick_win_tc<true, false>(p, smem, st) : pick_win_tc<false, false>(p, smem, st);
 }
