@@ -370,7 +370,10 @@ typedef struct SxSsdArgs {
   void* y; long long y_ld;        // [T, H P]
   SxRagged ragged;
   SxChunks chunks;
-  int* status;
+  // tensor-core prompt form with few sequences: portions cut into segments of seg_rows rows (a multiple of 64), or n_seg 0
+  const int* seg_seq; const int* seg_first;   // [n_seg] portion, [n + 1] first segment of each portion
+  float* seg_state; float* seg_la;            // scratch: [n_seg, H, N, P], [n_seg, H]
+  int n_seg, seg_rows;
   int T, H, P, N, G, taps, xp, np, f32;
 } SxSsdArgs;
 int sx_ssd_operands(const SxSsdArgs* args, cudaStream_t stream);   // u -> x, b, c, dt, la

@@ -123,7 +123,8 @@ class SxSsdArgs(C.Structure):
     _fields_ = [
         ("u", c_void_p), ("u_ld", c_ll), ("wconv", c_void_p), ("bconv", c_void_p), ("ring", c_void_p), ("dt_bias", c_void_p),
         ("a_log", c_void_p), ("D", c_void_p), ("x", c_void_p), ("b", c_void_p), ("c", c_void_p), ("dt", c_void_p), ("la", c_void_p),
-        ("state", c_void_p), ("y", c_void_p), ("y_ld", c_ll), ("ragged", SxRagged), ("chunks", SxChunks), ("status", c_void_p),
+        ("state", c_void_p), ("y", c_void_p), ("y_ld", c_ll), ("ragged", SxRagged), ("chunks", SxChunks),
+        ("seg_seq", c_void_p), ("seg_first", c_void_p), ("seg_state", c_void_p), ("seg_la", c_void_p), ("n_seg", c_int), ("seg_rows", c_int),
         ("T", c_int), ("H", c_int), ("P", c_int), ("N", c_int), ("G", c_int), ("taps", c_int), ("xp", c_int), ("np", c_int), ("f32", c_int),
     ]
 

@@ -165,7 +165,6 @@ def _ssd_args(u, wconv, bconv, ring, dt_bias, a_log, D, state, y, batch, H, P, N
     a.ragged = batch.struct()
     if not batch.decode:
         a.chunks = batch.chunks()
-    a.status = _lib.status_word(u.device).data_ptr()
     a.T, a.H, a.P, a.N, a.G, a.taps, a.xp, a.np, a.f32 = batch.T, H, P, N, G, taps, P, N, _f32(u)
     return a
 
@@ -196,6 +195,11 @@ def ssd_scan(operands, batch: RaggedBatch):
     read-outs."""
     a, (u, x, _, _, _, _, state, _, _) = operands
     if ssd_scan_tc(u.dtype, a.P, a.N):
+        if batch.n_segments > batch.n and batch.n * a.H * ((a.P + 63) // 64) < 2 * 148:    # two CTAs per SM
+            seg = torch.empty(batch.n_segments * a.H * (a.N * a.P + 1), dtype=torch.float32, device=u.device)
+            a.seg_seq, a.seg_first, a.seg_state = batch.seg_seq.data_ptr(), batch.seg_first.data_ptr(), seg.data_ptr()
+            a.seg_la = seg.data_ptr() + 4 * batch.n_segments * a.H * a.N * a.P
+            a.n_seg, a.seg_rows = batch.n_segments, batch.segment_rows
         _lib.call("sx_ssd_scan", C.byref(a), stream())
         return
     rec = _records(batch, a.H, a.N, False, u.device)

@@ -98,11 +98,12 @@ class RaggedBatch:
 
     @classmethod
     def prompt(cls, device, tokens: List[List[int]], pos0: List[int], slots: List[int], entries: List[List[int]],
-               earlier: Dict[object, List[List[int]]], want: List[int], tile_rows: int = 128, averages=None) -> "RaggedBatch":
+               earlier: Dict[object, List[List[int]]], want: List[int], tile_rows: int = 128, averages=None,
+               segment_rows: int = 512) -> "RaggedBatch":
         """``earlier[mask][i]``: cache entries of the positions before sequence i's portion that its first token still
         needs (a chunk length may stand for its mask). ``averages[mask][i]``: for masks that pool, the cache entries of the
         averaged blocks complete before the portion and of those that it completes. ``want``: rows whose logits are asked
-        for."""
+        for. ``segment_rows``: length of the segments that a scan may run side by side."""
         b = cls()
         b.n, b.T = len(tokens), sum(len(t) for t in tokens)
         lens = np.array([len(t) for t in tokens], dtype=np.int32)
@@ -122,6 +123,11 @@ class RaggedBatch:
         chunk_seq = np.repeat(np.arange(b.n, dtype=np.int32), per)
         parts += [chunk_seq, (np.arange(first[-1], dtype=np.int32) - first[chunk_seq]) * RECUR_CHUNK, first]
         b.n_chunks = int(first[-1])
+        per = (lens + segment_rows - 1) // segment_rows
+        seg_first = np.zeros(b.n + 1, dtype=np.int32)
+        np.cumsum(per, out=seg_first[1:])
+        parts += [np.repeat(np.arange(b.n, dtype=np.int32), per), seg_first]
+        b.n_segments, b.segment_rows = int(seg_first[-1]), segment_rows
         views, none = [], np.zeros(0, np.int32)
         cat = lambda xs: np.concatenate([np.asarray(x, dtype=np.int32) for x in xs]) if xs else none  # noqa: E731
         for key in earlier:
@@ -144,7 +150,8 @@ class RaggedBatch:
             views.append((key, int(start[-1]), int(n_new.sum())))
         dev = cls._upload(device, parts)
         b.ids, b.cu, b.pos0, b.slot, b.tok_seq, b.tok_pos, b.entry, b.want, tl, b.chunk_seq, b.chunk_start, b.chunk_first = dev[:12]
-        at = 12
+        b.seg_seq, b.seg_first = dev[12:14]
+        at = 14
         for key, rows, n_pool in views:
             v = b.views[key] = ChunkView(rows, *dev[at: at + 4], tl, len(tiles))
             at += 4

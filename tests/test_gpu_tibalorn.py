@@ -198,7 +198,8 @@ def test_recurrence_prompt_forms_and_steps_leave_the_same_state(P, N, G):
     y = y.reshape(T, -1) * oracle.silu(ud[:, :H * P])
     dev = lambda t: t.float().contiguous().cuda()  # noqa: E731
     ws = [dev(conv.T), dev(cb)], [dev(dtb), dev(al), dev(D)]
-    for dtype, cuts in ((BF16, [150]), (F32, [150]), (BF16, [64, 1, 2, 60, 23]), (F32, [1] * 20 + [130]), (BF16, [1] * 150)):
+    for dtype, cuts, seg in ((BF16, [150], 512), (F32, [150], 512), (BF16, [64, 1, 2, 60, 23], 512), (F32, [1] * 20 + [130], 512),
+                             (BF16, [1] * 150, 512), (BF16, [150], 64), (BF16, [2, 128, 20], 64), (BF16, [10, 140], 128)):
         ring, state = torch.full((2, taps, c), float("nan"), dtype=dtype, device="cuda"), torch.full((2, H, N, P), float("nan"), device="cuda")
         out, at = [], 0
         for n in cuts:
@@ -209,7 +210,7 @@ def test_recurrence_prompt_forms_and_steps_leave_the_same_state(P, N, G):
                 RaggedBatch.fill_decode(buf.numpy(), 1, 0, [0], [at], [1], [-1], [[]], [0])
                 hybrid.ssd_step(rows, *ws[0], ring, *ws[1], state, o, RaggedBatch.decode_views(buf.cuda(), 1, 0), H, P, N, G, taps)
             else:
-                b = RaggedBatch.prompt("cuda", [[0] * n], [at], [1], [[-1] * n], {}, [0])
+                b = RaggedBatch.prompt("cuda", [[0] * n], [at], [1], [[-1] * n], {}, [0], segment_rows=seg)
                 hybrid.ssd_prompt(rows, *ws[0], ring, *ws[1], state, o, b, H, P, N, G, taps)
             out.append(o.double().cpu())
             at += n
@@ -219,6 +220,27 @@ def test_recurrence_prompt_forms_and_steps_leave_the_same_state(P, N, G):
         assert float((state[1].double().cpu() - S).abs().max()) < (1e-5 if dtype == F32 else 8e-3) * float(S.abs().max())
         assert torch.isnan(state[0]).all()
     check_status()
+
+
+def test_segments_of_several_sequences_run_side_by_side():
+    """Unequal portions, some of one segment, one that goes on from a stored state: the same as without segments."""
+    H, P, N, G, taps = 2, 40, 24, 1, 3
+    c = H * P + 2 * G * N
+    lens, pos0 = [300, 64, 65, 1, 190], [0, 7, 0, 12, 90]
+    g = torch.Generator().manual_seed(1)
+    u = torch.randn(sum(lens), (H * P + c + H + 7) // 8 * 8, generator=g).bfloat16().cuda()[:, :H * P + c + H]
+    w = [torch.randn(taps, c, generator=g).cuda() * 0.4, torch.randn(c, generator=g).cuda() * 0.2]
+    v = [torch.randn(H, generator=g).cuda() - 2, torch.randn(H, generator=g).cuda() * 0.5 - 1, torch.randn(H, generator=g).cuda()]
+    S0, R0 = torch.randn(5, H, N, P, generator=g), torch.randn(5, taps, c, generator=g).bfloat16()
+    out = []
+    for seg in (512, 64, 128):
+        state, y = S0.cuda(), torch.empty(sum(lens), H * P, dtype=BF16, device="cuda")
+        b = RaggedBatch.prompt("cuda", [[0] * n for n in lens], pos0, [4, 0, 2, 1, 3], [[-1] * n for n in lens], {}, [0], segment_rows=seg)
+        hybrid.ssd_prompt(u, *w, R0.cuda(), *v, state, y, b, H, P, N, G, taps)
+        out.append((y.double(), state.double()))
+    assert b.n_segments == 3 + 1 + 1 + 1 + 2
+    for y, state in out[1:]:
+        assert torch.allclose(state, out[0][1], atol=2e-4, rtol=2e-4) and torch.allclose(y, out[0][0], atol=2e-2, rtol=2e-2)
 
 
 # ------------------------------------------------------------------ visibility of single keys and blocks
