@@ -25,7 +25,7 @@ def _tibalorn_fields(d: Dict[str, Any]) -> Dict[str, Any]:
     """The keys of a Tibalorn ``config.json`` under this schema's names; other keys pass through."""
     out = {k: v for k, v in d.items() if k not in ("layers", "vocab", "width", "norm", "embedding")}
     out.update(architecture="tibalorn", layer_specs=d["layers"], vocab_size=d["vocab"], hidden_size=d["width"],
-               layer_norm_eps=d["norm"]["eps"], num_hidden_layers=len(d["layers"]), embedding_scale=d["embedding"]["scale"],
+               layer_norm_eps=d["norm"]["eps"], num_hidden_layers=len(d["layers"]), embedding_scale=d.get("embedding", {}).get("scale", 1.0),
                tie_word_embeddings=True, use_rms_norm=False)
     return out
 
