@@ -195,7 +195,8 @@ def ssd_scan(operands, batch: RaggedBatch):
     read-outs."""
     a, (u, x, _, _, _, _, state, _, _) = operands
     if ssd_scan_tc(u.dtype, a.P, a.N):
-        if batch.n_segments > batch.n and batch.n * a.H * ((a.P + 63) // 64) < 2 * 148:    # two CTAs per SM
+        # segments cost a pass over the states: worth it while one CTA per portion and head leaves a third of the SMs idle
+        if batch.n_segments > batch.n and batch.n * a.H * ((a.P + 63) // 64) <= 100:
             seg = torch.empty(batch.n_segments * a.H * (a.N * a.P + 1), dtype=torch.float32, device=u.device)
             a.seg_seq, a.seg_first, a.seg_state = batch.seg_seq.data_ptr(), batch.seg_first.data_ptr(), seg.data_ptr()
             a.seg_la = seg.data_ptr() + 4 * batch.n_segments * a.H * a.N * a.P
