@@ -82,7 +82,7 @@ def test_activations_match_their_definitions():
     assert float(oracle.softcap(z, 2.5).abs().max()) <= 2.5
 
 
-@pytest.mark.parametrize("dims,base,scaling", [(8, 500.0, None), (16, 1e4, yarn(4.0, 64, 6.0, 1.0)), (64, 2.5e5, yarn(8.0, 2048, 32.0, 1.0)),
+@pytest.mark.parametrize("dims,base,scaling", [(8, 500.0, None), (16, 1e4, yarn(4.0, 64, 6.0, 1.0)), (64, 3e5, yarn(6.0, 4096, 24.0, 1.5)),
                                                (32, 1e4, yarn(16.0, 128, 64.0, 32.0)), (6, 1e4, yarn(2.0, 10 ** 9, 1e-3, 1e-4)), (0, 1e4, None)])
 def test_rotary_frequencies(dims, base, scaling):
     f, mul = rotary_frequencies(dims, base, scaling)
